@@ -196,6 +196,31 @@ int litnice_b200_session_create(const litnice_b200_dims *dims, int32_t max_strea
  * session's device first, so a session may be driven from any one thread at a time. */
 int litnice_b200_session_create_on(const litnice_b200_dims *dims, int32_t max_streams, int32_t device,
                                    litnice_b200_session **out);
+/* A session on a model folder (config.json + model.safetensors) of one of the registered decoder
+ * designs, weights loaded. config.json's "architecture" names the design; the names known are
+ * litnice_b200_architectures(), with commas between them. dtype: LITNICE_B200_DTYPE_BF16 (bfloat16
+ * weights and matrix products with 32-bit accumulation; norms, attention scores and weights, the
+ * residual stream and state in 32-bit) or LITNICE_B200_DTYPE_F32 (everything in 32-bit). device:
+ * CUDA ordinal, negative for LITNICE_B200_DEVICE or the current device. Such a session keeps its
+ * caches and state in max_streams slots and serves generate / upload_prompts / run /
+ * download_tokens, forward, inspect and sample_logits like any other (a step computes the new rows
+ * only), and extend / release below. On failure *out may be null; litnice_b200_last_error(NULL)
+ * then has the reason. */
+#define LITNICE_B200_DTYPE_BF16 0
+#define LITNICE_B200_DTYPE_F32 1
+int litnice_b200_session_create_model(const char *model_dir, int32_t dtype, int32_t max_streams, int32_t device,
+                                      litnice_b200_session **out);
+const char *litnice_b200_architectures(void);
+/* Sizes of the session's model (n_layers, d_model, vocab_size and max_seq_len for a registered design). */
+int litnice_b200_model_dims(const litnice_b200_session *s, litnice_b200_dims *out);
+/* Appends n tokens to the sequence in a slot (0 .. max_streams - 1; empty at first) and computes
+ * their rows from the cache and state that earlier calls left. want: places 0 .. n-1 among the new
+ * tokens whose logits go to out_logits [n_want, vocab] (host), in that order. Portions may be cut
+ * anywhere. On failure the slot is empty. Sessions of registered designs only. */
+int litnice_b200_extend(litnice_b200_session *s, int32_t slot, const int32_t *tokens, int32_t n, const int32_t *want,
+                        int32_t n_want, float *out_logits);
+/* Gives a slot back: its next extend starts a new sequence. */
+int litnice_b200_release(litnice_b200_session *s, int32_t slot);
 void litnice_b200_session_destroy(litnice_b200_session *s);
 const char *litnice_b200_last_error(const litnice_b200_session *s);
 
@@ -331,6 +356,30 @@ int litnice_b200_gemv_host(const float *x, int32_t m, const float *w, int32_t k,
  * microseconds per call; *launches: kernels per call. */
 int litnice_b200_gemv_time(int32_t m, int32_t k, int32_t n, int32_t repeats, int32_t cold_l2,
                            int32_t force_tn, int32_t force_splits, double *avg_us, int32_t *launches);
+
+/* Single operators of the registered designs on host float buffers (rounded to bfloat16 where the
+ * operator stores bfloat16); see csrc/model.cuh for what each computes. They allocate and free
+ * their own device memory.
+ *
+ * c[m, n] = a[m, k] w[n, k]^T on bfloat16 operands. engine 0: few-row kernel (m <= 64), 1: tensor-core
+ * kernel. Columns below n_half come back rounded to bfloat16 (through GELU when gelu is set), the
+ * others as floats, added to what c holds when accumulate is set. */
+int litnice_b200_bf16_product_host(int32_t engine, const float *a, int32_t m, int32_t k, const float *w, int32_t n,
+                                   int32_t n_half, int32_t gelu, int32_t accumulate, float *c);
+/* h = x / sqrt(mean(x^2) + eps) * gain for the rows of one sequence, out_i = h + conv_i(h) with the causal
+ * per-channel convolutions w_i [d, taps] (w2 and out2 both or neither), computed in the given portions
+ * with the state carried between them. */
+int litnice_b200_rms_canon_host(int32_t dtype, const float *x, int32_t n, int32_t d, float gain, float eps, int32_t taps,
+                                const float *w1, const float *w2, const int32_t *portions, int32_t n_portions, float *out1,
+                                float *out2);
+/* Latent attention of the rows p0 .. p0 + n - 1 of n_streams sequences: q [n_streams, n, heads * dim],
+ * dkv [n_streams, p0 + n, rank] (normalised into the cache with latent_gain and eps), w_uk
+ * [heads * dim, rank], w_uv [heads * vdim, rank], out [n_streams, n, heads * vdim]. engine 0: any size
+ * in 32-bit, 1: the same on bfloat16 storage, 2: few-row kernels, 3: tensor-core kernel. */
+int litnice_b200_latent_attention_host(int32_t engine, const float *q, const float *dkv, const float *latent_gain,
+                                       float eps, const float *w_uk, const float *w_uv, int32_t n_streams, int32_t p0,
+                                       int32_t n, int32_t heads, int32_t dim, int32_t vdim, int32_t rank, float scale,
+                                       int32_t window, float *out);
 
 /* Self-test of the bounded waits: a one-CTA kernel waits on a barrier that nothing
  * completes, with a limit of limit_us microseconds (1..1000). It must come back on

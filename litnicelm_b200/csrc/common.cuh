@@ -35,6 +35,7 @@ enum DevErrCode : int {
   DEVERR_WAIT_TIMEOUT = 2,   // a bounded mbarrier / TMEM wait ran out
   DEVERR_BAD_ARGUMENT = 3,
   DEVERR_BAD_TARGET = 4,     // cross-entropy target outside [0, vocab)
+  DEVERR_NON_FINITE = 5,     // a weight is NaN or infinite
 };
 struct DevErr {
   int code;

@@ -11,6 +11,10 @@
 //                            [--max_new N] [--temp T] [--top_k K] [--top_p P] [--seed S]
 //                            [--streams N] [--gpus G] [--out-ids-file out.i32]
 //   litnice_b200_run inspect --config cfg.yaml [--prompt TEXT | --ids-file ids.i32]
+//   litnice_b200_run infer|inspect --model DIR [--dtype bfloat16|float32] [--library LIB.so]
+//                            --ids 1,2,3 | --ids-file ids.i32   [the options of infer above]
+//   litnice_b200_run trace   --model DIR --dtype bfloat16|float32 --out DIR [--max-tokens N] [--library LIB.so]
+//   litnice_b200_run designs [--library LIB.so]           (architectures the library serves)
 //   litnice_b200_run partition --streams N --gpus G      (prints the split; needs no GPU)
 //
 // --ids-file holds int32 token ids, streams*len of them (row-major); with
@@ -18,7 +22,16 @@
 // With --gpus G the streams are cut into G contiguous blocks, one host thread
 // per GPU decodes its block on its own session (weights replicated, nothing is
 // exchanged between GPUs), and the threads are joined before anything is printed.
+//
+// --model serves a folder with config.json and model.safetensors of a registered design
+// (litnice_b200_session_create_model) instead of a litnicelm checkpoint; it has no
+// tokenizer, so prompts are token ids and text is printed as ids. `trace` replays
+// given token ids: one JSON step per line of standard input,
+//   {"step": 0, "entries": [{"id": "a", "tokens": [5, 17], "want": [0, 1]}], "end": ["a"]}
+// feeds each entry's tokens to its sequence, writes the logits of the wanted places to
+// DIR/<step>.f32 (little-endian floats, [wanted, vocab]) and answers "done <step>".
 #include <dlfcn.h>
+#include <unistd.h>
 
 #include <algorithm>
 #include <cmath>
@@ -26,6 +39,7 @@
 #include <cstdio>
 #include <cstring>
 #include <fstream>
+#include <functional>
 #include <iomanip>
 #include <iostream>
 #include <map>
@@ -37,6 +51,7 @@
 #include <vector>
 
 #include "../../../include/litnice_backend_b200.h"
+#include "../json.hpp"
 
 namespace {
 
@@ -197,6 +212,11 @@ struct Api {
   decltype(&litnice_b200_inspect) inspect = nullptr;
   decltype(&litnice_b200_forward) forward = nullptr;
   decltype(&litnice_b200_get_stats) get_stats = nullptr;
+  decltype(&litnice_b200_session_create_model) create_model = nullptr;
+  decltype(&litnice_b200_architectures) architectures = nullptr;
+  decltype(&litnice_b200_model_dims) model_dims = nullptr;
+  decltype(&litnice_b200_extend) extend = nullptr;
+  decltype(&litnice_b200_release) release = nullptr;
 
   explicit Api(const std::string &path) {
     handle = dlopen(path.c_str(), RTLD_NOW | RTLD_LOCAL);
@@ -213,9 +233,109 @@ struct Api {
     RESOLVE(inspect, "litnice_b200_inspect");
     RESOLVE(forward, "litnice_b200_forward");
     RESOLVE(get_stats, "litnice_b200_get_stats");
+    RESOLVE(create_model, "litnice_b200_session_create_model");
+    RESOLVE(architectures, "litnice_b200_architectures");
+    RESOLVE(model_dims, "litnice_b200_model_dims");
+    RESOLVE(extend, "litnice_b200_extend");
+    RESOLVE(release, "litnice_b200_release");
 #undef RESOLVE
   }
 };
+
+// The library beside this program, where no YAML names one.
+std::string default_library() {
+  char buf[4096];
+  const ssize_t n = readlink("/proc/self/exe", buf, sizeof(buf) - 1);
+  std::string dir = n > 0 ? std::string(buf, (size_t)n) : std::string("./x");
+  return dir.substr(0, dir.rfind('/') + 1) + "liblitnice_backend_b200.so";
+}
+
+int parse_dtype(const std::map<std::string, std::string> &opt) {
+  auto it = opt.find("--dtype");
+  if (it == opt.end() || it->second == "bfloat16") return LITNICE_B200_DTYPE_BF16;
+  if (it->second == "float32") return LITNICE_B200_DTYPE_F32;
+  throw std::runtime_error("--dtype must be bfloat16 or float32");
+}
+
+std::vector<int32_t> parse_ids(const std::string &text) {
+  std::vector<int32_t> ids;
+  std::string t = text;
+  std::replace(t.begin(), t.end(), ',', ' ');
+  std::istringstream in(t);
+  long long v;
+  while (in >> v) ids.push_back((int32_t)v);
+  if (!in.eof() || ids.empty()) throw std::runtime_error("--ids wants token ids with commas between them");
+  return ids;
+}
+
+// Replays steps of given token ids through one model. Sequences live in slots; a slot is given back
+// when its sequence ends.
+int trace(Api &api, const std::map<std::string, std::string> &opt) {
+  constexpr int kSlots = 16;
+  const std::string out_dir = opt.at("--out");
+  litnice_b200_session *s = nullptr;
+  int rc = api.create_model(opt.at("--model").c_str(), parse_dtype(opt), kSlots, -1, &s);
+  auto check = [&](int code, const char *what) {
+    if (code == LITNICE_B200_OK) return;
+    const std::string msg = std::string(what) + " failed (" + std::to_string(code) + "): " + api.last_error(s);
+    if (s) api.destroy(s);
+    throw std::runtime_error(msg);
+  };
+  check(rc, "session_create_model");
+  litnice_b200_dims d{};
+  check(api.model_dims(s, &d), "model_dims");
+  std::map<std::string, int> slot_of;
+  std::vector<bool> used(kSlots, false);
+  std::string line;
+  std::vector<int32_t> tokens, want;
+  std::vector<float> logits;
+  while (std::getline(std::cin, line)) {
+    if (trim(line).empty()) continue;
+    const lb::Json step = lb::Json::parse(line);
+    const long long number = step.at("step").as_int();
+    logits.clear();
+    for (const lb::Json &e : step.at("entries").as_array()) {
+      const std::string &id = e.at("id").as_string();
+      auto it = slot_of.find(id);
+      if (it == slot_of.end()) {
+        int slot = 0;
+        while (slot < kSlots && used[(size_t)slot]) ++slot;
+        if (slot == kSlots) throw std::runtime_error("more than " + std::to_string(kSlots) + " live sequences");
+        used[(size_t)slot] = true;
+        it = slot_of.emplace(id, slot).first;
+      }
+      tokens.clear();
+      want.clear();
+      for (const lb::Json &t : e.at("tokens").as_array()) tokens.push_back((int32_t)t.as_int());
+      if (e.has("want"))
+        for (const lb::Json &w : e.at("want").as_array()) want.push_back((int32_t)w.as_int());
+      if (tokens.empty()) continue;
+      const size_t at = logits.size();
+      logits.resize(at + want.size() * (size_t)d.vocab_size);
+      check(api.extend(s, it->second, tokens.data(), (int32_t)tokens.size(), want.empty() ? nullptr : want.data(),
+                       (int32_t)want.size(), want.empty() ? nullptr : logits.data() + at),
+            "extend");
+    }
+    if (step.has("end"))
+      for (const lb::Json &e : step.at("end").as_array()) {
+        auto it = slot_of.find(e.as_string());
+        if (it == slot_of.end()) continue;
+        check(api.release(s, it->second), "release");
+        used[(size_t)it->second] = false;
+        slot_of.erase(it);
+      }
+    if (!logits.empty()) {
+      const std::string path = out_dir + "/" + std::to_string(number) + ".f32";
+      std::ofstream o(path, std::ios::binary | std::ios::trunc);
+      o.write(reinterpret_cast<const char *>(logits.data()), (std::streamsize)(logits.size() * sizeof(float)));
+      o.close();
+      if (!o) throw std::runtime_error("cannot write " + path);
+    }
+    std::cout << "done " << number << std::endl;
+  }
+  api.destroy(s);
+  return 0;
+}
 
 int run(int argc, char **argv) {
   if (argc < 2) throw std::runtime_error("usage: litnice_b200_run infer|inspect --config cfg.yaml [...]");
@@ -232,19 +352,40 @@ int run(int argc, char **argv) {
     }
     return 0;
   }
-  if (!opt.count("--config")) throw std::runtime_error("--config is required");
-  auto cfg = parse_yaml(opt["--config"]);
+  const std::string library = opt.count("--library") ? opt["--library"] : default_library();
+  if (mode == "designs") {
+    std::cout << Api(library).architectures() << "\n";
+    return 0;
+  }
+  if (mode == "trace") {
+    if (!opt.count("--model") || !opt.count("--out")) throw std::runtime_error("trace needs --model and --out");
+    parse_dtype(opt);
+    Api api(library);
+    return trace(api, opt);
+  }
+  const bool folder = opt.count("--model") != 0;  // a registered design instead of a litnicelm checkpoint
+  if (!folder && !opt.count("--config")) throw std::runtime_error("--config is required");
+  std::map<std::string, std::string> cfg;
+  if (folder)
+    cfg = {{"inference.prompt", ""}, {"inference.max_new", "16"}, {"inference.temp", "0"}, {"inference.top_k", "0"},
+           {"inference.top_p", "1"}, {"inference.seed", "12345"}, {"backend.library", library}};
+  else
+    cfg = parse_yaml(opt["--config"]);
   auto get = [&](const char *flag, const char *key) { return opt.count(flag) ? opt[flag] : cfg.at(key); };
 
-  Tokenizer tok = make_tokenizer(cfg);
+  Tokenizer tok;
+  if (!folder) tok = make_tokenizer(cfg);
+  auto token_text = [&](int32_t id) { return folder ? " " + std::to_string(id) : tok.decode(id); };
   litnice_b200_dims d{};
-  d.n_layers = std::stoi(cfg.at("model.n_layers"));
-  d.n_heads = std::stoi(cfg.at("model.n_heads"));
-  d.d_model = std::stoi(cfg.at("model.d_model"));
-  d.d_ff = std::stoi(cfg.at("model.d_ff"));
-  d.max_seq_len = std::stoi(cfg.at("model.max_seq_len"));
-  d.vocab_size = tok.vocab;  // model.target_vocab_size follows the tokenizer (inference.cpp:64-65)
-  d.alignment_bytes = std::stoull(cfg.at("memory.alignment_bytes"));
+  if (!folder) {
+    d.n_layers = std::stoi(cfg.at("model.n_layers"));
+    d.n_heads = std::stoi(cfg.at("model.n_heads"));
+    d.d_model = std::stoi(cfg.at("model.d_model"));
+    d.d_ff = std::stoi(cfg.at("model.d_ff"));
+    d.max_seq_len = std::stoi(cfg.at("model.max_seq_len"));
+    d.vocab_size = tok.vocab;  // model.target_vocab_size follows the tokenizer (inference.cpp:64-65)
+    d.alignment_bytes = std::stoull(cfg.at("memory.alignment_bytes"));
+  }
 
   const std::string prompt = get("--prompt", "inference.prompt");
   const int max_new = std::stoi(get("--max_new", "inference.max_new"));
@@ -264,6 +405,10 @@ int run(int argc, char **argv) {
     in.seekg(0);
     ids.resize((size_t)n / 4);
     in.read(reinterpret_cast<char *>(ids.data()), n);
+  } else if (folder) {
+    if (!opt.count("--ids")) throw std::runtime_error("--model needs --ids or --ids-file");
+    const std::vector<int32_t> one = parse_ids(opt["--ids"]);
+    for (int i = 0; i < streams; ++i) ids.insert(ids.end(), one.begin(), one.end());
   } else {
     ids = tok.encode(prompt);
     if (ids.empty()) ids.push_back(0);  // inference.cpp:121-123
@@ -275,7 +420,20 @@ int run(int argc, char **argv) {
 
   Api api(cfg.at("backend.library"));
   std::cout << "[DeviceBackend] Loaded backend library: " << cfg.at("backend.library") << " (native loop)\n";
-  const std::string ckpt = cfg.at("paths.model_file_best");
+  const std::string ckpt = folder ? opt["--model"] : cfg.at("paths.model_file_best");
+  const int dtype = parse_dtype(opt);
+  // A session for n streams with its weights; device < 0 leaves the choice to the library.
+  auto open_session = [&](int n, int device, litnice_b200_session **out, const char **what) {
+    if (folder) {
+      *what = "session_create_model";
+      return api.create_model(ckpt.c_str(), dtype, n, device, out);
+    }
+    *what = "session_create";
+    const int code = device < 0 ? api.create(&d, n, out) : api.create_on(&d, n, device, out);
+    if (code != LITNICE_B200_OK) return code;
+    *what = "load_checkpoint";
+    return api.load_checkpoint(*out, ckpt.c_str());
+  };
 
   if (mode == "infer" && gpus > 1) {
     // One host thread per GPU, each with its own session and its own block of streams.
@@ -298,10 +456,9 @@ int run(int argc, char **argv) {
                               "): " + api.last_error(ws);
           if (ws) api.destroy(ws);
         };
-        int rc = api.create_on(&d, n, g, &ws);
-        if (rc != LITNICE_B200_OK) return fail("session_create", rc);
-        rc = api.load_checkpoint(ws, ckpt.c_str());
-        if (rc != LITNICE_B200_OK) return fail("load_checkpoint", rc);
+        const char *what = "";
+        int rc = open_session(n, g, &ws, &what);
+        if (rc != LITNICE_B200_OK) return fail(what, rc);
         rc = api.generate(ws, ids.data() + (size_t)first * len, n, len, max_new, &sp, seeds.data() + first,
                           out.data() + (size_t)first * std::max(1, max_new), &counts[(size_t)g]);
         if (rc != LITNICE_B200_OK) return fail("generate", rc);
@@ -321,8 +478,8 @@ int run(int argc, char **argv) {
                                  " GPUs, max_new=" + std::to_string(max_new));
     for (int b = 0; b < streams; ++b) {
       std::string text;
-      for (int i = 0; i < len; ++i) text += tok.decode(ids[(size_t)b * len + i]);
-      for (int i = 0; i < count; ++i) text += tok.decode(out[(size_t)b * max_new + i]);
+      for (int i = 0; i < len; ++i) text += token_text(ids[(size_t)b * len + i]);
+      for (int i = 0; i < count; ++i) text += token_text(out[(size_t)b * max_new + i]);
       if (b == 0) report("END", (uint32_t)(len + count), 0.0f, "Inference complete");
       report("TOKEN_GEN", 0, 0.0f, text);
     }
@@ -340,7 +497,8 @@ int run(int argc, char **argv) {
   }
 
   litnice_b200_session *s = nullptr;
-  int rc = api.create(&d, streams, &s);
+  const char *what = "";
+  const int rc = open_session(streams, -1, &s, &what);
   auto check = [&](int code, const char *what) {
     if (code != LITNICE_B200_OK) {
       const std::string msg = std::string(what) + " failed (" + std::to_string(code) + "): " + api.last_error(s);
@@ -348,8 +506,8 @@ int run(int argc, char **argv) {
       throw std::runtime_error(msg);
     }
   };
-  check(rc, "session_create");
-  check(api.load_checkpoint(s, ckpt.c_str()), "load_checkpoint");
+  check(rc, what);
+  if (folder) check(api.model_dims(s, &d), "model_dims");
 
   if (mode == "infer") {
     std::ostringstream start;
@@ -363,13 +521,13 @@ int run(int argc, char **argv) {
     check(api.generate(s, ids.data(), streams, len, max_new, &sp, seeds.data(), out.data(), &count), "generate");
     for (int b = 0; b < streams; ++b) {
       std::string text;
-      for (int i = 0; i < len; ++i) text += tok.decode(ids[(size_t)b * len + i]);
+      for (int i = 0; i < len; ++i) text += token_text(ids[(size_t)b * len + i]);
       for (int i = 0; i < count; ++i) {
         const int32_t t = out[(size_t)b * max_new + i];
         if (streams == 1)
           report("TOKEN_GEN", (uint32_t)i + 1, (float)t,
-                 "Generated token id=" + std::to_string(t) + " token=\"" + escape_for_log(tok.decode(t)) + "\"");
-        text += tok.decode(t);
+                 "Generated token id=" + std::to_string(t) + " token=\"" + escape_for_log(token_text(t)) + "\"");
+        text += token_text(t);
       }
       if (b == 0) report("END", (uint32_t)(len + count), 0.0f, "Inference complete");
       report("TOKEN_GEN", 0, 0.0f, text);
@@ -397,13 +555,13 @@ int run(int argc, char **argv) {
       if (probs[(size_t)i] > 0.0f) entropy -= (double)probs[(size_t)i] * std::log((double)probs[(size_t)i]);
     std::ostringstream oss;
     oss << "[INFERENCE][INSPECT] Prompt=\"" << prompt << "\"\n";
-    oss << "Argmax: id=" << order.front() << " token=\"" << tok.decode(order.front()) << "\"\n";
+    oss << "Argmax: id=" << order.front() << " token=\"" << token_text(order.front()) << "\"\n";
     oss << "Entropy: " << std::fixed << std::setprecision(6) << entropy << "\n";
     const size_t top = std::min<size_t>(5, order.size());
     oss << "Top-" << top << " next-token distribution:\n";
     for (size_t i = 0; i < top; ++i) {
       const int32_t id = order[i];
-      oss << (i + 1) << ". id=" << id << " token=\"" << tok.decode(id) << "\" logit=" << std::fixed
+      oss << (i + 1) << ". id=" << id << " token=\"" << token_text(id) << "\" logit=" << std::fixed
           << std::setprecision(6) << logits[(size_t)id] << " prob=" << probs[(size_t)id] << "\n";
     }
     report("TOKEN_GEN", 0, 0.0f, oss.str());

@@ -5,6 +5,9 @@
 // launch sized for an upper bound `s_cap` serves every shorter context.
 #include "common.cuh"
 #include "gemm_tc.cuh"
+#include "model.cuh"
+
+#include <cuda_bf16.h>
 
 namespace lb {
 
@@ -124,6 +127,28 @@ __global__ void advance_state_kernel(LoopState *state) {
   state->step += 1;
 }
 
+// The rows of a batch (new positions only): x[r, :] = table[ids[slot, p]] + pos[p], in 32-bit.
+template <typename T>
+__global__ void embed_rows_kernel(const T *__restrict__ table, const T *__restrict__ pos, const int *__restrict__ ids,
+                                  int ids_ld, const LoopState *state, int p0_host, int n, int slot0, int d, int vocab,
+                                  float *__restrict__ x, DevErr *err) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.y, t = blockIdx.x;
+  const int p = (state ? state->s - n : p0_host) + t;
+  int id = ids[(long long)(slot0 + b) * ids_ld + p];
+  if (id < 0 || id >= vocab) {
+    if (threadIdx.x == 0) {
+      err->code = DEVERR_BAD_TOKEN_ID;
+      err->detail = id;
+    }
+    id = 0;
+  }
+  const T *tp = table + (long long)id * d, *pp = pos + (long long)p * d;
+  float *xp = x + ((long long)b * n + t) * d;
+  for (int c = threadIdx.x; c < d; c += blockDim.x) xp[c] = (float)tp[c] + (float)pp[c];
+}
+
 }  // namespace
 
 void launch_embed_pos(const float *tok_emb, const float *pos_emb, const int *ids, int ids_ld,
@@ -146,6 +171,18 @@ void launch_gather_last_ln(const float *x, const float *gamma, const float *beta
 
 void launch_advance_state(LoopState *state, cudaStream_t st) {
   launch_pdl(advance_state_kernel, dim3(1), dim3(1), 0, st, g_pdl_enabled, state);
+}
+
+void launch_embed_rows(const void *table, const void *pos, Precision type, const RowBatch &b, int d, int vocab, float *x,
+                       cudaStream_t st, DevErr *err) {
+  const dim3 grid((unsigned)b.n, (unsigned)b.streams);
+  if (type == Precision::BF16)
+    launch_pdl(embed_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, g_pdl_enabled,
+               static_cast<const __nv_bfloat16 *>(table), static_cast<const __nv_bfloat16 *>(pos), b.ids, b.ids_ld, b.state,
+               b.p0, b.n, b.slot0, d, vocab, x, err);
+  else
+    launch_pdl(embed_rows_kernel<float>, grid, dim3(256), 0, st, g_pdl_enabled, static_cast<const float *>(table),
+               static_cast<const float *>(pos), b.ids, b.ids_ld, b.state, b.p0, b.n, b.slot0, d, vocab, x, err);
 }
 
 }  // namespace lb

@@ -1,0 +1,137 @@
+// Few-row products on bfloat16 weights: C[m, n] = A[m, k] W[n, k]^T for m <= 64 rows, bound by the
+// bytes of W, which every launch reads once.
+//
+// W rows are the M side of mma.sync m16n8k16 tiles and the activation rows the N side, so one
+// instruction serves 16 output columns and 8 rows. A CTA owns 16 rows of W and all of k; its eight
+// warps take interleaved blocks of 64 k, and their sums meet in shared memory. The order of k inside a
+// dot product is free, so a lane loads 16 consecutive bytes (8 k) of its W row and of its activation
+// row and feeds them to two k-steps as they lie: no shared memory, no shuffles, whole 128-byte lines
+// of W per warp and row. Up to two products with inputs of their own share a launch.
+#include "model.cuh"
+
+#include <cuda_bf16.h>
+
+namespace lb {
+
+namespace {
+
+typedef __nv_bfloat16 bf16;
+
+constexpr int FR_WARPS = 8;
+constexpr int FR_COLS = 16;  // rows of W (output columns) per CTA
+
+struct FewRowPair {
+  Bf16Product p[2];
+  int blocks0;  // CTAs of the first product
+};
+
+__device__ __forceinline__ void fr_mma(float (&d)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3, unsigned b0,
+                                       unsigned b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint4 ld_stream(const bf16 *p) {  // weights: read once per launch
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];"
+               : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
+               : "l"(p));
+  return v;
+}
+
+// NT: tiles of 8 activation rows; UNROLL: blocks of 32 k in flight per lane and row.
+template <int NT, int UNROLL>
+__global__ void __launch_bounds__(FR_WARPS * 32)
+few_row_bf16_kernel(FewRowPair pair, int m) {
+  __shared__ float red[FR_WARPS][NT][FR_COLS][8];
+  const bool second = (int)blockIdx.x >= pair.blocks0;
+  const Bf16Product &p = pair.p[second ? 1 : 0];
+  const int n0 = ((int)blockIdx.x - (second ? pair.blocks0 : 0)) * FR_COLS;
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+  const int k8 = (p.k + 7) & ~7;  // rows end on a multiple of 8, zeros behind k
+  const bf16 *w = static_cast<const bf16 *>(p.w), *a = static_cast<const bf16 *>(p.a);
+  const bool v0 = n0 + g < p.n, v1 = n0 + g + 8 < p.n;
+  const bf16 *w0 = w + (long long)(n0 + g) * p.w_ld + t * 8, *w1 = w0 + (long long)8 * p.w_ld;
+  constexpr int SPAN = 32 * UNROLL;  // k per warp and trip
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  uint4 wa[UNROLL], wb[UNROLL];
+  auto load_w = [&](int k0) {
+#pragma unroll
+    for (int u = 0; u < UNROLL; ++u) {
+      const int k = k0 + u * 32;
+      const bool in = k + t * 8 < k8;
+      wa[u] = in && v0 ? ld_stream(w0 + k) : zero;
+      wb[u] = in && v1 ? ld_stream(w1 + k) : zero;
+    }
+  };
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  pdl_launch_dependents();
+  load_w(wid * SPAN);  // the weights do not depend on the predecessor
+  pdl_wait();
+  for (int k0 = wid * SPAN; k0 < k8; k0 += FR_WARPS * SPAN) {
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int row = i * 8 + g;
+      const bf16 *ar = a + (long long)row * p.a_ld + t * 8;
+      uint4 x[UNROLL];
+#pragma unroll
+      for (int u = 0; u < UNROLL; ++u) {
+        const int k = k0 + u * 32;
+        x[u] = row < m && k + t * 8 < k8 ? *reinterpret_cast<const uint4 *>(ar + k) : zero;
+      }
+#pragma unroll
+      for (int u = 0; u < UNROLL; ++u) {
+        fr_mma(acc[i], wa[u].x, wb[u].x, wa[u].y, wb[u].y, x[u].x, x[u].y);
+        fr_mma(acc[i], wa[u].z, wb[u].z, wa[u].w, wb[u].w, x[u].z, x[u].w);
+      }
+    }
+    if (k0 + FR_WARPS * SPAN < k8) load_w(k0 + FR_WARPS * SPAN);
+  }
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    *reinterpret_cast<float2 *>(&red[wid][i][g][t * 2]) = make_float2(acc[i][0], acc[i][1]);
+    *reinterpret_cast<float2 *>(&red[wid][i][g + 8][t * 2]) = make_float2(acc[i][2], acc[i][3]);
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < NT * 8 * FR_COLS; e += FR_WARPS * 32) {
+    const int c = e & (FR_COLS - 1), row = e / FR_COLS;
+    const int col = n0 + c;
+    if (row >= m || col >= p.n) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int q = 0; q < FR_WARPS; ++q) v += red[q][row >> 3][c][row & 7];
+    if (col < p.n_half) {
+      if (p.gelu) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
+      static_cast<bf16 *>(p.half_out)[(long long)row * p.half_ld + col] = __float2bfloat16_rn(v);
+    } else {
+      float *o = p.float_out + (long long)row * p.float_ld + (col - p.n_half);
+      *o = p.accumulate ? *o + v : v;
+    }
+  }
+}
+
+}  // namespace
+
+void launch_few_row_bf16(const Bf16Product *p, int count, int m, cudaStream_t st) {
+  if (m < 1 || m > FEW_ROWS_MAX || count < 1 || count > 2) throw std::invalid_argument("launch_few_row_bf16: bad shape");
+  FewRowPair pair{};
+  unsigned blocks = 0;
+  for (int i = 0; i < count; ++i) {
+    pair.p[i] = p[i];
+    blocks += (unsigned)((p[i].n + FR_COLS - 1) / FR_COLS);
+    if (i == 0) pair.blocks0 = (int)blocks;
+  }
+  const dim3 grid(blocks), block(FR_WARPS * 32);
+  const int nt = (m + 7) / 8;
+  if (nt <= 1) launch_pdl(few_row_bf16_kernel<1, 4>, grid, block, 0, st, g_pdl_enabled, pair, m);
+  else if (nt <= 2) launch_pdl(few_row_bf16_kernel<2, 4>, grid, block, 0, st, g_pdl_enabled, pair, m);
+  else if (nt <= 4) launch_pdl(few_row_bf16_kernel<4, 4>, grid, block, 0, st, g_pdl_enabled, pair, m);
+  else launch_pdl(few_row_bf16_kernel<8, 4>, grid, block, 0, st, g_pdl_enabled, pair, m);
+}
+
+}  // namespace lb

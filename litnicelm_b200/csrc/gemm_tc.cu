@@ -646,6 +646,24 @@ void tc_make_map_plain(CUtensorMap *map, const float *base, unsigned long long r
     throw std::runtime_error("litnice_b200: cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
 }
 
+void tc_make_map_bf16(CUtensorMap *map, const void *base, unsigned long long rows, unsigned long long cols,
+                      unsigned long long ld, unsigned box_rows) {
+  EncodeTiledFn fn = encode_tiled_fn();
+  if (fn == nullptr) throw std::runtime_error("litnice_b200: cuTensorMapEncodeTiled is not available");
+  if ((reinterpret_cast<uintptr_t>(base) & 15) != 0 || ld % 8 != 0 || cols > ld || rows == 0 || cols == 0 ||
+      box_rows == 0 || box_rows > 256)
+    throw std::invalid_argument("litnice_b200: bfloat16 tensor map operand must be 16-byte aligned with ld % 8 == 0");
+  const cuuint64_t dims[2] = {cols, rows};
+  const cuuint64_t strides[1] = {ld * 2};  // bytes between rows
+  const cuuint32_t box[2] = {64, box_rows};
+  const cuuint32_t estr[2] = {1, 1};
+  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr,
+                        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS)
+    throw std::runtime_error("litnice_b200: cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
+}
+
 // How many clusters of 2..8 CTAs of these kernels the device holds at once (a cluster sits inside
 // one GPC); -1 where the runtime cannot say. Every configuration runs one CTA per SM, so one of them
 // stands for all.

@@ -99,6 +99,12 @@ void tc_make_map_f16(CUtensorMap *map, const __half *base, unsigned long long ro
 void tc_make_map_plain(CUtensorMap *map, const float *base, unsigned long long rows, unsigned long long cols,
                        unsigned box_rows, unsigned box_cols);
 
+// Tensor map over a bfloat16 array [rows, cols] whose rows are ld elements apart (ld % 8 == 0, base
+// 16-byte aligned), boxes of box_rows x 64 elements with the 128-byte swizzle; what lies outside
+// [rows, cols] reads as zero.
+void tc_make_map_bf16(CUtensorMap *map, const void *base, unsigned long long rows, unsigned long long cols,
+                      unsigned long long ld, unsigned box_rows);
+
 // How one product is tiled: tile width (64, 128 or 256 columns), how many CTAs share
 // the k range of a tile, and the scratch that sharing needs (floats of partial
 // tiles; int counters that must be zero before the first launch and are left

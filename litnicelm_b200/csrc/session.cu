@@ -16,9 +16,17 @@
 // Work elided because nothing can observe it (the loop reads row s-1 only,
 // inference.cpp:109-115): LN_f and the output head on rows 0..s-2, the dead
 // zero-fill of the attention context, the attention-weights cache.
+//
+// A session may instead serve one of the registered decoder designs (model.cuh):
+// litnice_b200_session_create_model. Such a model keeps a cache and state per
+// slot; the loop, the sampler, the graphs and the entry points stay the ones
+// below, with the model's own step where the transformer's passes stand, and
+// slots may also be extended in portions (litnice_b200_extend).
 #include "common.cuh"
 #include "gemm_tc.cuh"
+#include "model.cuh"
 
+#include <algorithm>
 #include <array>
 #include <cmath>
 #include <cstdio>
@@ -218,6 +226,12 @@ struct litnice_b200_session {
   float *pk_scratch = nullptr;
   size_t pk_scratch_floats = 0;
   unsigned *pk_barrier = nullptr;
+
+  // Registered decoder design served instead of the litnicelm transformer (null: the transformer).
+  std::unique_ptr<DecoderModel> model;
+  std::vector<int> slot_len;      // positions each slot holds (litnice_b200_extend)
+  int *rows_list = nullptr;       // device: rows of a portion whose logits are asked for
+  long long rows_list_cap = 0;
 
   bool keep_logits = false;
   float *step_logits = nullptr;
@@ -857,12 +871,106 @@ void prepare_tc_weights(litnice_b200_session *s) {
   prepare_one(s, &s->tc_head, P(s, s->lay.lm_head), D, d.vocab_size);
 }
 
+// ---- registered decoder designs ------------------------------------------------
+
+RowBatch row_batch(const litnice_b200_session *s, int streams, int slot0, int p0, int n) {
+  RowBatch b;
+  b.streams = streams;
+  b.slot0 = slot0;
+  b.p0 = p0;
+  b.n = n;
+  b.s_cap = p0 + n;
+  b.ids = s->ids;
+  b.ids_ld = s->dims.max_seq_len;
+  return b;
+}
+
+int portion_len(const litnice_b200_session *s, int streams) {
+  const long long n = s->model->portion_rows() / streams;
+  return n < 1 ? 1 : (int)n;
+}
+
+void model_reserve(litnice_b200_session *s, int streams, int cap, int longest_portion) {
+  const int part = portion_len(s, streams);
+  const long long n = longest_portion < part ? longest_portion : part;
+  if (s->model->reserve(s->max_streams, cap, n * streams, s->st)) ++s->generation;
+}
+
+// Positions from .. to - 1 of the first B slots, in portions; returns the last portion.
+RowBatch model_advance(litnice_b200_session *s, int B, int from, int to) {
+  RowBatch b;
+  const int part = portion_len(s, B);
+  for (int p = from; p < to; p += b.n) {
+    b = row_batch(s, B, 0, p, to - p < part ? to - p : part);
+    s->launches += s->model->enqueue_rows(b, s->st, s->err_dev);
+  }
+  return b;
+}
+
+// The newest position of every stream, ending with its logits (n == 1: one row per stream).
+void model_decode_step(litnice_b200_session *s, int B, int s_cap, int sl, const LoopState *dstate) {
+  RowBatch b = row_batch(s, B, 0, sl - 1, 1);
+  b.s_cap = s_cap;
+  b.state = dstate;
+  s->launches += s->model->enqueue_rows(b, s->st, s->err_dev);
+  s->launches += s->model->enqueue_head(b, nullptr, B, s->logits, s->st, s->err_dev);
+}
+
+void ensure_logits_all(litnice_b200_session *s, long long rows) {
+  if (s->logits_all_rows >= rows) return;
+  LB_CUDA(cudaStreamSynchronize(s->st));
+  if (s->logits_all) cudaFree(s->logits_all);
+  s->logits_all = nullptr;
+  s->logits_all_rows = 0;
+  if (cudaMalloc(reinterpret_cast<void **>(&s->logits_all), (size_t)rows * s->dims.vocab_size * 4) != cudaSuccess)
+    throw std::bad_alloc();
+  s->logits_all_rows = rows;
+}
+
+// Whole-context forward of a registered design on the first B slots (forward / inspect): logits of
+// every row to host memory at all_rows_out, or (null) of the last rows to s->logits.
+void model_forward(litnice_b200_session *s, int B, int seq_len, float *all_rows_out) {
+  const int V = s->dims.vocab_size, part = portion_len(s, B);
+  std::fill(s->slot_len.begin(), s->slot_len.end(), 0);
+  s->kv_len = 0;
+  model_reserve(s, B, seq_len, seq_len);
+  if (all_rows_out == nullptr) {
+    const RowBatch b = model_advance(s, B, 0, seq_len);
+    s->launches += s->model->enqueue_head(b, nullptr, B, s->logits, s->st, s->err_dev);
+    return;
+  }
+  std::vector<int> rows;
+  for (int p = 0, n = 0; p < seq_len; p += n) {
+    n = seq_len - p < part ? seq_len - p : part;
+    const RowBatch b = row_batch(s, B, 0, p, n);
+    s->launches += s->model->enqueue_rows(b, s->st, s->err_dev);
+    ensure_logits_all(s, b.rows());
+    if (s->rows_list_cap < b.rows()) {
+      LB_CUDA(cudaStreamSynchronize(s->st));
+      if (s->rows_list) cudaFree(s->rows_list);
+      s->rows_list = nullptr;
+      s->rows_list_cap = 0;
+      if (cudaMalloc(reinterpret_cast<void **>(&s->rows_list), (size_t)b.rows() * 4) != cudaSuccess) throw std::bad_alloc();
+      s->rows_list_cap = b.rows();
+    }
+    rows.resize((size_t)b.rows());
+    for (size_t i = 0; i < rows.size(); ++i) rows[i] = (int)i;
+    LB_CUDA(cudaMemcpyAsync(s->rows_list, rows.data(), rows.size() * 4, cudaMemcpyHostToDevice, s->st));
+    s->launches += s->model->enqueue_head(b, s->rows_list, (int)b.rows(), s->logits_all, s->st, s->err_dev);
+    // rows of a portion are [stream][n]; the caller's array is [stream][seq_len]
+    LB_CUDA(cudaMemcpy2DAsync(all_rows_out + (size_t)p * V, (size_t)seq_len * V * 4, s->logits_all, (size_t)n * V * 4,
+                              (size_t)n * V * 4, (size_t)B, cudaMemcpyDeviceToHost, s->st));
+    LB_CUDA(cudaStreamSynchronize(s->st));
+  }
+}
+
 void check_device_error(litnice_b200_session *s) {
   if (s->err_host->code == DEVERR_NONE) return;
   const int code = s->err_host->code, detail = s->err_host->detail;
   s->err_host->code = DEVERR_NONE;
   if (code == DEVERR_BAD_TOKEN_ID)
     throw std::runtime_error("embedding id out of range (id=" + std::to_string(detail) + ")");
+  if (code == DEVERR_NON_FINITE) throw std::runtime_error("a weight is not finite");
   if (code == DEVERR_WAIT_TIMEOUT)
     throw std::runtime_error("a bounded wait inside the tensor-core GEMM ran out (role " + std::to_string(detail) +
                              ")");
@@ -916,10 +1024,215 @@ int litnice_b200_session_create_on(const litnice_b200_dims *dims, int32_t max_st
   return session_create_impl(dims, max_streams, device, out);
 }
 
+// The device a new session runs on; negative: a status code.
+static int pick_device(int32_t device_or_negative) {
+  int count = 0;
+  if (cudaGetDeviceCount(&count) != cudaSuccess || count == 0) return LITNICE_B200_ECUDA;
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (device_or_negative >= 0) dev = device_or_negative;
+  else if (const char *env = std::getenv("LITNICE_B200_DEVICE")) dev = std::atoi(env);
+  return dev < 0 || dev >= count ? LITNICE_B200_EINVAL : dev;
+}
+
+// What every session has: stream, events, error word, loop state, ids and logits for `logit_rows` rows.
+static cudaDeviceProp session_common(litnice_b200_session *s) {
+  cudaDeviceProp prop{};
+  LB_CUDA(cudaGetDeviceProperties(&prop, s->device));
+  if (prop.major != 10)
+    throw std::invalid_argument("built for sm_100a (B200) only; found sm_" + std::to_string(prop.major) +
+                                std::to_string(prop.minor));
+  LB_CUDA(cudaStreamCreateWithFlags(&s->st, cudaStreamNonBlocking));
+  LB_CUDA(cudaEventCreate(&s->ev0));
+  LB_CUDA(cudaEventCreate(&s->ev1));
+  LB_CUDA(cudaHostAlloc(reinterpret_cast<void **>(&s->err_host), sizeof(DevErr), cudaHostAllocMapped));
+  s->err_host->code = DEVERR_NONE;
+  s->err_host->detail = 0;
+  LB_CUDA(cudaHostGetDevicePointer(reinterpret_cast<void **>(&s->err_dev), s->err_host, 0));
+  const char *pdl_env = std::getenv("LITNICE_B200_PDL");
+  s->pdl = !(pdl_env && pdl_env[0] == '0');
+  const char *graph_env = std::getenv("LITNICE_B200_GRAPHS");
+  s->use_graphs = !(graph_env && graph_env[0] == '0');
+  s->sm_count = prop.multiProcessorCount;
+  return prop;
+}
+
+static void session_loop_buffers(litnice_b200_session *s, size_t logit_rows) {
+  auto must = [&](cudaError_t e) { if (e != cudaSuccess) throw std::bad_alloc(); };
+  const litnice_b200_dims &d = s->dims;
+  must(cudaMalloc(reinterpret_cast<void **>(&s->logits), logit_rows * d.vocab_size * 4));
+  must(cudaMalloc(reinterpret_cast<void **>(&s->probs), logit_rows * d.vocab_size * 4));
+  LB_CUDA(cudaMemsetAsync(s->logits, 0, logit_rows * d.vocab_size * 4, s->st));
+  must(cudaMalloc(reinterpret_cast<void **>(&s->ids), (size_t)s->max_streams * d.max_seq_len * 4));
+  LB_CUDA(cudaMemsetAsync(s->ids, 0, (size_t)s->max_streams * d.max_seq_len * 4, s->st));
+  must(cudaMalloc(reinterpret_cast<void **>(&s->mt), (size_t)s->max_streams * 625 * 4));
+  // the loop state, followed by the fused greedy tail's finished-CTA counter
+  must(cudaMalloc(reinterpret_cast<void **>(&s->state), sizeof(LoopState) + 16));
+  LB_CUDA(cudaMemsetAsync(s->state, 0, sizeof(LoopState) + 16, s->st));
+}
+
+// Names the reason a model folder was refused when no session exists to carry it.
+static thread_local std::string g_create_error = "null session";
+
+int litnice_b200_session_create_model(const char *model_dir, int32_t dtype, int32_t max_streams, int32_t device,
+                                      litnice_b200_session **out) {
+  if (out == nullptr) return LITNICE_B200_EINVAL;
+  *out = nullptr;
+  g_create_error = "null session";
+  if (model_dir == nullptr || max_streams <= 0 ||
+      (dtype != LITNICE_B200_DTYPE_BF16 && dtype != LITNICE_B200_DTYPE_F32))
+    return LITNICE_B200_EINVAL;
+  auto *s = new litnice_b200_session();
+  s->max_streams = max_streams;
+  std::unique_ptr<TensorFile> file;
+  try {  // the folder is checked before a device is touched
+    const std::string dir(model_dir);
+    s->model = make_model(Json::parse(read_text_file(dir + "/config.json")),
+                          dtype == LITNICE_B200_DTYPE_F32 ? Precision::F32 : Precision::BF16);
+    file.reset(new TensorFile(dir + "/model.safetensors"));
+  } catch (const std::exception &e) {
+    g_create_error = e.what();
+    delete s;
+    return LITNICE_B200_EIO;
+  }
+  const int dev = pick_device(device);
+  if (dev < 0) {
+    g_create_error = "no usable CUDA device";
+    delete s;
+    return dev;
+  }
+  s->device = dev;
+  s->dims.n_layers = s->model->n_layers();
+  s->dims.n_heads = 1;
+  s->dims.d_model = s->model->width();
+  s->dims.vocab_size = s->model->vocab();
+  s->dims.max_seq_len = s->model->max_positions();
+  s->slot_len.assign((size_t)max_streams, 0);
+  *out = s;  // handed out even on failure below so the caller can read the error text
+  const int rc = guarded(s, [&]() {
+    session_common(s);
+    if (!tc_runtime_available()) throw std::runtime_error("cuTensorMapEncodeTiled is not available");
+    session_loop_buffers(s, (size_t)(max_streams < 8 ? 8 : max_streams));
+    try {
+      s->model->load(*file, s->st, s->err_dev);
+    } catch (const CudaError &) {
+      throw;
+    } catch (const std::runtime_error &e) {
+      return fail(s, LITNICE_B200_EIO, e.what());
+    }
+    if (s->err_host->code == DEVERR_NON_FINITE) {
+      s->err_host->code = DEVERR_NONE;
+      return fail(s, LITNICE_B200_EIO, "a weight is not finite");
+    }
+    check_device_error(s);
+    s->params_loaded = true;
+    return LITNICE_B200_OK;
+  });
+  return rc;
+}
+
+const char *litnice_b200_architectures(void) { return registered_architectures(); }
+
+int litnice_b200_model_dims(const litnice_b200_session *s, litnice_b200_dims *out) {
+  if (s == nullptr || out == nullptr) return LITNICE_B200_EINVAL;
+  *out = s->dims;
+  return LITNICE_B200_OK;
+}
+
+int litnice_b200_extend(litnice_b200_session *s, int32_t slot, const int32_t *tokens, int32_t n, const int32_t *want,
+                        int32_t n_want, float *out_logits) {
+  return guarded(s, [&]() {
+    if (!s->model) throw std::invalid_argument("extend needs a model with a state per slot (session_create_model)");
+    if (!s->params_loaded) throw std::invalid_argument("no parameters loaded");
+    if (slot < 0 || slot >= s->max_streams || tokens == nullptr || n <= 0 || n_want < 0 ||
+        (n_want > 0 && (want == nullptr || out_logits == nullptr)))
+      throw std::invalid_argument("bad extend arguments");
+    const int V = s->dims.vocab_size, S = s->dims.max_seq_len, have = s->slot_len[(size_t)slot];
+    if (n > S - have)
+      throw std::invalid_argument("slot " + std::to_string(slot) + " would exceed " + std::to_string(S) + " positions");
+    for (int i = 0; i < n; ++i)
+      if (tokens[i] < 0 || tokens[i] >= V)
+        throw std::invalid_argument("embedding id out of range (id=" + std::to_string(tokens[i]) + ")");
+    std::vector<bool> seen((size_t)n, false);
+    for (int i = 0; i < n_want; ++i) {
+      if (want[i] < 0 || want[i] >= n) throw std::invalid_argument("a wanted place lies outside the new tokens");
+      if (seen[(size_t)want[i]]) throw std::invalid_argument("a place is wanted twice");
+      seen[(size_t)want[i]] = true;
+    }
+    PdlScope pdl_scope(s->pdl);
+    s->stats = litnice_b200_stats{};
+    s->cur_streams = 0;  // slots are shared with the lockstep batch
+    s->kv_len = 0;
+    s->slot_len[(size_t)slot] = 0;  // until the step has gone through
+    int cap = 256;
+    while (cap < have + n) cap *= 2;
+    model_reserve(s, 1, cap < S ? cap : S, n);
+    ensure_logits_all(s, n_want > 0 ? n_want : 1);
+    if (s->rows_list_cap < n_want) {
+      if (s->rows_list) cudaFree(s->rows_list);
+      s->rows_list = nullptr;
+      s->rows_list_cap = 0;
+      if (cudaMalloc(reinterpret_cast<void **>(&s->rows_list), (size_t)n_want * 4) != cudaSuccess) throw std::bad_alloc();
+      s->rows_list_cap = n_want;
+    }
+    LB_CUDA(cudaMemcpyAsync(s->ids + (size_t)slot * S + have, tokens, (size_t)n * 4, cudaMemcpyHostToDevice, s->st));
+    s->stats.h2d_bytes += (long long)n * 4;
+    const long long launches0 = s->launches;
+    LB_CUDA(cudaEventRecord(s->ev0, s->st));
+    // `want` may come in any order: per portion its rows are gathered, and the logits scattered back
+    const int part = portion_len(s, 1);
+    std::vector<int> rows, places;
+    for (int p = 0; p < n; p += part) {
+      const int m = n - p < part ? n - p : part;
+      const RowBatch b = row_batch(s, 1, slot, have + p, m);
+      s->launches += s->model->enqueue_rows(b, s->st, s->err_dev);
+      rows.clear();
+      places.clear();
+      for (int i = 0; i < n_want; ++i)
+        if (want[i] >= p && want[i] < p + m) {
+          rows.push_back(want[i] - p);
+          places.push_back(i);
+        }
+      if (rows.empty()) continue;
+      LB_CUDA(cudaMemcpyAsync(s->rows_list, rows.data(), rows.size() * 4, cudaMemcpyHostToDevice, s->st));
+      s->launches += s->model->enqueue_head(b, s->rows_list, (int)rows.size(), s->logits_all, s->st, s->err_dev);
+      bool in_order = true;
+      for (size_t i = 1; i < places.size(); ++i) in_order &= places[i] == places[0] + (int)i;
+      if (in_order) {
+        LB_CUDA(cudaMemcpyAsync(out_logits + (size_t)places[0] * V, s->logits_all, rows.size() * V * 4,
+                                cudaMemcpyDeviceToHost, s->st));
+      } else {
+        for (size_t i = 0; i < places.size(); ++i)
+          LB_CUDA(cudaMemcpyAsync(out_logits + (size_t)places[i] * V, s->logits_all + i * V, (size_t)V * 4,
+                                  cudaMemcpyDeviceToHost, s->st));
+      }
+      s->stats.d2h_bytes += (long long)rows.size() * V * 4;
+      LB_CUDA(cudaStreamSynchronize(s->st));
+    }
+    LB_CUDA(cudaEventRecord(s->ev1, s->st));
+    LB_CUDA(cudaStreamSynchronize(s->st));
+    check_device_error(s);
+    float ms = 0.f;
+    LB_CUDA(cudaEventElapsedTime(&ms, s->ev0, s->ev1));
+    s->stats.device_ms = ms;
+    s->stats.kernel_launches = s->launches - launches0;
+    s->stats.tokens = n;
+    s->slot_len[(size_t)slot] = have + n;
+    return LITNICE_B200_OK;
+  });
+}
+
+int litnice_b200_release(litnice_b200_session *s, int32_t slot) {
+  if (s == nullptr || !s->model || slot < 0 || slot >= s->max_streams) return LITNICE_B200_EINVAL;
+  s->slot_len[(size_t)slot] = 0;  // rows are read by position, so a new sequence sees nothing of the old one
+  return LITNICE_B200_OK;
+}
+
 static int session_create_impl(const litnice_b200_dims *dims, int32_t max_streams, int32_t device_or_negative,
                                litnice_b200_session **out) {
   if (out == nullptr) return LITNICE_B200_EINVAL;
   *out = nullptr;
+  g_create_error = "null session";
   if (dims == nullptr || max_streams <= 0) return LITNICE_B200_EINVAL;
   const litnice_b200_dims &d = *dims;
   if (d.n_layers <= 0 || d.n_heads <= 0 || d.d_model <= 0 || d.d_ff <= 0 || d.vocab_size <= 0 ||
@@ -932,43 +1245,20 @@ static int session_create_impl(const litnice_b200_dims *dims, int32_t max_stream
   auto *s = new litnice_b200_session();
   s->dims = d;
   s->max_streams = max_streams;
-  int count = 0;
-  if (cudaGetDeviceCount(&count) != cudaSuccess || count == 0) {
+  const int dev = pick_device(device_or_negative);
+  if (dev < 0) {
     delete s;
-    return LITNICE_B200_ECUDA;
-  }
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (device_or_negative >= 0) dev = device_or_negative;
-  else if (const char *env = std::getenv("LITNICE_B200_DEVICE")) dev = std::atoi(env);
-  if (dev < 0 || dev >= count) {
-    delete s;
-    return LITNICE_B200_EINVAL;
+    return dev;
   }
   s->device = dev;
   *out = s;  // handed out even on failure below so the caller can read the error text
   return guarded(s, [&]() {
-    cudaDeviceProp prop{};
-    LB_CUDA(cudaGetDeviceProperties(&prop, dev));
-    if (prop.major != 10)
-      throw std::invalid_argument("built for sm_100a (B200) only; found sm_" + std::to_string(prop.major) +
-                                  std::to_string(prop.minor));
+    const cudaDeviceProp prop = session_common(s);
     s->lay = build_layout(d);
-    LB_CUDA(cudaStreamCreateWithFlags(&s->st, cudaStreamNonBlocking));
-    LB_CUDA(cudaEventCreate(&s->ev0));
-    LB_CUDA(cudaEventCreate(&s->ev1));
-    LB_CUDA(cudaHostAlloc(reinterpret_cast<void **>(&s->err_host), sizeof(DevErr), cudaHostAllocMapped));
-    s->err_host->code = DEVERR_NONE;
-    s->err_host->detail = 0;
-    LB_CUDA(cudaHostGetDevicePointer(reinterpret_cast<void **>(&s->err_dev), s->err_host, 0));
     auto must = [&](cudaError_t e) { if (e != cudaSuccess) throw std::bad_alloc(); };
     must(cudaMalloc(reinterpret_cast<void **>(&s->params), s->lay.total));
     // Tensor-core projections need k % 32 == 0 and n % 64 == 0 for all four
     // layer matrices; LITNICE_B200_TC=0 forces the fp32 SIMT kernels.
-    const char *pdl_env = std::getenv("LITNICE_B200_PDL");
-    s->pdl = !(pdl_env && pdl_env[0] == '0');
-    const char *graph_env = std::getenv("LITNICE_B200_GRAPHS");
-    s->use_graphs = !(graph_env && graph_env[0] == '0');
     const char *tail_env = std::getenv("LITNICE_B200_FUSED_TAIL");
     s->fused_tail = !(tail_env && tail_env[0] == '0');
     const char *kv_env = std::getenv("LITNICE_B200_KV_CACHE");
@@ -977,7 +1267,6 @@ static int session_create_impl(const litnice_b200_dims *dims, int32_t max_stream
     s->kv_fuse = !(kvf_env && kvf_env[0] == '0');
     const char *kvp_env = std::getenv("LITNICE_B200_KV_PERSIST");
     s->kv_persist = !(kvp_env && kvp_env[0] == '0') && prop.cooperativeLaunch != 0;
-    s->sm_count = prop.multiProcessorCount;
     if (s->kv) {
       std::vector<unsigned long long> offs;
       for (const LayerOff &o : s->lay.layer)
@@ -1020,10 +1309,8 @@ static int session_create_impl(const litnice_b200_dims *dims, int32_t max_stream
       must(cudaMalloc(reinterpret_cast<void **>(&s->tc_counters), 148 * 4));
       LB_CUDA(cudaMemsetAsync(s->tc_counters, 0, 148 * 4, s->st));
     }
-    must(cudaMalloc(reinterpret_cast<void **>(&s->logits), lr * d.vocab_size * 4));
-    must(cudaMalloc(reinterpret_cast<void **>(&s->probs), lr * d.vocab_size * 4));
+    session_loop_buffers(s, lr);
     LB_CUDA(cudaMemsetAsync(s->xl, 0, lr * d.d_model * 4, s->st));
-    LB_CUDA(cudaMemsetAsync(s->logits, 0, lr * d.vocab_size * 4, s->st));
     size_t gs = gemv_scratch_floats(8, d.vocab_size, d.d_model);
     if (s->kv) {
       // the step's rows and the few-row products of the layers
@@ -1039,12 +1326,6 @@ static int session_create_impl(const litnice_b200_dims *dims, int32_t max_stream
       }
     }
     if (gs) must(cudaMalloc(reinterpret_cast<void **>(&s->gemv_scratch), gs * 4));
-    must(cudaMalloc(reinterpret_cast<void **>(&s->ids), (size_t)max_streams * d.max_seq_len * 4));
-    LB_CUDA(cudaMemsetAsync(s->ids, 0, (size_t)max_streams * d.max_seq_len * 4, s->st));
-    must(cudaMalloc(reinterpret_cast<void **>(&s->mt), (size_t)max_streams * 625 * 4));
-    // the loop state, followed by the fused greedy tail's finished-CTA counter
-    must(cudaMalloc(reinterpret_cast<void **>(&s->state), sizeof(LoopState) + 16));
-    LB_CUDA(cudaMemsetAsync(s->state, 0, sizeof(LoopState) + 16, s->st));
     LB_CUDA(cudaStreamSynchronize(s->st));
     return LITNICE_B200_OK;
   });
@@ -1054,6 +1335,8 @@ void litnice_b200_session_destroy(litnice_b200_session *s) {
   if (s == nullptr) return;
   cudaSetDevice(s->device);
   if (s->st) cudaStreamSynchronize(s->st);
+  s->model.reset();
+  if (s->rows_list) cudaFree(s->rows_list);
   free_activations(s);
   for (void *p : {(void *)s->params, (void *)s->xl, (void *)s->logits, (void *)s->probs, (void *)s->gemv_scratch,
                   (void *)s->logits_all, (void *)s->ids, (void *)s->out_tokens, (void *)s->mt, (void *)s->state,
@@ -1101,11 +1384,12 @@ void litnice_b200_session_destroy(litnice_b200_session *s) {
 }
 
 const char *litnice_b200_last_error(const litnice_b200_session *s) {
-  return s ? s->error.c_str() : "null session";
+  return s ? s->error.c_str() : g_create_error.c_str();
 }
 
 int litnice_b200_load_params(litnice_b200_session *s, const void *host_arena, uint64_t bytes) {
   return guarded(s, [&]() {
+    if (s->model) throw std::invalid_argument("the weights of this session come from its model folder");
     if (host_arena == nullptr || bytes != s->lay.total)
       throw std::invalid_argument("parameter arena must be " + std::to_string(s->lay.total) + " bytes, got " +
                                   std::to_string(bytes));
@@ -1119,6 +1403,7 @@ int litnice_b200_load_params(litnice_b200_session *s, const void *host_arena, ui
 
 int litnice_b200_load_checkpoint(litnice_b200_session *s, const char *path) {
   if (s == nullptr || path == nullptr) return LITNICE_B200_EINVAL;
+  if (s->model) return fail(s, LITNICE_B200_EINVAL, "the weights of this session come from its model folder");
   // CkptHeaderV6 (checkpoint.cpp:98-116): 136 bytes.
 #pragma pack(push, 1)
   struct Header {
@@ -1198,7 +1483,8 @@ int litnice_b200_upload_prompts(litnice_b200_session *s, const int32_t *prompts,
     s->cur_streams = n_streams;
     s->cur_prompt_len = prompt_len;
     s->cur_tokens = 0;
-    s->kv_len = 0;  // cached mode: the caches hold another batch's positions
+    s->kv_len = 0;  // the caches hold another batch's positions
+    std::fill(s->slot_len.begin(), s->slot_len.end(), 0);
     return LITNICE_B200_OK;
   });
 }
@@ -1220,7 +1506,9 @@ int litnice_b200_run(litnice_b200_session *s, int32_t max_new, const litnice_b20
     if (steps < 0) steps = 0;
     const int s_last = s0 + (steps > 0 ? steps - 1 : 0);
     const int s_last_cap = (s_last + 63) / 64 * 64;  // graph replay sizes launches per 64-token bucket
-    if (s->kv) {
+    if (s->model) {
+      if (steps > 0) model_reserve(s, B, s_last, s->kv_len != s0 - 1 ? s0 - s->kv_len : 1);
+    } else if (s->kv) {
       // cached mode: whole-context buffers only for the pass over the prompt that fills the caches
       if (steps > 0) {
         ensure_kv(s, B, s_last_cap);
@@ -1288,12 +1576,19 @@ int litnice_b200_run(litnice_b200_session *s, int32_t max_new, const litnice_b20
     // the host issues one launch per token instead of ~50.
     const bool graphs = s->use_graphs && !s->keep_logits;
     const bool fused_tail =
-        greedy && !s->keep_logits && s->fused_tail && !s->kv && head_greedy_supports(B, s->dims.d_model, V);
+        greedy && !s->keep_logits && s->fused_tail && !s->kv && !s->model && head_greedy_supports(B, s->dims.d_model, V);
     // cached mode, greedy, few streams, small vocabulary: the step ends in the one-launch tail too
     const bool decode_tail = s->kv && s->kv_fuse && greedy && !s->keep_logits && s->fused_tail &&
                              head_greedy_supports(B, s->dims.d_model, V);
     auto enqueue_step = [&](int sl_cap, const LoopState *dstate, int step, bool decode) {
-      if (decode) {
+      if (s->model) {
+        if (decode) {
+          model_decode_step(s, B, sl_cap, s0 + step, dstate);
+        } else {  // the positions the slots do not hold yet
+          const RowBatch b = model_advance(s, B, s->kv_len, s0 + step);
+          s->launches += s->model->enqueue_head(b, nullptr, B, s->logits, s->st, s->err_dev);
+        }
+      } else if (decode) {
         enqueue_decode_step(s, B, sl_cap, dstate, !decode_tail);
         if (decode_tail) {  // the step's rows are the last rows: one row per stream
           launch_head_greedy(s->dx, P(s, s->lay.lnf_g), P(s, s->lay.lnf_b), P(s, s->lay.lm_head), s->dims.d_model, V, B,
@@ -1319,7 +1614,7 @@ int litnice_b200_run(litnice_b200_session *s, int32_t max_new, const litnice_b20
         ++s->launches;
         return;
       }
-      if (!decode) enqueue_head_last(s, B, sl_cap, dstate);
+      if (!decode && !s->model) enqueue_head_last(s, B, sl_cap, dstate);
       if (s->keep_logits) {
         LB_CUDA(cudaMemcpyAsync(s->step_logits + (long long)(s->cur_tokens + step) * B * V, s->logits,
                                 (size_t)B * V * 4, cudaMemcpyDeviceToDevice, s->st));
@@ -1334,8 +1629,8 @@ int litnice_b200_run(litnice_b200_session *s, int32_t max_new, const litnice_b20
       const int sl = s0 + step;
       // cached mode: a step on one new row per stream when the caches hold every earlier
       // position, else a whole-context pass that also fills them (the first step of a batch)
-      const bool decode = s->kv && s->kv_len == sl - 1;
-      if (decode && s->kv_persist && greedy && !s->keep_logits && B <= 8 && s->pk_scratch != nullptr &&
+      const bool decode = (s->kv || s->model) && s->kv_len == sl - 1;
+      if (decode && s->kv && s->kv_persist && greedy && !s->keep_logits && B <= 8 && s->pk_scratch != nullptr &&
           decode_persistent_supports(B, s->dims.n_heads, s->dims.d_model, s->dims.d_ff, V)) {
         // every remaining step in one resident kernel
         DecodePersistentArgs a{};
@@ -1385,12 +1680,14 @@ int litnice_b200_run(litnice_b200_session *s, int32_t max_new, const litnice_b20
         s->kv_len = s0 + steps - 1;
         break;
       }
-      if (s->kv) s->kv_len = sl;
-      if (!graphs || (s->kv && !decode)) {
+      if (!graphs || ((s->kv || s->model) && !decode)) {
         enqueue_step(sl, nullptr, step, decode);
+        if (s->kv || s->model) s->kv_len = sl;
         continue;
       }
-      const int bucket = (sl + 63) / 64;
+      if (s->kv || s->model) s->kv_len = sl;
+      const int bound = s->model ? s->model->context_bound(sl) : (sl + 63) / 64 * 64;
+      const int bucket = (bound + 63) / 64;
       if ((int)s->graphs.size() <= bucket) s->graphs.resize(bucket + 1);
       litnice_b200_session::StepGraph &g = s->graphs[bucket];
       const bool valid = g.exec != nullptr && g.streams == B && g.generation == s->generation &&
@@ -1404,7 +1701,7 @@ int litnice_b200_run(litnice_b200_session *s, int32_t max_new, const litnice_b20
         cudaGraph_t graph = nullptr;
         LB_CUDA(cudaStreamBeginCapture(s->st, cudaStreamCaptureModeRelaxed));
         try {
-          enqueue_step(bucket * 64, s->state, step, decode);
+          enqueue_step(bound, s->state, step, decode);
         } catch (...) {
           cudaStreamEndCapture(s->st, &graph);
           if (graph) cudaGraphDestroy(graph);
@@ -1490,6 +1787,23 @@ int litnice_b200_forward(litnice_b200_session *s, const int32_t *ids, int32_t n_
     const long long R = (long long)B * seq_len;
     s->stats = litnice_b200_stats{};
     s->cur_streams = 0;  // the ids of an uploaded prompt batch are overwritten: run needs a fresh upload
+    if (s->model) {
+      upload_ids(s, ids, B, seq_len);
+      const long long before = s->launches;
+      LB_CUDA(cudaEventRecord(s->ev0, s->st));
+      model_forward(s, B, seq_len, all_rows ? out_logits : nullptr);
+      LB_CUDA(cudaEventRecord(s->ev1, s->st));
+      if (!all_rows)
+        LB_CUDA(cudaMemcpyAsync(out_logits, s->logits, (size_t)B * V * 4, cudaMemcpyDeviceToHost, s->st));
+      s->stats.d2h_bytes += (all_rows ? R : (long long)B) * V * 4;
+      LB_CUDA(cudaStreamSynchronize(s->st));
+      check_device_error(s);
+      float model_ms = 0.f;
+      LB_CUDA(cudaEventElapsedTime(&model_ms, s->ev0, s->ev1));
+      s->stats.device_ms = model_ms;
+      s->stats.kernel_launches = s->launches - before;
+      return LITNICE_B200_OK;
+    }
     ensure_rows(s, R);
     ensure_attention_scratch(s, B, seq_len, seq_len);
     upload_ids(s, ids, B, seq_len);
@@ -1497,15 +1811,7 @@ int litnice_b200_forward(litnice_b200_session *s, const int32_t *ids, int32_t n_
     LB_CUDA(cudaEventRecord(s->ev0, s->st));
     enqueue_body(s, B, seq_len);
     if (all_rows) {
-      if (s->logits_all_rows < R) {
-        LB_CUDA(cudaStreamSynchronize(s->st));
-        if (s->logits_all) cudaFree(s->logits_all);
-        s->logits_all = nullptr;
-        s->logits_all_rows = 0;
-        if (cudaMalloc(reinterpret_cast<void **>(&s->logits_all), (size_t)R * V * 4) != cudaSuccess)
-          throw std::bad_alloc();
-        s->logits_all_rows = R;
-      }
+      ensure_logits_all(s, R);
       // OutputHead::forward over every row (output_head.cpp:58-70)
       const bool head_tc = s->tc && s->tc_head.usable();
       launch_layernorm_dense(s->x, P(s, s->lay.lnf_g), P(s, s->lay.lnf_b), R, D, s->ln,
@@ -1543,13 +1849,21 @@ int litnice_b200_inspect(litnice_b200_session *s, const int32_t *ids, int32_t n_
     const int B = n_streams, V = s->dims.vocab_size;
     s->stats = litnice_b200_stats{};
     s->cur_streams = 0;  // as in forward: the uploaded prompt batch is gone
-    ensure_rows(s, (long long)B * seq_len);
-    ensure_attention_scratch(s, B, seq_len, seq_len);
+    if (!s->model) {
+      ensure_rows(s, (long long)B * seq_len);
+      ensure_attention_scratch(s, B, seq_len, seq_len);
+    } else {
+      model_reserve(s, B, seq_len, seq_len);
+    }
     upload_ids(s, ids, B, seq_len);
     const long long launches0 = s->launches;
     LB_CUDA(cudaEventRecord(s->ev0, s->st));
-    enqueue_body(s, B, seq_len);
-    enqueue_head_last(s, B, seq_len);
+    if (s->model) {
+      model_forward(s, B, seq_len, nullptr);
+    } else {
+      enqueue_body(s, B, seq_len);
+      enqueue_head_last(s, B, seq_len);
+    }
     launch_softmax_probs_f64(s->logits, V, B, s->probs, s->st);
     ++s->launches;
     LB_CUDA(cudaEventRecord(s->ev1, s->st));
@@ -1620,6 +1934,7 @@ int litnice_b200_profile_step(litnice_b200_session *s, int32_t n_streams, int32_
     if (n_streams <= 0 || n_streams > s->max_streams || seq_len <= 0 || seq_len > s->dims.max_seq_len ||
         repeats <= 0)
       throw std::invalid_argument("bad profile_step shape");
+    if (s->model) throw std::invalid_argument("profile_step covers the litnicelm transformer only");
     PdlScope pdl_scope(s->pdl);
     ensure_rows(s, (long long)n_streams * seq_len);
     ensure_attention_scratch(s, n_streams, seq_len, seq_len);

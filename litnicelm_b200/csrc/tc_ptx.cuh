@@ -166,6 +166,8 @@ __device__ __forceinline__ unsigned long long umma_desc_k128(unsigned smem_addr)
 __host__ __device__ constexpr unsigned umma_idesc_f16(int bn) {
   return (1u << 4) | ((unsigned)(bn >> 3) << 17) | ((unsigned)(TC_BM >> 4) << 24);
 }
+// bfloat16 operands (format code 1).
+__host__ __device__ constexpr unsigned umma_idesc_bf16(int bn) { return umma_idesc_f16(bn) | (1u << 7) | (1u << 10); }
 __host__ __device__ constexpr unsigned umma_idesc_tf32(int bn) {
   return (1u << 4) | (2u << 7) | (2u << 10) | ((unsigned)(bn >> 3) << 17) | ((unsigned)(TC_BM >> 4) << 24);
 }

@@ -306,3 +306,99 @@ def zipf_prompt(vocab: int, length: int, seed: int, s: float = 1.1) -> np.ndarra
     cdf /= cdf[-1]
     u = np.random.default_rng(seed).random(length)
     return np.minimum(np.searchsorted(cdf, u, side="left"), vocab - 1).astype(np.int32)
+
+
+# ---- model folders of the registered designs (config.json + model.safetensors) ----
+
+def to_bf16_bits(a: np.ndarray) -> np.ndarray:
+    """float32 -> bfloat16 bit patterns, round to nearest even."""
+    u = np.ascontiguousarray(a, np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16).reshape(np.shape(a))
+
+
+def from_bf16_bits(h: np.ndarray) -> np.ndarray:
+    return (h.astype(np.uint32) << 16).view(np.float32)
+
+
+def write_safetensors(path: str, tensors: Dict[str, np.ndarray]) -> None:
+    """Float arrays as bfloat16, in the given order: 8-byte little-endian header length, JSON header, data."""
+    header, at, blobs = {}, 0, []
+    for name, a in tensors.items():
+        a = np.asarray(a)
+        data = to_bf16_bits(a).tobytes() if a.dtype != np.uint16 else np.ascontiguousarray(a).tobytes()
+        header[name] = {"dtype": "BF16", "shape": list(a.shape), "data_offsets": [at, at + len(data)]}
+        at += len(data)
+        blobs.append(data)
+    text = json.dumps(header).encode()
+    text += b" " * (-len(text) % 8)
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(text)))
+        f.write(text)
+        for b in blobs:
+            f.write(b)
+
+
+def write_model_folder(folder: str, config: dict, tensors: Dict[str, np.ndarray]) -> None:
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(config, f, indent=1)
+    write_safetensors(os.path.join(folder, "model.safetensors"), tensors)
+
+
+def mitilix_config(width: int, vocab: int, max_positions: int, layers: List[dict], taps: int, eps: float) -> dict:
+    """config.json of a Mitilix model. layers: dicts with heads, dim, vdim, kv_rank, window, scale and
+    optionally kv_from and ff (absent: no feed-forward)."""
+    out = []
+    for l in layers:
+        mixer = {"heads": l["heads"], "dim": l["dim"], "vdim": l["vdim"], "kv_rank": l["kv_rank"],
+                 "mask": {"size": l["window"]}, "scale": l["scale"]}
+        if l.get("kv_from") is not None:
+            mixer["kv_from"] = l["kv_from"]
+        out.append({"type": "latent_attention", "mixer": mixer,
+                    "mlp": {"kind": "dense", "ff": l["ff"]} if l.get("ff") else None})
+    return {"architecture": "Mitilix", "width": width, "vocab": vocab, "max_positions": max_positions,
+            "canon": {"taps": taps}, "norm": {"eps": eps}, "layers": out}
+
+
+def mitilix_shapes(config: dict) -> Dict[str, Tuple[int, ...]]:
+    """Name and shape of every tensor of a Mitilix model."""
+    d, taps = config["width"], config["canon"]["taps"]
+    shapes: Dict[str, Tuple[int, ...]] = {"embed": (config["vocab"], d), "pos": (config["max_positions"], d)}
+    for i, e in enumerate(config["layers"]):
+        m, p = e["mixer"], f"l{i}."
+        q, o, r = m["heads"] * m["dim"], m["heads"] * m["vdim"], m["kv_rank"]
+        shapes[p + "norm1"] = ()
+        shapes[p + "mix.q"] = (q, d)
+        if m.get("kv_from") is None:
+            shapes[p + "mix.dkv"] = (r, d)
+            shapes[p + "mix.dkv.norm"] = (r,)
+        shapes[p + "mix.uk"] = (q, r)
+        shapes[p + "mix.uv"] = (o, r)
+        shapes[p + "mix.o"] = (d, o)
+        shapes[p + "canon1"] = (d, taps)
+        if e.get("mlp") is not None:
+            shapes[p + "mlp.up"] = (e["mlp"]["ff"], d)
+            shapes[p + "mlp.down"] = (d, e["mlp"]["ff"])
+            shapes[p + "canon2"] = (d, taps)
+    shapes["final.norm"] = ()
+    shapes["head"] = (config["vocab"], d)
+    return shapes
+
+
+def mitilix_random_weights(config: dict, seed: int) -> Dict[str, np.ndarray]:
+    """Random weights that keep the residual stream and the scores at a moderate size (rounded to bfloat16)."""
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in mitilix_shapes(config).items():
+        if name.endswith("norm1") or name == "final.norm" or name.endswith("dkv.norm"):
+            a = 1.0 + 0.2 * rng.standard_normal(shape)
+        elif "canon" in name:
+            a = 0.4 * rng.standard_normal(shape)
+        elif name == "embed":
+            a = rng.standard_normal(shape, dtype=np.float32)
+        elif name == "pos":
+            a = 0.3 * rng.standard_normal(shape, dtype=np.float32)
+        else:
+            a = rng.standard_normal(shape, dtype=np.float32) * (shape[-1] ** -0.5)
+        out[name] = from_bf16_bits(to_bf16_bits(np.asarray(a, np.float32)))
+    return out

@@ -126,6 +126,8 @@ NATIVE_SYMBOLS = [
     "litnice_b200_keep_step_logits", "litnice_b200_read_step_logits", "litnice_b200_forward",
     "litnice_b200_inspect", "litnice_b200_sample_logits", "litnice_b200_get_stats",
     "litnice_b200_gemv_noalloc",
+    "litnice_b200_session_create_model", "litnice_b200_architectures", "litnice_b200_model_dims",
+    "litnice_b200_extend", "litnice_b200_release",
 ]
 
 
@@ -346,8 +348,7 @@ class Session:
     """Native token loop: generate_text of the reference (inference.cpp:265-296)
     for n independent streams in lockstep, entirely on the GPU."""
 
-    def __init__(self, dims: ModelDims, max_streams: int = 1, lib_path: Optional[str] = None,
-                 device: Optional[int] = None):
+    def _bind(self, lib_path: Optional[str]):
         self.lib = load_library(lib_path)
         L = self.lib
         i32p, f32p, u32p = C.POINTER(C.c_int32), C.POINTER(C.c_float), C.POINTER(C.c_uint32)
@@ -371,6 +372,16 @@ class Session:
                                                  u32p, C.c_int32, i32p]
         L.litnice_b200_get_stats.argtypes = [C.c_void_p, C.POINTER(B200Stats)]
         L.litnice_b200_profile_step.argtypes = [C.c_void_p, C.c_int32, C.c_int32, C.c_int32]
+        L.litnice_b200_session_create_model.argtypes = [C.c_char_p, C.c_int32, C.c_int32, C.c_int32,
+                                                        C.POINTER(C.c_void_p)]
+        L.litnice_b200_model_dims.argtypes = [C.c_void_p, C.POINTER(B200Dims)]
+        L.litnice_b200_extend.argtypes = [C.c_void_p, C.c_int32, i32p, C.c_int32, i32p, C.c_int32, f32p]
+        L.litnice_b200_release.argtypes = [C.c_void_p, C.c_int32]
+        return L
+
+    def __init__(self, dims: ModelDims, max_streams: int = 1, lib_path: Optional[str] = None,
+                 device: Optional[int] = None):
+        L = self._bind(lib_path)
         self.dims = dims
         self.max_streams = max_streams
         cd = B200Dims(dims.n_layers, dims.n_heads, dims.d_model, dims.d_ff, dims.vocab, dims.max_seq,
@@ -510,3 +521,112 @@ class Session:
     def profile_step(self, n_streams: int, seq_len: int, repeats: int = 3) -> B200Stats:
         self._check(self.lib.litnice_b200_profile_step(self.h, n_streams, seq_len, repeats), "profile_step")
         return self.stats()
+
+
+DTYPES = {"bfloat16": 0, "float32": 1}
+
+
+def architectures(lib_path: Optional[str] = None) -> list:
+    """Names of the decoder designs the library serves from a model folder."""
+    lib = load_library(lib_path)
+    lib.litnice_b200_architectures.restype = C.c_char_p
+    return lib.litnice_b200_architectures().decode().split(",")
+
+
+class ModelSession(Session):
+    """The native loop on a model folder (config.json + model.safetensors) of a registered
+    design: everything a Session does on the slots' caches and state, plus ``extend`` and
+    ``release`` for sequences fed in portions."""
+
+    def __init__(self, model_dir: str, dtype: str = "bfloat16", max_streams: int = 1,
+                 lib_path: Optional[str] = None, device: int = -1):
+        L = self._bind(lib_path)
+        self.max_streams = max_streams
+        self.h = C.c_void_p()
+        rc = L.litnice_b200_session_create_model(os.fspath(model_dir).encode(), DTYPES[dtype], max_streams, device,
+                                                 C.byref(self.h))
+        if rc != 0:
+            msg = L.litnice_b200_last_error(self.h).decode()
+            if self.h:
+                L.litnice_b200_session_destroy(self.h)
+                self.h = None
+            raise NativeError(f"session_create_model failed ({rc}): {msg}")
+        d = B200Dims()
+        self._check(L.litnice_b200_model_dims(self.h, C.byref(d)), "model_dims")
+        self.dims = ModelDims(d.n_layers, 1, d.d_model, 0, d.vocab_size, d.max_seq_len)
+
+    def extend(self, slot: int, tokens, want=()) -> np.ndarray:
+        """Appends tokens to the sequence in `slot`; logits [len(want), vocab] of the wanted places."""
+        tokens = np.ascontiguousarray(tokens, dtype=np.int32)
+        want = np.ascontiguousarray(want, dtype=np.int32)
+        out = np.empty((len(want), self.dims.vocab), dtype=np.float32)
+        self._check(self.lib.litnice_b200_extend(self.h, slot, self._i32(tokens), len(tokens), self._i32(want), len(want),
+                                                 self._f32(out)), "extend")
+        return out
+
+    def release(self, slot: int):
+        rc = self.lib.litnice_b200_release(self.h, slot)
+        if rc != 0:
+            raise NativeError(f"release failed ({rc})")
+
+
+def bf16_product_host(a: np.ndarray, w: np.ndarray, engine: int, n_half: int = 0, gelu: bool = False,
+                      c: Optional[np.ndarray] = None, lib: Optional[C.CDLL] = None) -> np.ndarray:
+    """c[m, n] = a[m, k] w[n, k]^T on bfloat16 operands (litnice_b200_bf16_product_host); c given: added to."""
+    lib = lib or load_library()
+    f32p = C.POINTER(C.c_float)
+    fn = lib.litnice_b200_bf16_product_host
+    fn.argtypes = [C.c_int32, f32p, C.c_int32, C.c_int32, f32p, C.c_int32, C.c_int32, C.c_int32, C.c_int32, f32p]
+    a, w = np.ascontiguousarray(a, np.float32), np.ascontiguousarray(w, np.float32)
+    m, k = a.shape
+    n = w.shape[0]
+    out = np.zeros((m, n), np.float32) if c is None else np.array(c, np.float32, order="C")
+    p = lambda x: x.ctypes.data_as(f32p)
+    rc = fn(engine, p(a), m, k, p(w), n, n_half, int(gelu), int(c is not None), p(out))
+    if rc != 0:
+        raise RuntimeError(f"litnice_b200_bf16_product_host failed with status {rc}")
+    return out
+
+
+def rms_canon_host(x: np.ndarray, gain: float, eps: float, w1: np.ndarray, w2: Optional[np.ndarray] = None,
+                   portions: Optional[Sequence[int]] = None, dtype: str = "float32", lib: Optional[C.CDLL] = None):
+    """(h + conv1(h), h + conv2(h) or None) with h the scalar-gain RMS norm of x (litnice_b200_rms_canon_host)."""
+    lib = lib or load_library()
+    f32p, i32p = C.POINTER(C.c_float), C.POINTER(C.c_int32)
+    fn = lib.litnice_b200_rms_canon_host
+    fn.argtypes = [C.c_int32, f32p, C.c_int32, C.c_int32, C.c_float, C.c_float, C.c_int32, f32p, f32p, i32p, C.c_int32,
+                   f32p, f32p]
+    x = np.ascontiguousarray(x, np.float32)
+    n, d = x.shape
+    w1 = np.ascontiguousarray(w1, np.float32)
+    por = np.ascontiguousarray([n] if portions is None else portions, np.int32)
+    o1 = np.empty((n, d), np.float32)
+    p = lambda v: None if v is None else v.ctypes.data_as(f32p)
+    o2 = None
+    if w2 is not None:
+        w2, o2 = np.ascontiguousarray(w2, np.float32), np.empty((n, d), np.float32)
+    rc = fn(DTYPES[dtype], p(x), n, d, gain, eps, w1.shape[1], p(w1), p(w2), por.ctypes.data_as(i32p), len(por), p(o1), p(o2))
+    if rc != 0:
+        raise RuntimeError(f"litnice_b200_rms_canon_host failed with status {rc}")
+    return o1, o2
+
+
+def latent_attention_host(engine: int, q: np.ndarray, dkv: np.ndarray, gain: np.ndarray, eps: float, w_uk: np.ndarray,
+                          w_uv: np.ndarray, heads: int, dim: int, vdim: int, scale: float, window: int,
+                          lib: Optional[C.CDLL] = None) -> np.ndarray:
+    """q [streams, n, heads * dim], dkv [streams, T, rank]: outputs of the last n positions
+    (litnice_b200_latent_attention_host)."""
+    lib = lib or load_library()
+    f32p = C.POINTER(C.c_float)
+    fn = lib.litnice_b200_latent_attention_host
+    fn.argtypes = [C.c_int32, f32p, f32p, f32p, C.c_float, f32p, f32p] + [C.c_int32] * 7 + [C.c_float, C.c_int32, f32p]
+    arrs = [np.ascontiguousarray(v, np.float32) for v in (q, dkv, gain, w_uk, w_uv)]
+    q, dkv, gain, w_uk, w_uv = arrs
+    b, n = q.shape[:2]
+    t, rank = dkv.shape[1:]
+    out = np.empty((b, n, heads * vdim), np.float32)
+    p = lambda v: v.ctypes.data_as(f32p)
+    rc = fn(engine, p(q), p(dkv), p(gain), eps, p(w_uk), p(w_uv), b, t - n, n, heads, dim, vdim, rank, scale, window, p(out))
+    if rc != 0:
+        raise RuntimeError(f"litnice_b200_latent_attention_host failed with status {rc}")
+    return out
