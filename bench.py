@@ -16,6 +16,9 @@ prints one JSON line. Beside the headline the default line carries: `parity`
 `extra` (config 3: 64 lockstep streams with the fused sampler; config 5 cut
 over the GPUs; config 2 in the opt-in cached mode).
 
+`--design mitilix` measures a registered decoder design instead (prefill and decode at a few
+sizes, beside the transformer of equal size), one JSON line per size.
+
 `--impl reference` times the reference's own CPU backend (oracle/_ref, built
 from the reference sources) on a bounded sample of the same workload.
 """
@@ -692,6 +695,163 @@ def check_prefill_against_fixture(probs: np.ndarray) -> dict:
     return out
 
 
+# The registered design's throughput arm: sizes that resemble a real model's layers, and the litnicelm
+# transformer of equal size (same layers, width, heads, head dimension, feed-forward and vocabulary).
+# heads, dim, vdim, kv_rank, window, ff: one layer's sizes; every third layer shares the latents before it.
+DESIGN_SIZES = {
+    "d512": dict(n_layers=6, width=512, heads=8, dim=64, vdim=64, kv_rank=128, window=512, ff=2048, vocab=8192),
+    "d1024": dict(n_layers=12, width=1024, heads=16, dim=64, vdim=64, kv_rank=256, window=1024, ff=4096, vocab=32000),
+    "d2048": dict(n_layers=12, width=2048, heads=32, dim=64, vdim=64, kv_rank=512, window=1024, ff=8192, vocab=32000),
+    "d2048h128": dict(n_layers=12, width=2048, heads=16, dim=128, vdim=128, kv_rank=512, window=1024, ff=8192,
+                      vocab=32000),
+}
+DESIGN_PREFILL = (8, 2048)       # sequences x tokens
+DESIGN_CONTEXT = 1024            # decoding starts behind a prompt of this length
+DESIGN_STREAMS = (1, 8, 64)
+DESIGN_NEW = 64                  # timed tokens per stream
+
+
+def design_config(z: dict) -> dict:
+    layers = [{"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"], "window": z["window"],
+               "scale": z["dim"] ** -0.5, "ff": z["ff"], "kv_from": i - 1 if i % 3 == 2 else None}
+              for i in range(z["n_layers"])]
+    return formats.mitilix_config(z["width"], z["vocab"], 2048, layers, taps=4, eps=1e-6)
+
+
+def design_weights(config: dict, seed: int):
+    """Random bfloat16 weights of the configuration's shapes, drawn on the device."""
+    import torch
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    out = {}
+    for name, shape in formats.mitilix_shapes(config).items():
+        if name.endswith("norm1") or name in ("final.norm",) or name.endswith("dkv.norm"):
+            t = torch.ones(shape, device="cuda")
+        else:
+            fan = 1.0 if name in ("embed", "pos") else shape[-1]
+            t = torch.randn(shape, generator=g, device="cuda") * fan ** -0.5
+        out[name] = t.to(torch.bfloat16).view(torch.int16).cpu().numpy().view(np.uint16)
+    return out
+
+
+def design_work(z: dict, config: dict):
+    """Algorithmic flops per prefill token (projections) and per visible key (attention), and the bytes of the
+    layers' and the head's weights a decoding step reads."""
+    d, n = z["width"], z["n_layers"]
+    own = sum(e["mixer"].get("kv_from") is None for e in config["layers"])
+    q, o, r = z["heads"] * z["dim"], z["heads"] * z["vdim"], z["kv_rank"]
+    per_layer = d * q + r * (q + o) + d * o + 2 * d * z["ff"]
+    weights = n * per_layer + own * d * r
+    return 2.0 * weights, 2.0 * n * (q + o), 2.0 * (weights + d * z["vocab"]), 2.0 * n * r
+
+
+def measure_session(box, sess, vocab, steps, warmup, streams_list, context, new, prefill):
+    """Device-timed prefill (last-row logits) and greedy decoding of one session, medians over `steps`."""
+    rng = np.random.default_rng(5)
+    out = {"prefill": None, "decode": {}}
+    b, s = prefill
+    ids = rng.integers(0, vocab, (b, s)).astype(np.int32)
+    ms = []
+    for i in range(warmup + steps):
+        box.flush.fill_(1)
+        box.torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        sess.forward(ids)
+        wall = (time.perf_counter() - t0) * 1e3
+        ms.append((sess.stats().device_ms, wall))
+    ms = ms[warmup:]
+    dev = statistics.median(m[0] for m in ms)
+    out["prefill"] = {"sequences": b, "tokens": s, "ms": dev, "tokens_per_s": b * s / dev * 1e3,
+                      "e2e_ms": statistics.median(m[1] for m in ms), "launches": int(sess.stats().kernel_launches)}
+    for n in streams_list:
+        prompts = rng.integers(0, vocab, (n, context)).astype(np.int32)
+        per = []
+        for i in range(2 + steps):
+            sess.upload_prompts(prompts)
+            sess.run(4)                       # the prompt and the first steps (captures)
+            sess.run(new)
+            st = sess.stats()
+            per.append((st.device_ms / new, st.kernel_launches))
+        per = per[2:]
+        t = statistics.median(p[0] for p in per)
+        out["decode"][str(n)] = {"ms_per_token": t, "tokens_per_s": n / t * 1e3, "launches_per_token": per[-1][1] / new}
+    return out
+
+
+def run_design_arm(args, rank, local_rank, world):
+    """Prefill and decode throughput of the registered design beside the litnicelm transformer of equal size (its
+    cached mode for decoding, its whole-context pass for prefill). One JSON line per size."""
+    import shutil
+    from litnicelm_b200.plugin import ModelSession, Session
+    if world > 1:
+        raise SystemExit("--design runs on one GPU")
+    box = Box(rank, local_rank, world)
+    peaks = load_peaks()
+    names = args.design_sizes.split(",") if args.design_sizes else list(DESIGN_SIZES)
+    for name in names:
+        z = DESIGN_SIZES[name]
+        config = design_config(z)
+        folder = tempfile.mkdtemp(prefix="mitilix_")
+        clocks = ClockSampler(local_rank)
+        try:
+            formats.write_model_folder(folder, config, design_weights(config, 3))
+            with ModelSession(folder, "bfloat16", max(DESIGN_STREAMS)) as sess:
+                clocks.start()
+                ours = measure_session(box, sess, z["vocab"], args.steps, args.warmup, DESIGN_STREAMS, DESIGN_CONTEXT,
+                                       DESIGN_NEW, DESIGN_PREFILL)
+                clock_info = clocks.stop()
+        finally:
+            shutil.rmtree(folder, ignore_errors=True)
+        proj, per_key, wbytes, cbytes = design_work(z, config)
+        s, w = DESIGN_PREFILL[1], z["window"]
+        keys = sum(min(i + 1, w) for i in range(s)) / s
+        pf = ours["prefill"]
+        tflops = pf["tokens_per_s"] * (proj + per_key * keys) / 1e12
+        pf.update(achieved_tflops=tflops, frac_of_bf16_peak=tflops / peaks["bf16_tflops"])
+        for n, d in ours["decode"].items():
+            by = wbytes + int(n) * cbytes * min(w, DESIGN_CONTEXT)
+            d.update(bytes_per_step=by, achieved_gbs=by / (d["ms_per_token"] * 1e-3) / 1e9)
+            d["frac_of_hbm_peak"] = d["achieved_gbs"] / peaks["hbm_gbs"]
+        base = None
+        if not args.no_extras and z["dim"] == 64 and z["heads"] * z["dim"] == z["width"]:
+            gd = formats.ModelDims(z["n_layers"], z["heads"], z["width"], z["ff"], z["vocab"], 2048)
+            arena = formats.make_param_arena(gd, 1004)
+            base = {}
+            with Session(gd, DESIGN_PREFILL[0]) as sess:
+                sess.load_params(arena)
+                base["prefill"] = measure_session(box, sess, z["vocab"], args.steps, args.warmup, (), DESIGN_CONTEXT,
+                                                  DESIGN_NEW, DESIGN_PREFILL)["prefill"]
+            os.environ["LITNICE_B200_KV_CACHE"] = "1"
+            if z["width"] > 1024:             # the resident kernel's CTAs do not fit an SM at this width
+                os.environ["LITNICE_B200_KV_PERSIST"] = "0"
+            try:
+                with Session(gd, max(DESIGN_STREAMS)) as sess:
+                    sess.load_params(arena)
+                    base["decode"] = measure_session(box, sess, z["vocab"], args.steps, 1, DESIGN_STREAMS, DESIGN_CONTEXT,
+                                                     DESIGN_NEW, (1, 64))["decode"]
+            finally:
+                del os.environ["LITNICE_B200_KV_CACHE"]
+                os.environ.pop("LITNICE_B200_KV_PERSIST", None)
+            keys = (s + 1) / 2
+            flops = gd.n_layers * (2.0 * (4 * gd.d_model ** 2 + 2 * gd.d_model * gd.d_ff) + 4.0 * gd.d_model * keys)
+            b = base["prefill"]
+            b["achieved_tflops"] = b["tokens_per_s"] * flops / 1e12
+            b["frac_of_bf16_peak"] = b["achieved_tflops"] / peaks["bf16_tflops"]
+            for n, d in base["decode"].items():
+                by = 4.0 * (gd.n_layers * (4 * gd.d_model ** 2 + 2 * gd.d_model * gd.d_ff) + gd.d_model * gd.vocab)
+                by += int(n) * 8.0 * gd.n_layers * gd.d_model * DESIGN_CONTEXT
+                d.update(bytes_per_step=by, achieved_gbs=by / (d["ms_per_token"] * 1e-3) / 1e9)
+                d["frac_of_hbm_peak"] = d["achieved_gbs"] / peaks["hbm_gbs"]
+        print(json.dumps({
+            "metric": "prefill and decode throughput of a registered design", "design": "Mitilix", "size": name,
+            "sizes": z, "value": pf["tokens_per_s"], "unit": "prefill tokens/s", "higher_is_better": True,
+            "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "dtype": "bf16", "data": "synthetic",
+            "design_figures": ours, "transformer_of_equal_size": base,
+            "peaks": peaks, "clocks": clock_info,
+            "l2": "256 MB buffer written before each prefill; a decoding step's weights exceed L2 from d1024 on"}),
+            flush=True)
+    box.close()
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -704,6 +864,9 @@ def main():
                     help="run the workload in the opt-in cached mode (an extension; not the headline)")
     ap.add_argument("--no-extras", action="store_true",
                     help="skip the output-head bandwidth block and the config-3 / config-5 side measurements")
+    ap.add_argument("--design", default=None, choices=["mitilix"],
+                    help="throughput of a registered decoder design beside the transformer of equal size (not the headline)")
+    ap.add_argument("--design-sizes", default="", help="sizes of --design to run, with commas between them (default: all)")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
@@ -715,6 +878,9 @@ def main():
         return
     if args.warmup < 3:
         args.warmup = 3
+    if args.design:
+        run_design_arm(args, rank, local_rank, world)
+        return
     if args.workload == "c4":
         run_prefill_arm(args, rank, local_rank, world)
         return

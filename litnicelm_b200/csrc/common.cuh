@@ -331,6 +331,11 @@ size_t sampler_scratch_bytes(int vocab);
 void launch_sampler(const float *logits, int vocab, int n_streams, const SamplerParams &sp,
                     unsigned *mt_state, int *ids, int ids_ld, int *out_tokens, int out_ld,
                     LoopState *state, void *scratch, cudaStream_t st);
+// Greedy selection, append and state advance in one launch for large vocabularies. best: one word per
+// stream, all ones at rest; done: one counter, zero at rest.
+bool greedy_select_supports(int vocab);
+void launch_greedy_select(const float *logits, int vocab, int n_streams, unsigned long long *best, unsigned *done, int *ids,
+                          int ids_ld, int *out_tokens, int out_ld, LoopState *state, cudaStream_t st);
 void launch_sampler_rows(const float *logits, int vocab, int n_rows, const SamplerParams &sp,
                          unsigned *mt_state, int draws, int *out, void *scratch, cudaStream_t st);
 void launch_mt_seed(unsigned *mt_state, const unsigned *seeds, int n, cudaStream_t st);

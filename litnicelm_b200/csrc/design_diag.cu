@@ -240,13 +240,13 @@ int litnice_b200_latent_attention_host(int32_t engine, const float *q, const flo
     b.n = n;
     b.s_cap = T;
     const float *fresh = slice(p0, n);
-    if (engine <= 1 || engine == 2) {
-      launch_latent_store(fresh, rank, gain, eps, a.cache, nullptr, 0, 0, type, b, nullptr);
+    if (engine <= 2) {
+      if (engine != 2) launch_latent_store(fresh, rank, gain, eps, a.cache, nullptr, 0, 0, type, b, nullptr);
       if (engine == 2) {
         if (!latent_decode_supports(a)) return LITNICE_B200_EINVAL;
         float *scratch = static_cast<float *>(
             dev.alloc(latent_decode_scratch_floats(heads, rank, window, T, b.rows()) * 4));
-        launch_latent_decode(a, scratch, b, nullptr);
+        launch_latent_decode(a, LatentFresh{fresh, rank, gain, eps}, scratch, b, nullptr);
       } else {
         launch_latent_attention_rows(a, type, b, nullptr);
       }

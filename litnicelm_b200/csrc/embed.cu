@@ -129,9 +129,9 @@ __global__ void advance_state_kernel(LoopState *state) {
 
 // The rows of a batch (new positions only): x[r, :] = table[ids[slot, p]] + pos[p], in 32-bit.
 template <typename T>
-__global__ void embed_rows_kernel(const T *__restrict__ table, const T *__restrict__ pos, const int *__restrict__ ids,
+__global__ void embed_rows_kernel(const T *__restrict__ table, const T *__restrict__ pos, const int *ids,
                                   int ids_ld, const LoopState *state, int p0_host, int n, int slot0, int d, int vocab,
-                                  float *__restrict__ x, DevErr *err) {
+                                  float *x, DevErr *err) {
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.y, t = blockIdx.x;
@@ -146,6 +146,23 @@ __global__ void embed_rows_kernel(const T *__restrict__ table, const T *__restri
   }
   const T *tp = table + (long long)id * d, *pp = pos + (long long)p * d;
   float *xp = x + ((long long)b * n + t) * d;
+  if ((d & 3) == 0) {
+    for (int c = threadIdx.x * 4; c < d; c += blockDim.x * 4) {
+      float4 v;
+      if (sizeof(T) == 2) {  // two bfloat16 per word
+        const uint2 a = *reinterpret_cast<const uint2 *>(tp + c), q = *reinterpret_cast<const uint2 *>(pp + c);
+        v = make_float4(__uint_as_float(a.x << 16) + __uint_as_float(q.x << 16),
+                        __uint_as_float(a.x & 0xffff0000u) + __uint_as_float(q.x & 0xffff0000u),
+                        __uint_as_float(a.y << 16) + __uint_as_float(q.y << 16),
+                        __uint_as_float(a.y & 0xffff0000u) + __uint_as_float(q.y & 0xffff0000u));
+      } else {
+        const float4 a = *reinterpret_cast<const float4 *>(tp + c), q = *reinterpret_cast<const float4 *>(pp + c);
+        v = make_float4(a.x + q.x, a.y + q.y, a.z + q.z, a.w + q.w);
+      }
+      *reinterpret_cast<float4 *>(xp + c) = v;
+    }
+    return;
+  }
   for (int c = threadIdx.x; c < d; c += blockDim.x) xp[c] = (float)tp[c] + (float)pp[c];
 }
 

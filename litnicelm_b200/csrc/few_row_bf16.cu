@@ -6,8 +6,11 @@
 // warps take interleaved blocks of 64 k, and their sums meet in shared memory. The order of k inside a
 // dot product is free, so a lane loads 16 consecutive bytes (8 k) of its W row and of its activation
 // row and feeds them to two k-steps as they lie: no shared memory, no shuffles, whole 128-byte lines
-// of W per warp and row. Up to two products with inputs of their own share a launch.
+// of W per warp and row. Up to two products with inputs of their own share a launch. Where the columns
+// alone give too few CTAs, k is cut over the CTAs of a thread-block cluster, whose sums meet in the shared
+// memory of the rank that stores them (rank order, so results do not depend on scheduling).
 #include "model.cuh"
+#include "tc_ptx.cuh"
 
 #include <cuda_bf16.h>
 
@@ -43,8 +46,8 @@ __device__ __forceinline__ uint4 ld_stream(const bf16 *p) {  // weights: read on
 // NT: tiles of 8 activation rows; UNROLL: blocks of 32 k in flight per lane and row.
 template <int NT, int UNROLL>
 __global__ void __launch_bounds__(FR_WARPS * 32)
-few_row_bf16_kernel(FewRowPair pair, int m) {
-  __shared__ float red[FR_WARPS][NT][FR_COLS][8];
+few_row_bf16_kernel(FewRowPair pair, int m, int ranks) {
+  __shared__ __align__(16) float red[FR_WARPS][NT][FR_COLS][8];
   const bool second = (int)blockIdx.x >= pair.blocks0;
   const Bf16Product &p = pair.p[second ? 1 : 0];
   const int n0 = ((int)blockIdx.x - (second ? pair.blocks0 : 0)) * FR_COLS;
@@ -54,13 +57,16 @@ few_row_bf16_kernel(FewRowPair pair, int m) {
   const bool v0 = n0 + g < p.n, v1 = n0 + g + 8 < p.n;
   const bf16 *w0 = w + (long long)(n0 + g) * p.w_ld + t * 8, *w1 = w0 + (long long)8 * p.w_ld;
   constexpr int SPAN = 32 * UNROLL;  // k per warp and trip
+  // this CTA's range of k, in whole spans
+  const int per = ((k8 + SPAN - 1) / SPAN + ranks - 1) / ranks * SPAN;
+  const int k_begin = min(k8, (int)blockIdx.z * per), k_end = min(k8, k_begin + per);
   const uint4 zero = make_uint4(0, 0, 0, 0);
   uint4 wa[UNROLL], wb[UNROLL];
   auto load_w = [&](int k0) {
 #pragma unroll
     for (int u = 0; u < UNROLL; ++u) {
       const int k = k0 + u * 32;
-      const bool in = k + t * 8 < k8;
+      const bool in = k + t * 8 < k_end;
       wa[u] = in && v0 ? ld_stream(w0 + k) : zero;
       wb[u] = in && v1 ? ld_stream(w1 + k) : zero;
     }
@@ -71,9 +77,9 @@ few_row_bf16_kernel(FewRowPair pair, int m) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
   pdl_launch_dependents();
-  load_w(wid * SPAN);  // the weights do not depend on the predecessor
+  load_w(k_begin + wid * SPAN);  // the weights do not depend on the predecessor
   pdl_wait();
-  for (int k0 = wid * SPAN; k0 < k8; k0 += FR_WARPS * SPAN) {
+  for (int k0 = k_begin + wid * SPAN; k0 < k_end; k0 += FR_WARPS * SPAN) {
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
       const int row = i * 8 + g;
@@ -82,7 +88,7 @@ few_row_bf16_kernel(FewRowPair pair, int m) {
 #pragma unroll
       for (int u = 0; u < UNROLL; ++u) {
         const int k = k0 + u * 32;
-        x[u] = row < m && k + t * 8 < k8 ? *reinterpret_cast<const uint4 *>(ar + k) : zero;
+        x[u] = row < m && k + t * 8 < k_end ? *reinterpret_cast<const uint4 *>(ar + k) : zero;
       }
 #pragma unroll
       for (int u = 0; u < UNROLL; ++u) {
@@ -90,7 +96,7 @@ few_row_bf16_kernel(FewRowPair pair, int m) {
         fr_mma(acc[i], wa[u].z, wb[u].z, wa[u].w, wb[u].w, x[u].z, x[u].w);
       }
     }
-    if (k0 + FR_WARPS * SPAN < k8) load_w(k0 + FR_WARPS * SPAN);
+    if (k0 + FR_WARPS * SPAN < k_end) load_w(k0 + FR_WARPS * SPAN);
   }
 #pragma unroll
   for (int i = 0; i < NT; ++i) {
@@ -98,13 +104,34 @@ few_row_bf16_kernel(FewRowPair pair, int m) {
     *reinterpret_cast<float2 *>(&red[wid][i][g + 8][t * 2]) = make_float2(acc[i][2], acc[i][3]);
   }
   __syncthreads();
-  for (int e = threadIdx.x; e < NT * 8 * FR_COLS; e += FR_WARPS * 32) {
+  constexpr int TILE = NT * FR_COLS * 8;  // one warp's sums
+  int e_begin = 0, e_end = TILE;
+  if (ranks > 1) {  // the warps' sums first, in place; each rank then finishes its share of the tile
+    float *flat = &red[0][0][0][0];
+    for (int e = threadIdx.x; e < TILE; e += FR_WARPS * 32) {
+      float v = 0.f;
+#pragma unroll
+      for (int q = 0; q < FR_WARPS; ++q) v += flat[q * TILE + e];
+      flat[e] = v;  // this thread alone reads and writes element e of every warp
+    }
+    __syncwarp();
+    cluster_sync_all();
+    const int share = (TILE + ranks - 1) / ranks;
+    e_begin = min(TILE, (int)blockIdx.z * share);
+    e_end = min(TILE, e_begin + share);
+  }
+  for (int e = e_begin + threadIdx.x; e < e_end; e += FR_WARPS * 32) {
     const int c = e & (FR_COLS - 1), row = e / FR_COLS;
     const int col = n0 + c;
     if (row >= m || col >= p.n) continue;
     float v = 0.f;
+    if (ranks > 1) {
+      const unsigned at = smem_u32(&red[0][row >> 3][c][row & 7]);
+      for (int q = 0; q < ranks; ++q) v += ld_cluster_f32(cluster_map(at, (unsigned)q));
+    } else {
 #pragma unroll
-    for (int q = 0; q < FR_WARPS; ++q) v += red[q][row >> 3][c][row & 7];
+      for (int q = 0; q < FR_WARPS; ++q) v += red[q][row >> 3][c][row & 7];
+    }
     if (col < p.n_half) {
       if (p.gelu) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
       static_cast<bf16 *>(p.half_out)[(long long)row * p.half_ld + col] = __float2bfloat16_rn(v);
@@ -113,6 +140,8 @@ few_row_bf16_kernel(FewRowPair pair, int m) {
       *o = p.accumulate ? *o + v : v;
     }
   }
+  __syncwarp();
+  if (ranks > 1) cluster_sync_all();  // a rank's shared memory stays until every other has read it
 }
 
 }  // namespace
@@ -126,12 +155,27 @@ void launch_few_row_bf16(const Bf16Product *p, int count, int m, cudaStream_t st
     blocks += (unsigned)((p[i].n + FR_COLS - 1) / FR_COLS);
     if (i == 0) pair.blocks0 = (int)blocks;
   }
-  const dim3 grid(blocks), block(FR_WARPS * 32);
+  int k_max = 0;
+  for (int i = 0; i < count; ++i) k_max = p[i].k > k_max ? p[i].k : k_max;
+  // ranks of a cluster that share a tile's k: enough CTAs for two per SM, at least 512 k each
+  int ranks = 1;
+  while (ranks < 8 && blocks * ranks < 2 * 148 && k_max >= 1024 * ranks) ranks *= 2;
+  const dim3 grid(blocks, 1, (unsigned)ranks), block(FR_WARPS * 32);
+  auto go = [&](auto kernel) {
+    launch_pdl_cluster(kernel, grid, block, 0, st, g_pdl_enabled, (unsigned)ranks, pair, m, ranks);
+  };
   const int nt = (m + 7) / 8;
-  if (nt <= 1) launch_pdl(few_row_bf16_kernel<1, 4>, grid, block, 0, st, g_pdl_enabled, pair, m);
-  else if (nt <= 2) launch_pdl(few_row_bf16_kernel<2, 4>, grid, block, 0, st, g_pdl_enabled, pair, m);
-  else if (nt <= 4) launch_pdl(few_row_bf16_kernel<4, 4>, grid, block, 0, st, g_pdl_enabled, pair, m);
-  else launch_pdl(few_row_bf16_kernel<8, 4>, grid, block, 0, st, g_pdl_enabled, pair, m);
+  if (ranks > 1) {  // shorter ranges: two blocks of 32 k per lane and trip keep every warp busy
+    if (nt <= 1) go(few_row_bf16_kernel<1, 2>);
+    else if (nt <= 2) go(few_row_bf16_kernel<2, 2>);
+    else if (nt <= 4) go(few_row_bf16_kernel<4, 2>);
+    else go(few_row_bf16_kernel<8, 2>);
+    return;
+  }
+  if (nt <= 1) go(few_row_bf16_kernel<1, 4>);
+  else if (nt <= 2) go(few_row_bf16_kernel<2, 4>);
+  else if (nt <= 4) go(few_row_bf16_kernel<4, 4>);
+  else go(few_row_bf16_kernel<8, 4>);
 }
 
 }  // namespace lb

@@ -10,10 +10,10 @@
 //   latent_store_kernel          RMS norm of the new rows' W_dkv h into the cache, and the window's rows
 //                                side by side for the expanding kernels (latent_attention_tc.cu)
 //   latent_attention_rows_kernel any size, one CTA per row and head, float or bfloat16 storage
-//   latent_query / latent_chunk / latent_join   few rows on bfloat16: the absorbed query per head; key
-//                                chunks of 64 for 16 heads at a time on mma.sync tiles, the fp32 query
-//                                and weights entering as two bfloat16 terms each; the join of the chunks
-//                                followed by W_uv
+//   latent_query / latent_chunk / latent_join   few rows on bfloat16: the absorbed query per head (and the
+//                                new latents into the cache, by CTAs of their own); splits of the window
+//                                for 16 heads at a time on mma.sync tiles, the 32-bit query and weights
+//                                entering as two bfloat16 terms each; the join of the splits and W_uv
 // Scores, weights and norms are 32-bit throughout.
 #include "model.cuh"
 
@@ -30,6 +30,15 @@ __device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void put(float *p, float v) { *p = v; }
 __device__ __forceinline__ void put(bf16 *p, float v) { *p = __float2bfloat16_rn(v); }
 
+__device__ __forceinline__ void put4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void put4(bf16 *p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<const unsigned *>(&a);
+  u.y = *reinterpret_cast<const unsigned *>(&b);
+  *reinterpret_cast<uint2 *>(p) = u;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -43,13 +52,47 @@ __device__ __forceinline__ float warp_max(float v) {
 
 // ---- latents -------------------------------------------------------------------
 
+// The latent of one new position by one warp: RMS norm of its W_dkv h row, zeros behind the rank.
+template <typename T>
+__device__ __forceinline__ void store_latent(const float *src, const float *__restrict__ gain, float eps, int rank,
+                                             int ld, T *row, T *copy, int lane) {
+  float s = 0.f;
+  if ((rank & 3) == 0 && rank <= 1024) {  // the row in registers, four columns per lane and piece
+    float4 v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int c = (i * 32 + lane) * 4;
+      v[i] = c < rank ? *reinterpret_cast<const float4 *>(src + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      s += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(s) / (float)rank + eps);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int c = (i * 32 + lane) * 4;
+      if (c >= ld) break;
+      const float4 g = c < rank ? *reinterpret_cast<const float4 *>(gain + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 o = make_float4(v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z, v[i].w * inv * g.w);
+      put4(row + c, o);
+      if (copy) put4(copy + c, o);
+    }
+    return;
+  }
+  for (int c = lane; c < rank; c += 32) s = fmaf(src[c], src[c], s);
+  const float inv = 1.0f / sqrtf(warp_sum(s) / (float)rank + eps);
+  for (int c = lane; c < ld; c += 32) {
+    const float v = c < rank ? src[c] * inv * gain[c] : 0.f;
+    put(row + c, v);
+    if (copy) put(copy + c, v);
+  }
+}
+
 // One warp per position: positions first .. p0 + n - 1 (first <= p0) of stream b. Old positions are
 // copied from the cache to the packed rows, new ones normalised (dkv given) or, for a layer that uses
 // another layer's latents, copied as well.
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_store_kernel(const float *__restrict__ dkv, int dkv_ld, const float *__restrict__ gain, float eps, T *__restrict__ cache,
-                    int cap, int ld, int rank, T *__restrict__ packed, int packed_rows, int first, int n, int p0_host,
+latent_store_kernel(const float *dkv, int dkv_ld, const float *__restrict__ gain, float eps, T *cache,
+                    int cap, int ld, int rank, T *packed, int packed_rows, int first, int n, int p0_host,
                     const LoopState *state, int slot0) {
   pdl_launch_dependents();
   pdl_wait();
@@ -67,15 +110,7 @@ latent_store_kernel(const float *__restrict__ dkv, int dkv_ld, const float *__re
     for (int c = lane; c < ld * (int)sizeof(T) / 16; c += 32) dst4[c] = src4[c];
     return;
   }
-  const float *src = dkv + ((long long)b * n + (p - p0)) * dkv_ld;
-  float s = 0.f;
-  for (int c = lane; c < rank; c += 32) s = fmaf(src[c], src[c], s);
-  const float inv = 1.0f / sqrtf(warp_sum(s) / (float)rank + eps);
-  for (int c = lane; c < ld; c += 32) {
-    const float v = c < rank ? src[c] * inv * gain[c] : 0.f;
-    put(row + c, v);
-    if (dst) put(dst + c, v);
-  }
+  store_latent(dkv + ((long long)b * n + (p - p0)) * dkv_ld, gain, eps, rank, ld, row, dst, lane);
 }
 
 // ---- any size ------------------------------------------------------------------
@@ -85,9 +120,9 @@ constexpr int LR_KEYS = 64;  // keys per pass
 
 template <typename T>
 __global__ void __launch_bounds__(LR_THREADS)
-latent_attention_rows_kernel(const T *__restrict__ q, int q_ld, const T *__restrict__ w_uk, const T *__restrict__ w_uv,
-                             int w_ld, const T *__restrict__ cache, int cap, int ld, int rank, int dim, int vdim, float scale,
-                             int window, T *__restrict__ out, int out_ld, int n, int p0_host, const LoopState *state,
+latent_attention_rows_kernel(const T *q, int q_ld, const T *__restrict__ w_uk, const T *__restrict__ w_uv,
+                             int w_ld, const T *cache, int cap, int ld, int rank, int dim, int vdim, float scale,
+                             int window, T *out, int out_ld, int n, int p0_host, const LoopState *state,
                              int slot0) {
   extern __shared__ float sm[];
   float *qa = sm;              // [rank] absorbed, scaled query
@@ -150,11 +185,11 @@ latent_attention_rows_kernel(const T *__restrict__ q, int q_ld, const T *__restr
 
 // ---- few rows on bfloat16 --------------------------------------------------------
 
-constexpr int LD_KEYS = 64;      // keys per chunk
+constexpr int LD_KEYS = 64;      // keys per tile
 constexpr int LD_HEADS = 16;     // heads per CTA: the rows of an mma tile
 constexpr int LD_THREADS = 256;
-constexpr int LQ_COLS = 64;      // latent columns per CTA of the query kernel
-constexpr int LQ_ROWS = 4;       // rows per CTA of the query kernel
+constexpr int LQ_COLS = 256;     // latent columns per CTA of the query kernel, eight per thread
+constexpr int LD_ROWS = 4;       // rows per CTA of the query and join kernels
 constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
@@ -167,223 +202,368 @@ __device__ __forceinline__ void ldmatrix_x2_trans(unsigned &r0, unsigned &r1, co
   const unsigned addr = (unsigned)__cvta_generic_to_shared(p);
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
 }
+// 16 bytes to shared memory in the background; bytes = 0 stores zeros.
+__device__ __forceinline__ void copy16(void *dst, const void *src, int bytes) {
+  const unsigned addr = (unsigned)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(addr), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void copy_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
 __device__ __forceinline__ void split2(float v, bf16 &hi, bf16 &lo) {
   hi = __float2bfloat16_rn(v);
   lo = __float2bfloat16_rn(v - __bfloat162float(hi));
 }
+__device__ __forceinline__ void unpack8(uint4 v, float (&f)[8]) {
+  const unsigned u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    f[2 * i] = __uint_as_float(u[i] << 16);
+    f[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+  }
+}
 
-// qa[r, h, c] = scale * log2(e) * sum_e q[r, h, e] W_uk[h, e, c]: LQ_COLS columns of one head for up to
-// LQ_ROWS rows; the four thread groups of a CTA take quarters of e.
+// What the few-row kernels share. The absorbed queries are [rows][heads16][rk] in two bfloat16 terms
+// (heads16: heads rounded up to 16, rk: rank rounded up to 16), the partial results [rows][heads][splits].
+struct LdShape {
+  int heads, heads16, dim, vdim, rank, rk, rank4, window, splits, span;  // span: keys per split, a multiple of LD_KEYS
+  int n, p0, slot0;
+  const LoopState *state;
+  __device__ int position(long long r, int &b) const {
+    b = (int)(r / n);
+    return (state ? state->s - n : p0) + (int)(r - (long long)b * n);
+  }
+};
+
+// (hi + lo)[r, h, c] = scale * log2(e) * sum_e q[r, h, e] W_uk[h, e, c] for LD_ROWS rows of one head; the
+// eight warps take every eighth e. CTAs behind the last head (a layer with latents of its own) put the new
+// rows' latents into the cache meanwhile.
 __global__ void __launch_bounds__(LD_THREADS)
-latent_query_kernel(const bf16 *__restrict__ q, int q_ld, const bf16 *__restrict__ w_uk, int w_ld, int rank, int dim,
-                    float factor, int heads, long long n_rows, float *__restrict__ qa) {
-  __shared__ float part[4][LQ_ROWS][LQ_COLS];
+latent_query_kernel(LdShape g, const bf16 *q, int q_ld, const bf16 *__restrict__ w_uk, int w_ld, float factor,
+                    long long n_rows, bf16 *qh, bf16 *ql, LatentFresh fresh,
+                    bf16 *cache, int cap, int ld) {
+  __shared__ __align__(16) float part[8][LD_ROWS][LQ_COLS];
+  extern __shared__ float qs[];  // [LD_ROWS][dim]
   pdl_launch_dependents();
   pdl_wait();
-  const int h = blockIdx.y;
-  const int cl = threadIdx.x & (LQ_COLS - 1), grp = threadIdx.x / LQ_COLS;
-  const int c = blockIdx.x * LQ_COLS + cl;
-  const long long r0 = (long long)blockIdx.z * LQ_ROWS;
-  const int nr = (int)min((long long)LQ_ROWS, n_rows - r0);
-  float acc[LQ_ROWS] = {};
-  if (c < rank) {
-    const int e0 = dim * grp / 4, e1 = dim * (grp + 1) / 4;
+  const int h = blockIdx.y, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
+  const long long r0 = (long long)blockIdx.z * LD_ROWS;
+  const int nr = (int)min((long long)LD_ROWS, n_rows - r0);
+  if (h == g.heads) {
+    if (blockIdx.x == 0 && wid < nr) {
+      int b;
+      const int p = g.position(r0 + wid, b);
+      store_latent(fresh.dkv + (r0 + wid) * fresh.ld, fresh.gain, fresh.eps, g.rank, ld,
+                   cache + ((long long)(g.slot0 + b) * cap + p) * ld, (bf16 *)nullptr, lane);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < LD_ROWS * g.dim; i += LD_THREADS) {
+    const int r = i / g.dim, e = i - r * g.dim;
+    qs[i] = r < nr ? to_f(q[(r0 + r) * q_ld + (long long)h * g.dim + e]) : 0.f;
+  }
+  const int c = blockIdx.x * LQ_COLS + lane * 8;
+  float acc[LD_ROWS][8] = {};
+  __syncthreads();
+  if (c < g.rank) {  // rows of W_uk end on a multiple of 8 with zeros behind the rank
+    const bf16 *w = w_uk + (long long)h * g.dim * w_ld + c;
 #pragma unroll 8
-    for (int e = e0; e < e1; ++e) {
-      const float w = to_f(w_uk[((long long)h * dim + e) * w_ld + c]);
+    for (int e = wid; e < g.dim; e += 8) {
+      float f[8];
+      unpack8(*reinterpret_cast<const uint4 *>(w + (long long)e * w_ld), f);
 #pragma unroll
-      for (int i = 0; i < LQ_ROWS; ++i)
-        if (i < nr) acc[i] = fmaf(to_f(q[(r0 + i) * q_ld + (long long)h * dim + e]), w, acc[i]);
+      for (int r = 0; r < LD_ROWS; ++r) {
+        const float v = qs[r * g.dim + e];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) acc[r][k] = fmaf(v, f[k], acc[r][k]);
+      }
     }
   }
 #pragma unroll
-  for (int i = 0; i < LQ_ROWS; ++i) part[grp][i][cl] = acc[i];
+  for (int r = 0; r < LD_ROWS; ++r) {
+    *reinterpret_cast<float4 *>(&part[wid][r][lane * 8]) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+    *reinterpret_cast<float4 *>(&part[wid][r][lane * 8 + 4]) = make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]);
+  }
   __syncthreads();
-  // thread group i sums row i
-  if (grp < nr && c < rank)
-    qa[((r0 + grp) * heads + h) * rank + c] =
-        (part[0][grp][cl] + part[1][grp][cl] + part[2][grp][cl] + part[3][grp][cl]) * factor;
+  const int col = blockIdx.x * LQ_COLS + threadIdx.x;
+  if (col >= g.rk) return;
+  for (int r = 0; r < nr; ++r) {
+    float v = 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v += part[k][r][threadIdx.x];
+    const long long at = ((r0 + r) * g.heads16 + h) * g.rk + col;
+    bf16 hi, lo;
+    split2(col < g.rank ? v * factor : 0.f, hi, lo);
+    qh[at] = hi;
+    ql[at] = lo;
+  }
 }
 
-// Chunk blockIdx.x (LD_KEYS keys from the window's first one on) of row blockIdx.z for heads
-// blockIdx.y * 16 ..: partial o[head][rank] = sum_j 2^(s_j - m) c_j with m, l = sum of the weights.
+// Split blockIdx.x (span keys from the window's first one on) of row blockIdx.z for 16 heads: tiles of 64
+// keys, the next one's latents on their way while a tile is used (stages == 2), running maximum and
+// sum per head, o[head][rank] = sum_j 2^(s_j - m) c_j in registers. NT: tiles of 8 latent columns per warp.
+template <int NT>
 __global__ void __launch_bounds__(LD_THREADS)
-latent_chunk_kernel(const float *__restrict__ qa, const bf16 *__restrict__ cache, int cap, int ld, int rank, int heads,
-                    int window, int n, int p0_host, const LoopState *state, int slot0, float *__restrict__ part_o,
-                    float2 *__restrict__ part_ml) {
+latent_chunk_kernel(LdShape g, const bf16 *q_hi, const bf16 *q_lo, const bf16 *cache,
+                    int cap, int ld, int stages, float *part_o, float2 *part_ml) {
   extern __shared__ __align__(16) unsigned char smraw[];
-  const int rk = (rank + 15) & ~15, pitch = rk + 8;  // halves per row: 16-byte rows whose fragments hit distinct banks
-  bf16 *ck = reinterpret_cast<bf16 *>(smraw);        // [LD_KEYS][pitch]
-  bf16 *qh = ck + LD_KEYS * pitch;                   // [16][pitch] high and low terms of the query
+  const int rk = g.rk, pitch = rk + 8;               // 16-byte rows whose fragments hit distinct banks
+  bf16 *qh = reinterpret_cast<bf16 *>(smraw);        // [16][pitch] high and low terms of the query
   bf16 *ql = qh + LD_HEADS * pitch;
-  constexpr int PP = LD_KEYS + 8;
+  constexpr int PP = LD_KEYS + 8, SP = LD_KEYS + 4;
   bf16 *ph = ql + LD_HEADS * pitch;                  // [16][PP] high and low terms of the weights
   bf16 *pl = ph + LD_HEADS * PP;
-  float *sc = reinterpret_cast<float *>(pl + LD_HEADS * PP);  // [16][LD_KEYS + 4]
-  constexpr int SP = LD_KEYS + 4;
+  float *sc = reinterpret_cast<float *>(pl + LD_HEADS * PP);  // [16][SP]
+  float *fac = sc + LD_HEADS * SP;                   // [16] factors of what has been summed so far
+  bf16 *tiles = reinterpret_cast<bf16 *>(fac + LD_HEADS);     // [stages][LD_KEYS][pitch]
   pdl_launch_dependents();
   pdl_wait();
   const long long r = blockIdx.z;
-  const int b = (int)(r / n), t = (int)(r - (long long)b * n);
-  const int p = (state ? state->s - n : p0_host) + t;
-  const int lo = max(0, p - window + 1);
-  const int j0 = lo + blockIdx.x * LD_KEYS;
+  int b;
+  const int p = g.position(r, b);
+  const int j0 = max(0, p - g.window + 1) + blockIdx.x * g.span;
   if (j0 > p) return;
-  const int nk = min(LD_KEYS, p - j0 + 1);
-  const int h0 = blockIdx.y * LD_HEADS, nh = min(LD_HEADS, heads - h0);
+  const int total = min(g.span, p - j0 + 1), nt = (total + LD_KEYS - 1) / LD_KEYS;
+  const int h0 = blockIdx.y * LD_HEADS, nh = min(LD_HEADS, g.heads - h0);
   const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
-  const int g = lane >> 2, tq = lane & 3;
-  const bf16 *src = cache + ((long long)(slot0 + b) * cap + j0) * ld;
-  // latents: 16-byte pieces; the cache's rows end on a multiple of 8 columns with zeros behind the rank
-  for (int i = tid; i < LD_KEYS * (rk / 8); i += LD_THREADS) {
-    const int j = i / (rk / 8), c = (i - j * (rk / 8)) * 8;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (j < nk && c < ld) v = *reinterpret_cast<const uint4 *>(src + (long long)j * ld + c);
-    *reinterpret_cast<uint4 *>(ck + j * pitch + c) = v;
-  }
-  for (int i = tid; i < LD_HEADS * rk; i += LD_THREADS) {
-    const int hh = i / rk, c = i - hh * rk;
-    const float v = hh < nh && c < rank ? qa[(r * heads + h0 + hh) * rank + c] : 0.f;
-    bf16 hi, low;
-    split2(v, hi, low);
-    qh[hh * pitch + c] = hi;
-    ql[hh * pitch + c] = low;
-  }
-  __syncthreads();
-  {  // scores: warp w takes keys 8w .. 8w + 7
-    float d[4] = {0.f, 0.f, 0.f, 0.f};
-    const bf16 *kr = ck + (wid * 8 + g) * pitch + tq * 2;
-    const bf16 *ah = qh + g * pitch + tq * 2, *al = ql + g * pitch + tq * 2;
-    for (int k = 0; k < rk; k += 16) {
-      const unsigned b0 = *reinterpret_cast<const unsigned *>(kr + k), b1 = *reinterpret_cast<const unsigned *>(kr + k + 8);
-      const unsigned a[4] = {*reinterpret_cast<const unsigned *>(ah + k), *reinterpret_cast<const unsigned *>(ah + k + 8 * pitch),
-                             *reinterpret_cast<const unsigned *>(ah + k + 8),
-                             *reinterpret_cast<const unsigned *>(ah + k + 8 * pitch + 8)};
-      const unsigned a2[4] = {*reinterpret_cast<const unsigned *>(al + k), *reinterpret_cast<const unsigned *>(al + k + 8 * pitch),
-                              *reinterpret_cast<const unsigned *>(al + k + 8),
-                              *reinterpret_cast<const unsigned *>(al + k + 8 * pitch + 8)};
-      mma_bf16(d, a2, b0, b1);
-      mma_bf16(d, a, b0, b1);
+  const int gr = lane >> 2, tq = lane & 3;
+  const bf16 *src = cache + ((long long)(g.slot0 + b) * cap + j0) * ld;
+  const int pieces = rk >> 3;
+  auto fetch = [&](int tile) {  // the cache's rows end on a multiple of 8 columns with zeros behind the rank
+    bf16 *dst = tiles + (tile % stages) * LD_KEYS * pitch;
+    const int k0 = tile * LD_KEYS;
+#pragma unroll 4
+    for (int i = tid; i < LD_KEYS * pieces; i += LD_THREADS) {
+      const int j = i / pieces, c = (i - j * pieces) * 8;
+      const bool in = k0 + j < total && c < ld;
+      copy16(dst + j * pitch + c, in ? src + (long long)(k0 + j) * ld + c : src, in ? 16 : 0);
     }
-    const int j = wid * 8 + tq * 2;
-    sc[g * SP + j] = d[0];
-    sc[g * SP + j + 1] = d[1];
-    sc[(g + 8) * SP + j] = d[2];
-    sc[(g + 8) * SP + j + 1] = d[3];
+    copy_commit();
+  };
+  {
+    const long long at = (r * g.heads16 + h0) * rk;
+#pragma unroll 4
+    for (int i = tid; i < LD_HEADS * pieces; i += LD_THREADS) {
+      const int hh = i / pieces, c = (i - hh * pieces) * 8;
+      copy16(qh + hh * pitch + c, q_hi + at + hh * rk + c, 16);
+      copy16(ql + hh * pitch + c, q_lo + at + hh * rk + c, 16);
+    }
   }
-  __syncthreads();
+  fetch(0);
+  float o[NT][4];
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {  // weights: warp w takes heads 2w and 2w + 1, a lane two keys
-    const int hh = wid * 2 + i;
-    const float s0 = lane < nk ? sc[hh * SP + lane] : -INFINITY;
-    const float s1 = lane + 32 < nk ? sc[hh * SP + lane + 32] : -INFINITY;
-    const float m = warp_max(fmaxf(s0, s1));
-    const float p0 = exp2f(s0 - m), p1 = exp2f(s1 - m);
-    const float l = warp_sum(p0 + p1);
-    bf16 hi, low;
-    split2(p0, hi, low);
-    ph[hh * PP + lane] = hi;
-    pl[hh * PP + lane] = low;
-    split2(p1, hi, low);
-    ph[hh * PP + lane + 32] = hi;
-    pl[hh * PP + lane + 32] = low;
-    if (lane == 0 && hh < nh) part_ml[(r * heads + h0 + hh) * gridDim.x + blockIdx.x] = make_float2(m, l);
-  }
-  __syncthreads();
-  unsigned a[LD_KEYS / 16][4], a2[LD_KEYS / 16][4];
+  for (int i = 0; i < NT; ++i)
 #pragma unroll
-  for (int k = 0; k < LD_KEYS / 16; ++k) {
-    const bf16 *x = ph + g * PP + tq * 2 + k * 16, *y = pl + g * PP + tq * 2 + k * 16;
-    a[k][0] = *reinterpret_cast<const unsigned *>(x);
-    a[k][1] = *reinterpret_cast<const unsigned *>(x + 8 * PP);
-    a[k][2] = *reinterpret_cast<const unsigned *>(x + 8);
-    a[k][3] = *reinterpret_cast<const unsigned *>(x + 8 * PP + 8);
-    a2[k][0] = *reinterpret_cast<const unsigned *>(y);
-    a2[k][1] = *reinterpret_cast<const unsigned *>(y + 8 * PP);
-    a2[k][2] = *reinterpret_cast<const unsigned *>(y + 8);
-    a2[k][3] = *reinterpret_cast<const unsigned *>(y + 8 * PP + 8);
-  }
-  for (int c0 = wid * 8; c0 < rk; c0 += LD_THREADS / 32 * 8) {
-    float d[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int k = 0; k < 4; ++k) o[i][k] = 0.f;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};  // of heads 2 * wid and 2 * wid + 1, in every lane
+  for (int tile = 0; tile < nt; ++tile) {
+    if (stages > 1 && tile + 1 < nt) {
+      fetch(tile + 1);
+      copy_wait<1>();
+    } else {
+      copy_wait<0>();
+    }
+    __syncthreads();
+    const bf16 *ck = tiles + (tile % stages) * LD_KEYS * pitch;
+    const int nk = min(LD_KEYS, total - tile * LD_KEYS);
+    {  // scores: warp w takes keys 8w .. 8w + 7; two accumulators keep the products of the terms apart
+      float d[4] = {0.f, 0.f, 0.f, 0.f}, d2[4] = {0.f, 0.f, 0.f, 0.f};
+      const bf16 *kr = ck + (wid * 8 + gr) * pitch + tq * 2;
+      const bf16 *ah = qh + gr * pitch + tq * 2, *al = ql + gr * pitch + tq * 2;
+#pragma unroll 4
+      for (int k = 0; k < rk; k += 16) {
+        const unsigned b0 = *reinterpret_cast<const unsigned *>(kr + k), b1 = *reinterpret_cast<const unsigned *>(kr + k + 8);
+        const unsigned a[4] = {*reinterpret_cast<const unsigned *>(ah + k),
+                               *reinterpret_cast<const unsigned *>(ah + k + 8 * pitch),
+                               *reinterpret_cast<const unsigned *>(ah + k + 8),
+                               *reinterpret_cast<const unsigned *>(ah + k + 8 * pitch + 8)};
+        const unsigned a2[4] = {*reinterpret_cast<const unsigned *>(al + k),
+                                *reinterpret_cast<const unsigned *>(al + k + 8 * pitch),
+                                *reinterpret_cast<const unsigned *>(al + k + 8),
+                                *reinterpret_cast<const unsigned *>(al + k + 8 * pitch + 8)};
+        mma_bf16(d2, a2, b0, b1);
+        mma_bf16(d, a, b0, b1);
+      }
+      const int j = wid * 8 + tq * 2;
+      *reinterpret_cast<float2 *>(sc + gr * SP + j) = make_float2(d[0] + d2[0], d[1] + d2[1]);
+      *reinterpret_cast<float2 *>(sc + (gr + 8) * SP + j) = make_float2(d[2] + d2[2], d[3] + d2[3]);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {  // weights: a lane takes two keys
+      const int hh = wid * 2 + i;
+      const float s0 = lane < nk ? sc[hh * SP + lane] : -INFINITY;
+      const float s1 = lane + 32 < nk ? sc[hh * SP + lane + 32] : -INFINITY;
+      const float mn = fmaxf(m[i], warp_max(fmaxf(s0, s1)));
+      const float p0 = exp2f(s0 - mn), p1 = exp2f(s1 - mn), keep = exp2f(m[i] - mn);
+      l[i] = l[i] * keep + warp_sum(p0 + p1);
+      m[i] = mn;
+      bf16 hi, low;
+      split2(p0, hi, low);
+      ph[hh * PP + lane] = hi;
+      pl[hh * PP + lane] = low;
+      split2(p1, hi, low);
+      ph[hh * PP + lane + 32] = hi;
+      pl[hh * PP + lane + 32] = low;
+      if (lane == 0) fac[hh] = keep;
+    }
+    __syncthreads();
+    unsigned a[LD_KEYS / 16][4], a2[LD_KEYS / 16][4];
 #pragma unroll
     for (int k = 0; k < LD_KEYS / 16; ++k) {
-      unsigned b0, b1;
-      ldmatrix_x2_trans(b0, b1, ck + (k * 16 + (lane & 15)) * pitch + c0);
-      mma_bf16(d, a2[k], b0, b1);
-      mma_bf16(d, a[k], b0, b1);
+      const bf16 *x = ph + gr * PP + tq * 2 + k * 16, *y = pl + gr * PP + tq * 2 + k * 16;
+      a[k][0] = *reinterpret_cast<const unsigned *>(x);
+      a[k][1] = *reinterpret_cast<const unsigned *>(x + 8 * PP);
+      a[k][2] = *reinterpret_cast<const unsigned *>(x + 8);
+      a[k][3] = *reinterpret_cast<const unsigned *>(x + 8 * PP + 8);
+      a2[k][0] = *reinterpret_cast<const unsigned *>(y);
+      a2[k][1] = *reinterpret_cast<const unsigned *>(y + 8 * PP);
+      a2[k][2] = *reinterpret_cast<const unsigned *>(y + 8);
+      a2[k][3] = *reinterpret_cast<const unsigned *>(y + 8 * PP + 8);
     }
-    const int c = c0 + tq * 2;
+    const float f0 = fac[gr], f1 = fac[gr + 8];
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int hh = g + 8 * i;
-      if (hh >= nh) continue;
-      float *o = part_o + ((r * heads + h0 + hh) * gridDim.x + blockIdx.x) * (long long)rank;
-      if (c < rank) o[c] = d[2 * i];
-      if (c + 1 < rank) o[c + 1] = d[2 * i + 1];
+    for (int i = 0; i < NT; ++i) {
+      const int c0 = (i * 8 + wid) * 8;
+      if (c0 < rk) {
+        o[i][0] *= f0;
+        o[i][1] *= f0;
+        o[i][2] *= f1;
+        o[i][3] *= f1;
+#pragma unroll
+        for (int k = 0; k < LD_KEYS / 16; ++k) {
+          unsigned b0, b1;
+          ldmatrix_x2_trans(b0, b1, ck + (k * 16 + (lane & 15)) * pitch + c0);
+          mma_bf16(o[i], a2[k], b0, b1);
+          mma_bf16(o[i], a[k], b0, b1);
+        }
+      }
     }
+    if (stages == 1 && tile + 1 < nt) {
+      __syncthreads();
+      fetch(tile + 1);
+    } else if (stages > 1) {
+      __syncthreads();  // the tile after next goes over this one
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+    if (lane == 0 && wid * 2 + i < nh)
+      part_ml[(r * g.heads + h0 + wid * 2 + i) * g.splits + blockIdx.x] = make_float2(m[i], l[i]);
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    const int c = (i * 8 + wid) * 8 + tq * 2;
+    if (c >= g.rank4) continue;  // columns behind the rank are zeros
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+      if (gr + 8 * k < nh)
+        *reinterpret_cast<float2 *>(part_o + ((r * g.heads + h0 + gr + 8 * k) * g.splits + blockIdx.x) * (long long)g.rank4 +
+                                    c) = make_float2(o[i][2 * k], o[i][2 * k + 1]);
   }
 }
 
-// Joins the chunks of one row and head and maps the weighted latent through W_uv; the CTAs of grid.y
-// share the head's value rows.
+// Joins the splits of LD_ROWS rows of one head and maps the weighted latents through W_uv; the CTAs of
+// grid.y share the head's value rows.
 __global__ void __launch_bounds__(LD_THREADS)
-latent_join_kernel(const float *__restrict__ part_o, const float2 *__restrict__ part_ml, int chunks, const bf16 *__restrict__ w_uv,
-                   int w_ld, int rank, int vdim, int heads, int window, int n, int p0_host, const LoopState *state,
-                   bf16 *__restrict__ out, int out_ld) {
-  extern __shared__ float ol[];  // [rank rounded up to 8] weighted latent, then [chunks] factors
+latent_join_kernel(LdShape g, const float *part_o, const float2 *part_ml, const bf16 *__restrict__ w_uv,
+                   int w_ld, long long n_rows, bf16 *out, int out_ld) {
+  extern __shared__ __align__(16) float ol[];  // [LD_ROWS][rank rounded up to 8] weighted latents, then [LD_ROWS][splits]
   pdl_launch_dependents();
   pdl_wait();
   const int h = blockIdx.x, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
-  const long long r = blockIdx.z;
-  const int t = (int)(r % n);
-  const int p = (state ? state->s - n : p0_host) + t;
-  const int nc = (min(window, p + 1) + LD_KEYS - 1) / LD_KEYS;
-  const int r8 = (rank + 7) & ~7;
-  float *fac = ol + r8;
-  const float2 *ml = part_ml + (r * heads + h) * chunks;
-  float m = -INFINITY, l = 0.f;
-  for (int c = lane; c < nc; c += 32) m = fmaxf(m, ml[c].x);
-  m = warp_max(m);
-  for (int c = lane; c < nc; c += 32) l += ml[c].y * exp2f(ml[c].x - m);
-  l = warp_sum(l);
-  if (wid == 0)
-    for (int c = lane; c < nc; c += 32) fac[c] = exp2f(ml[c].x - m) / l;
-  __syncthreads();
-  const float *o = part_o + (r * heads + h) * (long long)chunks * rank;
-  for (int c = threadIdx.x; c < r8; c += LD_THREADS) {
-    float a = 0.f;
-    if (c < rank) {
-#pragma unroll 4
-      for (int i = 0; i < nc; ++i) a = fmaf(fac[i], o[(long long)i * rank + c], a);
-    }
-    ol[c] = a;
+  const long long r0 = (long long)blockIdx.z * LD_ROWS;
+  const int nr = (int)min((long long)LD_ROWS, n_rows - r0);
+  const int r8 = (g.rank + 7) & ~7;
+  float *fac = ol + LD_ROWS * r8;
+  __shared__ int counts[LD_ROWS];
+  if (wid < nr) {
+    int b;
+    const int p = g.position(r0 + wid, b);
+    const int nc = (min(g.window, p + 1) + g.span - 1) / g.span;
+    const float2 *ml = part_ml + ((r0 + wid) * g.heads + h) * g.splits;
+    float m = -INFINITY, l = 0.f;
+    for (int c = lane; c < nc; c += 32) m = fmaxf(m, ml[c].x);
+    m = warp_max(m);
+    for (int c = lane; c < nc; c += 32) l += ml[c].y * exp2f(ml[c].x - m);
+    l = warp_sum(l);
+    for (int c = lane; c < nc; c += 32) fac[wid * g.splits + c] = exp2f(ml[c].x - m) / l;
+    if (lane == 0) counts[wid] = nc;
   }
   __syncthreads();
-  const int e_per = (vdim + gridDim.y - 1) / gridDim.y;
-  const int e1 = min(vdim, (int)(blockIdx.y + 1) * e_per);
-  for (int e = blockIdx.y * e_per + wid; e < e1; e += LD_THREADS / 32) {
-    const bf16 *wr = w_uv + ((long long)h * vdim + e) * w_ld;
-    float s = 0.f;
-    for (int c = lane * 8; c < r8; c += 256) {  // rows of W_uv end on a multiple of 8 with zeros behind the rank
-      const uint4 v = *reinterpret_cast<const uint4 *>(wr + c);
-      const unsigned u[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        s = fmaf(__uint_as_float(u[i] << 16), ol[c + 2 * i], s);
-        s = fmaf(__uint_as_float(u[i] & 0xffff0000u), ol[c + 2 * i + 1], s);
+  const int cols = r8 >> 2;
+  for (int i = threadIdx.x; i < nr * cols; i += LD_THREADS) {
+    const int r = i / cols, c = (i - r * cols) * 4;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < g.rank4) {
+      const float *o = part_o + ((r0 + r) * g.heads + h) * (long long)g.splits * g.rank4 + c;
+      const float *f = fac + r * g.splits;
+      const int nc = counts[r];
+#pragma unroll 4
+      for (int k = 0; k < nc; ++k) {
+        const float4 v = *reinterpret_cast<const float4 *>(o + (long long)k * g.rank4);
+        a = make_float4(fmaf(f[k], v.x, a.x), fmaf(f[k], v.y, a.y), fmaf(f[k], v.z, a.z), fmaf(f[k], v.w, a.w));
       }
     }
-    s = warp_sum(s);
-    if (lane == 0) out[r * out_ld + (long long)h * vdim + e] = __float2bfloat16_rn(s);
+    *reinterpret_cast<float4 *>(ol + r * r8 + c) = a;
+  }
+  __syncthreads();
+  const int e_per = (g.vdim + gridDim.y - 1) / gridDim.y;
+  const int e1 = min(g.vdim, (int)(blockIdx.y + 1) * e_per);
+#pragma unroll 2
+  for (int e = blockIdx.y * e_per + wid; e < e1; e += LD_THREADS / 32) {
+    const bf16 *wr = w_uv + ((long long)h * g.vdim + e) * w_ld;
+    float s[LD_ROWS] = {};
+    for (int c = lane * 8; c < r8; c += 256) {  // rows of W_uv end on a multiple of 8 with zeros behind the rank
+      float f[8];
+      unpack8(*reinterpret_cast<const uint4 *>(wr + c), f);
+#pragma unroll
+      for (int r = 0; r < LD_ROWS; ++r) {
+        if (r >= nr) break;
+        const float4 x = *reinterpret_cast<const float4 *>(ol + r * r8 + c), y = *reinterpret_cast<const float4 *>(ol + r * r8 + c + 4);
+        s[r] = fmaf(f[0], x.x, fmaf(f[1], x.y, fmaf(f[2], x.z, fmaf(f[3], x.w, s[r]))));
+        s[r] = fmaf(f[4], y.x, fmaf(f[5], y.y, fmaf(f[6], y.z, fmaf(f[7], y.w, s[r]))));
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < LD_ROWS; ++r) {
+      if (r >= nr) break;
+      const float v = warp_sum(s[r]);
+      if (lane == 0) out[(r0 + r) * out_ld + (long long)h * g.vdim + e] = __float2bfloat16_rn(v);
+    }
   }
 }
 
-size_t chunk_smem(int rank) {
+size_t chunk_smem(int rank, int stages) {
   const int pitch = ((rank + 15) & ~15) + 8;
-  return (size_t)(LD_KEYS + 2 * LD_HEADS) * pitch * 2 + (size_t)2 * LD_HEADS * (LD_KEYS + 8) * 2 +
-         (size_t)LD_HEADS * (LD_KEYS + 4) * 4;
+  return (size_t)(stages * LD_KEYS + 2 * LD_HEADS) * pitch * 2 + (size_t)2 * LD_HEADS * (LD_KEYS + 8) * 2 +
+         (size_t)LD_HEADS * (LD_KEYS + 4) * 4 + LD_HEADS * 4;
 }
-int chunks_of(int window, int s_cap) { return ((window < s_cap ? window : s_cap) + LD_KEYS - 1) / LD_KEYS; }
+constexpr size_t LD_SMEM_LIMIT = 220 * 1024;
+
+// How a window of `window` keys (contexts up to s_cap) is cut for so many rows: about two CTAs per SM.
+int most_splits(int heads, int window, int s_cap, long long rows) {
+  const int tiles = ((window < s_cap ? window : s_cap) + LD_KEYS - 1) / LD_KEYS;
+  const long long groups = rows * ((heads + LD_HEADS - 1) / LD_HEADS);
+  const long long want = (2 * 148 + groups - 1) / groups;
+  return (int)(want < tiles ? want : tiles);
+}
+void plan_splits(int heads, int window, int s_cap, long long rows, int *splits, int *span) {
+  const int tiles = ((window < s_cap ? window : s_cap) + LD_KEYS - 1) / LD_KEYS;
+  const int want = most_splits(heads, window, s_cap, rows), per = (tiles + want - 1) / want;
+  *span = per * LD_KEYS;
+  *splits = (tiles + per - 1) / per;
+}
+
+struct LdScratch {
+  size_t q, ml, o;  // floats: both query terms, maxima and sums, partial results
+};
+LdScratch ld_scratch(int heads, int rank, int splits, long long rows) {
+  const size_t heads16 = (size_t)(heads + 15) / 16 * 16, rk = (size_t)(rank + 15) / 16 * 16;
+  const size_t rh = (size_t)rows * heads;
+  return {(size_t)rows * heads16 * rk, (rh * splits * 2 + 3) / 4 * 4, rh * splits * ((size_t)(rank + 3) / 4 * 4)};
+}
 
 }  // namespace
 
@@ -416,36 +596,70 @@ void launch_latent_attention_rows(const LatentAttention &a, Precision type, cons
   else go(latent_attention_rows_kernel<float>, (float *)nullptr);
 }
 
-bool latent_decode_supports(const LatentAttention &a) { return chunk_smem(a.cache.rank) <= 220 * 1024; }
-
-size_t latent_decode_scratch_floats(int heads, int rank, int window, int s_cap, long long rows) {
-  const size_t rh = (size_t)rows * heads, c = (size_t)chunks_of(window, s_cap);
-  return (rh * rank + 3) / 4 * 4 + rh * c * 2 + rh * c * rank;
+bool latent_decode_supports(const LatentAttention &a) {
+  return a.cache.rank <= 1024 && chunk_smem(a.cache.rank, 1) <= LD_SMEM_LIMIT && a.dim <= 2048;
 }
 
-int launch_latent_decode(const LatentAttention &a, float *scratch, const RowBatch &b, cudaStream_t st) {
+size_t latent_decode_scratch_floats(int heads, int rank, int window, int s_cap, long long rows) {
+  // fewer rows are cut into more splits, shorter contexts into no more than most_splits of the longest one
+  size_t need = 0;
+  for (long long r = 1; r <= rows; ++r) {
+    const LdScratch n = ld_scratch(heads, rank, most_splits(heads, window, s_cap, r), r);
+    need = n.q + n.ml + n.o > need ? n.q + n.ml + n.o : need;
+  }
+  return need;
+}
+
+int launch_latent_decode(const LatentAttention &a, const LatentFresh &fresh, float *scratch, const RowBatch &b,
+                         cudaStream_t st) {
   const long long rows = b.rows();
-  const int rank = a.cache.rank, chunks = chunks_of(a.window, b.s_cap);
-  float *qa = scratch;
-  float2 *ml = reinterpret_cast<float2 *>(scratch + ((size_t)rows * a.heads * rank + 3) / 4 * 4);
-  float *po = reinterpret_cast<float *>(ml + (size_t)rows * a.heads * chunks);
+  LdShape g{};
+  g.heads = a.heads;
+  g.heads16 = (a.heads + 15) / 16 * 16;
+  g.dim = a.dim;
+  g.vdim = a.vdim;
+  g.rank = a.cache.rank;
+  g.rk = (g.rank + 15) / 16 * 16;
+  g.rank4 = (g.rank + 3) / 4 * 4;
+  g.window = a.window;
+  g.n = b.n;
+  g.p0 = b.p0;
+  g.slot0 = b.slot0;
+  g.state = b.state;
+  plan_splits(a.heads, a.window, b.s_cap, rows, &g.splits, &g.span);
+  const LdScratch n = ld_scratch(a.heads, g.rank, g.splits, rows);
+  bf16 *qh = reinterpret_cast<bf16 *>(scratch), *ql = qh + n.q;
+  float2 *ml = reinterpret_cast<float2 *>(scratch + n.q);
+  float *po = scratch + n.q + n.ml;
+  const bf16 *cache = static_cast<const bf16 *>(a.cache.rows);
+  const unsigned row_groups = (unsigned)((rows + LD_ROWS - 1) / LD_ROWS);
+  const size_t q_smem = (size_t)LD_ROWS * a.dim * sizeof(float);
+  if (q_smem + 8 * LD_ROWS * LQ_COLS * 4 > 48 * 1024)
+    LB_CUDA(cudaFuncSetAttribute(latent_query_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)q_smem));
   launch_pdl(latent_query_kernel,
-             dim3((unsigned)((rank + LQ_COLS - 1) / LQ_COLS), (unsigned)a.heads, (unsigned)((rows + LQ_ROWS - 1) / LQ_ROWS)),
-             dim3(LD_THREADS), 0, st, g_pdl_enabled, static_cast<const bf16 *>(a.q), a.q_ld, static_cast<const bf16 *>(a.w_uk),
-             a.w_ld, rank, a.dim, a.scale * LOG2E, a.heads, rows, qa);
-  const size_t smem = chunk_smem(rank);
-  if (smem > 48 * 1024)
-    LB_CUDA(cudaFuncSetAttribute(latent_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  launch_pdl(latent_chunk_kernel,
-             dim3((unsigned)chunks, (unsigned)((a.heads + LD_HEADS - 1) / LD_HEADS), (unsigned)rows), dim3(LD_THREADS), smem,
-             st, g_pdl_enabled, (const float *)qa, static_cast<const bf16 *>(a.cache.rows), a.cache.cap, a.cache.ld, rank,
-             a.heads, a.window, b.n, b.p0, b.state, b.slot0, po, ml);
-  int parts = (int)(148 / (rows * a.heads > 148 ? 148 : rows * a.heads));
+             dim3((unsigned)((g.rk + LQ_COLS - 1) / LQ_COLS), (unsigned)(a.heads + (fresh.dkv ? 1 : 0)), row_groups),
+             dim3(LD_THREADS), q_smem, st, g_pdl_enabled, g, static_cast<const bf16 *>(a.q), a.q_ld,
+             static_cast<const bf16 *>(a.w_uk), a.w_ld, a.scale * LOG2E, rows, qh, ql, fresh,
+             static_cast<bf16 *>(a.cache.rows), a.cache.cap, a.cache.ld);
+  const int stages = g.span > LD_KEYS && chunk_smem(g.rank, 2) <= LD_SMEM_LIMIT ? 2 : 1;
+  const size_t smem = chunk_smem(g.rank, stages);
+  auto chunk = [&](auto kernel) {
+    if (smem > 48 * 1024) LB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    launch_pdl(kernel, dim3((unsigned)g.splits, (unsigned)(g.heads16 / LD_HEADS), (unsigned)rows), dim3(LD_THREADS), smem, st,
+               g_pdl_enabled, g, (const bf16 *)qh, (const bf16 *)ql, cache, a.cache.cap, a.cache.ld, stages, po, ml);
+  };
+  if (g.rk <= 128) chunk(latent_chunk_kernel<2>);
+  else if (g.rk <= 256) chunk(latent_chunk_kernel<4>);
+  else if (g.rk <= 512) chunk(latent_chunk_kernel<8>);
+  else chunk(latent_chunk_kernel<16>);
+  int parts = (int)(2 * 148 / ((long long)row_groups * a.heads > 2 * 148 ? 2 * 148 : (long long)row_groups * a.heads));
   const int most = (a.vdim + 7) / 8;
   parts = parts < 1 ? 1 : parts > most ? most : parts > 8 ? 8 : parts;
-  launch_pdl(latent_join_kernel, dim3((unsigned)a.heads, (unsigned)parts, (unsigned)rows), dim3(LD_THREADS),
-             ((size_t)((rank + 7) & ~7) + chunks) * sizeof(float), st, g_pdl_enabled, (const float *)po, (const float2 *)ml,
-             chunks, static_cast<const bf16 *>(a.w_uv), a.w_ld, rank, a.vdim, a.heads, a.window, b.n, b.p0, b.state,
+  const size_t j_smem = (size_t)LD_ROWS * (((g.rank + 7) & ~7) + g.splits) * sizeof(float);
+  if (j_smem > 48 * 1024)
+    LB_CUDA(cudaFuncSetAttribute(latent_join_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)j_smem));
+  launch_pdl(latent_join_kernel, dim3((unsigned)a.heads, (unsigned)parts, row_groups), dim3(LD_THREADS), j_smem, st,
+             g_pdl_enabled, g, (const float *)po, (const float2 *)ml, static_cast<const bf16 *>(a.w_uv), a.w_ld, rows,
              static_cast<bf16 *>(a.out), a.out_ld);
   return 3;
 }

@@ -10,8 +10,8 @@
 // with a shorter one fills), and the last taps - 1 rows h of every layer.
 //
 // A step's launches per layer, bfloat16:
-//   few rows    norm + convolutions | W_q, W_dkv and W_up (GELU) in one launch | latent store |
-//               query, chunks, join | W_o and W_down as one product over [attention | hidden], added to x
+//   few rows    norm + convolutions | W_q, W_dkv and W_up (GELU) in one launch | query and latent store,
+//               chunks, join | W_o and W_down as one product over [attention | hidden], added to x
 //   many rows   the same with the tensor-core products, and keys and values expanded from the window's
 //               latents for the tensor-core attention (V directly transposed, as W_uv c^T)
 // 32-bit runs the framework's float products and the CUDA-core attention.
@@ -428,13 +428,14 @@ class Mitilix final : public DecoderModel {
       launch_latent_prefill(at, k_.p, up8(l.q_cols()), vt_.p, up8((int)keys), key_rows, first, b, st, err);
       launches_ += 3;
     } else {
-      if (l.own()) {
-        launch_latent_store(dkv_.f(), l.rank, l.latent_gain.f(), eps_, at.cache, nullptr, 0, 0, prec_, b, st);
-        ++launches_;
-      }
       if (m <= decode_rows_ && latent_decode_supports(at)) {
-        launches_ += launch_latent_decode(at, scratch_.f(), b, st);
+        const LatentFresh fresh{l.own() ? dkv_.f() : nullptr, l.rank, l.latent_gain.f(), eps_};
+        launches_ += launch_latent_decode(at, fresh, scratch_.f(), b, st);
       } else {
+        if (l.own()) {
+          launch_latent_store(dkv_.f(), l.rank, l.latent_gain.f(), eps_, at.cache, nullptr, 0, 0, prec_, b, st);
+          ++launches_;
+        }
         launch_latent_attention_rows(at, prec_, b, st);
         ++launches_;
       }

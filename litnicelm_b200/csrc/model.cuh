@@ -91,6 +91,8 @@ const char *registered_architectures();  // names with commas between them
 std::string read_text_file(const std::string &path);
 
 // ---- kernels of these designs ------------------------------------------------
+// Inside these kernels only weights are __restrict__ const: such loads count as invariant and may be
+// scheduled ahead of the wait for the preceding kernel (pdl_wait), which wrote every other input.
 
 // embed.cu: x[r, :] = table[ids] + pos[p] for the rows of a batch; tables bfloat16 or float.
 void launch_embed_rows(const void *table, const void *pos, Precision type, const RowBatch &b, int d, int vocab, float *x,
@@ -139,10 +141,19 @@ struct LatentAttention {
 // Any size, 32-bit arithmetic on CUDA cores, one CTA per row and head.
 void launch_latent_attention_rows(const LatentAttention &a, Precision type, const RowBatch &b, cudaStream_t st);
 // Few new rows (decoding and short portions) on bfloat16: W_uk absorbed into the query, key chunks
-// shared by 16 heads, partial results joined and mapped through W_uv. Returns the kernels launched.
+// shared by 16 heads, partial results joined and mapped through W_uv. fresh: the rows' W_dkv h, stored
+// into the cache on the way (dkv == nullptr: the layer reads latents another layer has stored). Returns
+// the kernels launched.
+struct LatentFresh {
+  const float *dkv = nullptr;  // [rows, ld]
+  int ld = 0;
+  const float *gain = nullptr;
+  float eps = 0.f;
+};
 bool latent_decode_supports(const LatentAttention &a);
 size_t latent_decode_scratch_floats(int heads, int rank, int window, int s_cap, long long rows);
-int launch_latent_decode(const LatentAttention &a, float *scratch, const RowBatch &b, cudaStream_t st);
+int launch_latent_decode(const LatentAttention &a, const LatentFresh &fresh, float *scratch, const RowBatch &b,
+                         cudaStream_t st);
 
 // latent_attention_tc.cu: many new rows on bfloat16 tensor cores over expanded keys and values:
 // k [streams * key_rows, k_ld] row-major, vt [heads * vdim, vt_ld] with one column per key; key row j

@@ -339,6 +339,69 @@ int pow2_at_least(int v) {
   return p;
 }
 
+// Greedy selection over a large vocabulary: `parts` CTAs per stream look for the first maximum of their
+// share, the best of a stream meets in best[stream] (larger logit first, then smaller id, as composite()
+// orders them), and the CTA that finishes last appends every stream's token and advances the loop state.
+// best and done rest at all ones and zero between launches.
+constexpr int GS_THREADS = 256;
+constexpr int GS_UNROLL = 4;
+
+__global__ void __launch_bounds__(GS_THREADS)
+greedy_select_kernel(const float *__restrict__ logits, int vocab, int n_streams, unsigned long long *best, unsigned *done,
+                     int *ids, int ids_ld, int *out_tokens, int out_ld, LoopState *state) {
+  __shared__ unsigned long long part[GS_THREADS / 32];
+  __shared__ int last;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.y, per = (vocab + gridDim.x - 1) / gridDim.x;
+  const int i0 = blockIdx.x * per, i1 = min(vocab, i0 + per);
+  const float *row = logits + (long long)b * vocab;
+  unsigned long long m = ~0ull;
+  for (int i = i0 + threadIdx.x; i < i1; i += GS_THREADS * GS_UNROLL) {
+    float v[GS_UNROLL];
+#pragma unroll
+    for (int u = 0; u < GS_UNROLL; ++u) v[u] = i + u * GS_THREADS < i1 ? row[i + u * GS_THREADS] : 0.f;
+#pragma unroll
+    for (int u = 0; u < GS_UNROLL; ++u) {
+      // entries the scan of block_argmax_first cannot pick (NaN, below its sentinel) stay out here too;
+      // zeros of either sign are equal there
+      if (i + u * GS_THREADS >= i1 || !(v[u] >= -3.402823466e+38f)) continue;
+      const unsigned long long c = composite(v[u] == 0.f ? 0.f : v[u], i + u * GS_THREADS);
+      m = c < m ? c : m;
+    }
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const unsigned long long t = __shfl_xor_sync(0xffffffffu, m, o);
+    m = t < m ? t : m;
+  }
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = m;
+  __syncthreads();
+  if (threadIdx.x == 0) {
+#pragma unroll
+    for (int w = 1; w < GS_THREADS / 32; ++w) m = part[w] < m ? part[w] : m;
+    atomicMin(best + b, m);
+    __threadfence();
+    last = atomicAdd(done, 1u) == gridDim.x * gridDim.y - 1;
+  }
+  __syncthreads();
+  if (!last) return;
+  __threadfence();
+  const int s = state->s, step = state->step, max_seq = state->max_seq;
+  for (int i = threadIdx.x; i < n_streams; i += GS_THREADS) {
+    const unsigned long long c = atomicExch(best + i, ~0ull);
+    const int token = c == ~0ull ? 0 : (int)(unsigned)c;
+    out_tokens[(long long)i * out_ld + step] = token;
+    if (s < max_seq) ids[(long long)i * ids_ld + s] = token;
+  }
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    state->s = s + 1;
+    state->step = step + 1;
+    *done = 0;
+  }
+}
+
 }  // namespace
 
 // Bytes of global scratch per row for the path that sorts the whole vocabulary
@@ -365,6 +428,17 @@ static void run_sampler(const float *logits, int vocab, int n_rows, const Sample
   }
   launch_pdl(sampler_kernel, dim3(n_rows), dim3(SM_THREADS), 0, st, g_pdl_enabled, logits, vocab, sp, mt_state, draws, ids,
              ids_ld, out, out_ld, state, sk, sw, p2);
+}
+
+bool greedy_select_supports(int vocab) { return vocab >= 2048; }
+
+void launch_greedy_select(const float *logits, int vocab, int n_streams, unsigned long long *best, unsigned *done, int *ids,
+                          int ids_ld, int *out_tokens, int out_ld, LoopState *state, cudaStream_t st) {
+  int parts = (vocab + GS_THREADS * GS_UNROLL - 1) / (GS_THREADS * GS_UNROLL);
+  const int most = (2 * 148 + n_streams - 1) / n_streams;
+  if (parts > most) parts = most;
+  launch_pdl(greedy_select_kernel, dim3((unsigned)parts, (unsigned)n_streams), dim3(GS_THREADS), 0, st, g_pdl_enabled, logits,
+             vocab, n_streams, best, done, ids, ids_ld, out_tokens, out_ld, state);
 }
 
 void launch_sampler(const float *logits, int vocab, int n_streams, const SamplerParams &sp,

@@ -232,6 +232,8 @@ struct litnice_b200_session {
   std::vector<int> slot_len;      // positions each slot holds (litnice_b200_extend)
   int *rows_list = nullptr;       // device: rows of a portion whose logits are asked for
   long long rows_list_cap = 0;
+  unsigned long long *select_best = nullptr;  // greedy selection over a large vocabulary: all ones at rest
+  unsigned *select_done = nullptr;
 
   bool keep_logits = false;
   float *step_logits = nullptr;
@@ -1111,6 +1113,11 @@ int litnice_b200_session_create_model(const char *model_dir, int32_t dtype, int3
   *out = s;  // handed out even on failure below so the caller can read the error text
   const int rc = guarded(s, [&]() {
     session_common(s);
+    if (cudaMalloc(reinterpret_cast<void **>(&s->select_best), (size_t)max_streams * 8) != cudaSuccess ||
+        cudaMalloc(reinterpret_cast<void **>(&s->select_done), 16) != cudaSuccess)
+      throw std::bad_alloc();
+    LB_CUDA(cudaMemsetAsync(s->select_best, 0xff, (size_t)max_streams * 8, s->st));
+    LB_CUDA(cudaMemsetAsync(s->select_done, 0, 16, s->st));
     if (!tc_runtime_available()) throw std::runtime_error("cuTensorMapEncodeTiled is not available");
     session_loop_buffers(s, (size_t)(max_streams < 8 ? 8 : max_streams));
     try {
@@ -1337,6 +1344,8 @@ void litnice_b200_session_destroy(litnice_b200_session *s) {
   if (s->st) cudaStreamSynchronize(s->st);
   s->model.reset();
   if (s->rows_list) cudaFree(s->rows_list);
+  if (s->select_best) cudaFree(s->select_best);
+  if (s->select_done) cudaFree(s->select_done);
   free_activations(s);
   for (void *p : {(void *)s->params, (void *)s->xl, (void *)s->logits, (void *)s->probs, (void *)s->gemv_scratch,
                   (void *)s->logits_all, (void *)s->ids, (void *)s->out_tokens, (void *)s->mt, (void *)s->state,
@@ -1618,6 +1627,12 @@ int litnice_b200_run(litnice_b200_session *s, int32_t max_new, const litnice_b20
       if (s->keep_logits) {
         LB_CUDA(cudaMemcpyAsync(s->step_logits + (long long)(s->cur_tokens + step) * B * V, s->logits,
                                 (size_t)B * V * 4, cudaMemcpyDeviceToDevice, s->st));
+      }
+      if (s->model && greedy && greedy_select_supports(V)) {
+        launch_greedy_select(s->logits, V, B, s->select_best, s->select_done, s->ids, s->dims.max_seq_len, s->out_tokens,
+                             s->out_cap, s->state, s->st);
+        ++s->launches;
+        return;
       }
       launch_sampler(s->logits, V, B, sp, s->mt, s->ids, s->dims.max_seq_len, s->out_tokens, s->out_cap,
                      s->state, s->sampler_scratch, s->st);

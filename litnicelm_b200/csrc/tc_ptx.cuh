@@ -203,6 +203,11 @@ __device__ __forceinline__ void st_cluster_f4(unsigned cluster_addr, float4 v) {
                : "memory");
 }
 
+__device__ __forceinline__ float ld_cluster_f32(unsigned cluster_addr) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(cluster_addr) : "memory");
+  return v;
+}
 __device__ __forceinline__ float4 ld_cluster_f4(unsigned cluster_addr) {
   float4 v;
   asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];"

@@ -39,7 +39,7 @@ __global__ void expand_f32_kernel(const unsigned short *__restrict__ src, long l
   }
 }
 
-__global__ void gelu_f32_kernel(float *__restrict__ x, long long count) {
+__global__ void gelu_f32_kernel(float *x, long long count) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < count; i += (long long)gridDim.x * blockDim.x) {
