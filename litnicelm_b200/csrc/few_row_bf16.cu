@@ -80,21 +80,43 @@ few_row_bf16_kernel(FewRowPair pair, int m, int ranks) {
   load_w(k_begin + wid * SPAN);  // the weights do not depend on the predecessor
   pdl_wait();
   for (int k0 = k_begin + wid * SPAN; k0 < k_end; k0 += FR_WARPS * SPAN) {
+    if constexpr (NT >= 8) {  // one tile's activations of all blocks at a time: fewer registers
 #pragma unroll
-    for (int i = 0; i < NT; ++i) {
-      const int row = i * 8 + g;
-      const bf16 *ar = a + (long long)row * p.a_ld + t * 8;
-      uint4 x[UNROLL];
+      for (int i = 0; i < NT; ++i) {
+        const int row = i * 8 + g;
+        const bf16 *ar = a + (long long)row * p.a_ld + t * 8;
+        uint4 x[UNROLL];
+#pragma unroll
+        for (int u = 0; u < UNROLL; ++u) {
+          const int k = k0 + u * 32;
+          x[u] = row < m && k + t * 8 < k_end ? *reinterpret_cast<const uint4 *>(ar + k) : zero;
+        }
+#pragma unroll
+        for (int u = 0; u < UNROLL; ++u) {
+          fr_mma(acc[i], wa[u].x, wb[u].x, wa[u].y, wb[u].y, x[u].x, x[u].y);
+          fr_mma(acc[i], wa[u].z, wb[u].z, wa[u].w, wb[u].w, x[u].z, x[u].w);
+        }
+      }
+    } else {
+      // all tiles' activations of a block of 32 k are requested together, one block ahead of their use
+      uint4 x[2][NT];
+      auto load_x = [&](int u, uint4 (&dst)[NT]) {
+        const int k = k0 + u * 32 + t * 8;
+#pragma unroll
+        for (int i = 0; i < NT; ++i)
+          dst[i] = i * 8 + g < m && k < k_end ? *reinterpret_cast<const uint4 *>(a + (long long)(i * 8 + g) * p.a_ld + k) : zero;
+      };
+      load_x(0, x[0]);
 #pragma unroll
       for (int u = 0; u < UNROLL; ++u) {
-        const int k = k0 + u * 32;
-        x[u] = row < m && k + t * 8 < k_end ? *reinterpret_cast<const uint4 *>(ar + k) : zero;
-      }
+        if (u + 1 < UNROLL) load_x(u + 1, x[(u + 1) & 1]);
 #pragma unroll
-      for (int u = 0; u < UNROLL; ++u) {
-        fr_mma(acc[i], wa[u].x, wb[u].x, wa[u].y, wb[u].y, x[u].x, x[u].y);
-        fr_mma(acc[i], wa[u].z, wb[u].z, wa[u].w, wb[u].w, x[u].z, x[u].w);
-      }
+        for (int i = 0; i < NT; ++i) {
+          const uint4 v = x[u & 1][i];
+          fr_mma(acc[i], wa[u].x, wb[u].x, wa[u].y, wb[u].y, v.x, v.y);
+          fr_mma(acc[i], wa[u].z, wb[u].z, wa[u].w, wb[u].w, v.z, v.w);
+        }
+    }
     }
     if (k0 + FR_WARPS * SPAN < k_end) load_w(k0 + FR_WARPS * SPAN);
   }
@@ -159,7 +181,8 @@ void launch_few_row_bf16(const Bf16Product *p, int count, int m, cudaStream_t st
   for (int i = 0; i < count; ++i) k_max = p[i].k > k_max ? p[i].k : k_max;
   // ranks of a cluster that share a tile's k: enough CTAs for two per SM, at least 512 k each
   int ranks = 1;
-  while (ranks < 8 && blocks * ranks < 2 * 148 && k_max >= 1024 * ranks) ranks *= 2;
+  const int ranks_max = m > 16 ? 4 : 8;  // many rows: a CTA's share of the sums is work too
+  while (ranks < ranks_max && blocks * ranks < 2 * 148 && k_max >= 1024 * ranks) ranks *= 2;
   const dim3 grid(blocks, 1, (unsigned)ranks), block(FR_WARPS * 32);
   auto go = [&](auto kernel) {
     launch_pdl_cluster(kernel, grid, block, 0, st, g_pdl_enabled, (unsigned)ranks, pair, m, ranks);
@@ -169,7 +192,7 @@ void launch_few_row_bf16(const Bf16Product *p, int count, int m, cudaStream_t st
     if (nt <= 1) go(few_row_bf16_kernel<1, 2>);
     else if (nt <= 2) go(few_row_bf16_kernel<2, 2>);
     else if (nt <= 4) go(few_row_bf16_kernel<4, 2>);
-    else go(few_row_bf16_kernel<8, 2>);
+    else go(few_row_bf16_kernel<8, 4>);
     return;
   }
   if (nt <= 1) go(few_row_bf16_kernel<1, 4>);

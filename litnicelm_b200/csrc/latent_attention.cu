@@ -13,9 +13,11 @@
 //   latent_query / latent_chunk / latent_join   few rows on bfloat16: the absorbed query per head (and the
 //                                new latents into the cache, by CTAs of their own); splits of the window
 //                                for 16 heads at a time on mma.sync tiles, the 32-bit query and weights
-//                                entering as two bfloat16 terms each; the join of the splits and W_uv
+//                                entering as two bfloat16 terms each; the join of the splits and W_uv,
+//                                inside the same launch where the splits fit a thread-block cluster
 // Scores, weights and norms are 32-bit throughout.
 #include "model.cuh"
+#include "tc_ptx.cuh"
 
 #include <cuda_bf16.h>
 
@@ -90,7 +92,7 @@ __device__ __forceinline__ void store_latent(const float *src, const float *__re
 // copied from the cache to the packed rows, new ones normalised (dkv given) or, for a layer that uses
 // another layer's latents, copied as well.
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 latent_store_kernel(const float *dkv, int dkv_ld, const float *__restrict__ gain, float eps, T *cache,
                     int cap, int ld, int rank, T *packed, int packed_rows, int first, int n, int p0_host,
                     const LoopState *state, int slot0) {
@@ -190,6 +192,7 @@ constexpr int LD_HEADS = 16;     // heads per CTA: the rows of an mma tile
 constexpr int LD_THREADS = 256;
 constexpr int LQ_COLS = 256;     // latent columns per CTA of the query kernel, eight per thread
 constexpr int LD_ROWS = 4;       // rows per CTA of the query and join kernels
+constexpr int LD_CLUSTER = 8;    // CTAs of the largest cluster
 constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
@@ -237,20 +240,30 @@ struct LdShape {
   }
 };
 
-// (hi + lo)[r, h, c] = scale * log2(e) * sum_e q[r, h, e] W_uk[h, e, c] for LD_ROWS rows of one head; the
+// (hi + lo)[r, h, c] = scale * log2(e) * sum_e q[r, h, e] W_uk[h, e, c] for ROWS rows of one head; the
 // eight warps take every eighth e. CTAs behind the last head (a layer with latents of its own) put the new
 // rows' latents into the cache meanwhile.
+template <int ROWS>
 __global__ void __launch_bounds__(LD_THREADS)
 latent_query_kernel(LdShape g, const bf16 *q, int q_ld, const bf16 *__restrict__ w_uk, int w_ld, float factor,
                     long long n_rows, bf16 *qh, bf16 *ql, LatentFresh fresh,
                     bf16 *cache, int cap, int ld) {
-  __shared__ __align__(16) float part[8][LD_ROWS][LQ_COLS];
-  extern __shared__ float qs[];  // [LD_ROWS][dim]
+  __shared__ __align__(16) float part[8][ROWS][LQ_COLS];
+  extern __shared__ float qs[];  // [ROWS][dim]
   pdl_launch_dependents();
-  pdl_wait();
   const int h = blockIdx.y, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
-  const long long r0 = (long long)blockIdx.z * LD_ROWS;
-  const int nr = (int)min((long long)LD_ROWS, n_rows - r0);
+  const int c = blockIdx.x * LQ_COLS + lane * 8;
+  constexpr int PRE = 4;  // rows of W_uk per warp that are requested ahead of the wait
+  uint4 pre[PRE];
+  const bf16 *w = w_uk + (long long)h * g.dim * w_ld + c;  // rows end on a multiple of 8 with zeros behind the rank
+#pragma unroll
+  for (int i = 0; i < PRE; ++i)
+    pre[i] = h < g.heads && c < g.rank && wid + 8 * i < g.dim
+                 ? *reinterpret_cast<const uint4 *>(w + (long long)(wid + 8 * i) * w_ld)
+                 : make_uint4(0, 0, 0, 0);
+  pdl_wait();
+  const long long r0 = (long long)blockIdx.z * ROWS;
+  const int nr = (int)min((long long)ROWS, n_rows - r0);
   if (h == g.heads) {
     if (blockIdx.x == 0 && wid < nr) {
       int b;
@@ -260,29 +273,31 @@ latent_query_kernel(LdShape g, const bf16 *q, int q_ld, const bf16 *__restrict__
     }
     return;
   }
-  for (int i = threadIdx.x; i < LD_ROWS * g.dim; i += LD_THREADS) {
+  for (int i = threadIdx.x; i < ROWS * g.dim; i += LD_THREADS) {
     const int r = i / g.dim, e = i - r * g.dim;
     qs[i] = r < nr ? to_f(q[(r0 + r) * q_ld + (long long)h * g.dim + e]) : 0.f;
   }
-  const int c = blockIdx.x * LQ_COLS + lane * 8;
-  float acc[LD_ROWS][8] = {};
+  float acc[ROWS][8] = {};
   __syncthreads();
-  if (c < g.rank) {  // rows of W_uk end on a multiple of 8 with zeros behind the rank
-    const bf16 *w = w_uk + (long long)h * g.dim * w_ld + c;
-#pragma unroll 8
-    for (int e = wid; e < g.dim; e += 8) {
-      float f[8];
-      unpack8(*reinterpret_cast<const uint4 *>(w + (long long)e * w_ld), f);
+  auto add = [&](int e, uint4 row) {
+    float f[8];
+    unpack8(row, f);
 #pragma unroll
-      for (int r = 0; r < LD_ROWS; ++r) {
-        const float v = qs[r * g.dim + e];
+    for (int r = 0; r < ROWS; ++r) {
+      const float v = qs[r * g.dim + e];
 #pragma unroll
-        for (int k = 0; k < 8; ++k) acc[r][k] = fmaf(v, f[k], acc[r][k]);
-      }
+      for (int k = 0; k < 8; ++k) acc[r][k] = fmaf(v, f[k], acc[r][k]);
     }
+  };
+  if (c < g.rank) {
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+      if (wid + 8 * i < g.dim) add(wid + 8 * i, pre[i]);
+#pragma unroll 4
+    for (int e = wid + 8 * PRE; e < g.dim; e += 8) add(e, *reinterpret_cast<const uint4 *>(w + (long long)e * w_ld));
   }
 #pragma unroll
-  for (int r = 0; r < LD_ROWS; ++r) {
+  for (int r = 0; r < ROWS; ++r) {
     *reinterpret_cast<float4 *>(&part[wid][r][lane * 8]) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
     *reinterpret_cast<float4 *>(&part[wid][r][lane * 8 + 4]) = make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]);
   }
@@ -304,10 +319,14 @@ latent_query_kernel(LdShape g, const bf16 *q, int q_ld, const bf16 *__restrict__
 // Split blockIdx.x (span keys from the window's first one on) of row blockIdx.z for 16 heads: tiles of 64
 // keys, the next one's latents on their way while a tile is used (stages == 2), running maximum and
 // sum per head, o[head][rank] = sum_j 2^(s_j - m) c_j in registers. NT: tiles of 8 latent columns per warp.
-template <int NT>
+// CLUSTER: the splits of a row and head group are the CTAs of a thread-block cluster; their results meet in
+// shared memory, each CTA joins its share of the heads and maps it through W_uv (latent_join_kernel does
+// both where the splits are too many for a cluster).
+template <int NT, bool CLUSTER>
 __global__ void __launch_bounds__(LD_THREADS)
 latent_chunk_kernel(LdShape g, const bf16 *q_hi, const bf16 *q_lo, const bf16 *cache,
-                    int cap, int ld, int stages, float *part_o, float2 *part_ml) {
+                    int cap, int ld, int stages, float *part_o, float2 *part_ml, const bf16 *__restrict__ w_uv, int w_ld,
+                    bf16 *out, int out_ld) {
   extern __shared__ __align__(16) unsigned char smraw[];
   const int rk = g.rk, pitch = rk + 8;               // 16-byte rows whose fragments hit distinct banks
   bf16 *qh = reinterpret_cast<bf16 *>(smraw);        // [16][pitch] high and low terms of the query
@@ -324,8 +343,8 @@ latent_chunk_kernel(LdShape g, const bf16 *q_hi, const bf16 *q_lo, const bf16 *c
   int b;
   const int p = g.position(r, b);
   const int j0 = max(0, p - g.window + 1) + blockIdx.x * g.span;
-  if (j0 > p) return;
-  const int total = min(g.span, p - j0 + 1), nt = (total + LD_KEYS - 1) / LD_KEYS;
+  if (!CLUSTER && j0 > p) return;
+  const int total = max(0, min(g.span, p - j0 + 1)), nt = (total + LD_KEYS - 1) / LD_KEYS;
   const int h0 = blockIdx.y * LD_HEADS, nh = min(LD_HEADS, g.heads - h0);
   const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
   const int gr = lane >> 2, tq = lane & 3;
@@ -351,7 +370,8 @@ latent_chunk_kernel(LdShape g, const bf16 *q_hi, const bf16 *q_lo, const bf16 *c
       copy16(ql + hh * pitch + c, q_lo + at + hh * rk + c, 16);
     }
   }
-  fetch(0);
+  if (nt > 0) fetch(0);
+  else copy_commit();
   float o[NT][4];
 #pragma unroll
   for (int i = 0; i < NT; ++i)
@@ -448,34 +468,137 @@ latent_chunk_kernel(LdShape g, const bf16 *q_hi, const bf16 *q_lo, const bf16 *c
       __syncthreads();  // the tile after next goes over this one
     }
   }
+  if constexpr (CLUSTER) {
+    copy_wait<0>();
+    __syncthreads();  // the tiles' space becomes this split's results: [16][rank4], then [16] (maximum, sum)
+    float *os = reinterpret_cast<float *>(tiles);
+    float2 *mls = reinterpret_cast<float2 *>(os + LD_HEADS * g.rank4);
+    const int r8 = (g.rank + 7) & ~7, ranks = g.splits;
+    const int share = (nh - (int)blockIdx.x + ranks - 1) / ranks;  // heads blockIdx.x, blockIdx.x + ranks, ... are this CTA's
+    float *ol = reinterpret_cast<float *>(qh);                     // [share][r8] weighted latents, over the queries
+    float *join = sc;                                              // [share][8] factors of the splits, over the scores
 #pragma unroll
-  for (int i = 0; i < 2; ++i)
-    if (lane == 0 && wid * 2 + i < nh)
-      part_ml[(r * g.heads + h0 + wid * 2 + i) * g.splits + blockIdx.x] = make_float2(m[i], l[i]);
+    for (int i = 0; i < 2; ++i)
+      if (lane == 0) mls[wid * 2 + i] = make_float2(m[i], l[i]);
 #pragma unroll
-  for (int i = 0; i < NT; ++i) {
-    const int c = (i * 8 + wid) * 8 + tq * 2;
-    if (c >= g.rank4) continue;  // columns behind the rank are zeros
+    for (int i = 0; i < NT; ++i) {
+      const int c = (i * 8 + wid) * 8 + tq * 2;
+      if (c >= g.rank4) continue;
+      *reinterpret_cast<float2 *>(os + gr * g.rank4 + c) = make_float2(o[i][0], o[i][1]);
+      *reinterpret_cast<float2 *>(os + (gr + 8) * g.rank4 + c) = make_float2(o[i][2], o[i][3]);
+    }
+    __syncwarp();
+    cluster_sync_all();
+    const unsigned os_at = smem_u32(os), ml_at = smem_u32(mls);
+    for (int i = wid; i < share; i += LD_THREADS / 32) {  // lane q looks at split q
+      const unsigned at = ml_at + (unsigned)((int)blockIdx.x + i * ranks) * 8u;
+      const float mq = lane < ranks ? ld_cluster_f32(cluster_map(at, (unsigned)lane)) : -INFINITY;
+      const float lq = lane < ranks ? ld_cluster_f32(cluster_map(at + 4u, (unsigned)lane)) : 0.f;
+      const float e = exp2f(mq - warp_max(mq));
+      const float sum = warp_sum(lq * e);
+      if (lane < ranks) join[i * LD_CLUSTER + lane] = e / sum;
+    }
+    __syncthreads();
+    const int cols = r8 >> 2;
+    for (int k = tid; k < share * cols; k += LD_THREADS) {
+      const int i = k / cols, c = (k - i * cols) * 4;
+      float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < g.rank4) {
+        const unsigned at = os_at + (unsigned)(((int)blockIdx.x + i * ranks) * g.rank4 + c) * 4u;
+        float4 v[LD_CLUSTER];
 #pragma unroll
-    for (int k = 0; k < 2; ++k)
-      if (gr + 8 * k < nh)
-        *reinterpret_cast<float2 *>(part_o + ((r * g.heads + h0 + gr + 8 * k) * g.splits + blockIdx.x) * (long long)g.rank4 +
-                                    c) = make_float2(o[i][2 * k], o[i][2 * k + 1]);
+        for (int q = 0; q < LD_CLUSTER; ++q)
+          v[q] = q < ranks ? ld_cluster_f4(cluster_map(at, (unsigned)q)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int q = 0; q < LD_CLUSTER; ++q)
+          if (q < ranks) {
+            const float f = join[i * LD_CLUSTER + q];
+            acc = make_float4(fmaf(f, v[q].x, acc.x), fmaf(f, v[q].y, acc.y), fmaf(f, v[q].z, acc.z), fmaf(f, v[q].w, acc.w));
+          }
+      }
+      *reinterpret_cast<float4 *>(ol + i * r8 + c) = acc;
+    }
+    __syncthreads();
+    // the value rows of all the CTA's heads, four per warp and trip; a row's loads precede their use
+    const int n_rows = share * g.vdim;
+    for (int k0 = wid * 4; k0 < n_rows; k0 += LD_THREADS / 32 * 4) {
+      float sum[4] = {};
+      const bf16 *wr[4];
+      const float *x[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int k = min(k0 + u, n_rows - 1), i = k / g.vdim, e = k - i * g.vdim;
+        wr[u] = w_uv + ((long long)(h0 + (int)blockIdx.x + i * ranks) * g.vdim + e) * w_ld;
+        x[u] = ol + i * r8;
+      }
+      for (int c = lane * 8; c < r8; c += 256) {
+        uint4 w4[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) w4[u] = *reinterpret_cast<const uint4 *>(wr[u] + c);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          float f[8];
+          unpack8(w4[u], f);
+          const float4 y = *reinterpret_cast<const float4 *>(x[u] + c), z = *reinterpret_cast<const float4 *>(x[u] + c + 4);
+          sum[u] = fmaf(f[0], y.x, fmaf(f[1], y.y, fmaf(f[2], y.z, fmaf(f[3], y.w, sum[u]))));
+          sum[u] = fmaf(f[4], z.x, fmaf(f[5], z.y, fmaf(f[6], z.z, fmaf(f[7], z.w, sum[u]))));
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const float v = warp_sum(sum[u]);
+        const int k = k0 + u, i = k / g.vdim;
+        if (lane == 0 && k < n_rows)
+          out[r * out_ld + (long long)(h0 + (int)blockIdx.x + i * ranks) * g.vdim + (k - i * g.vdim)] = __float2bfloat16_rn(v);
+      }
+    }
+    __syncwarp();
+    cluster_sync_all();  // a split's shared memory stays until every other has read it
+  } else {
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (lane == 0 && wid * 2 + i < nh)
+        part_ml[(r * g.heads + h0 + wid * 2 + i) * g.splits + blockIdx.x] = make_float2(m[i], l[i]);
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int c = (i * 8 + wid) * 8 + tq * 2;
+      if (c >= g.rank4) continue;  // columns behind the rank are zeros
+#pragma unroll
+      for (int k = 0; k < 2; ++k)
+        if (gr + 8 * k < nh)
+          *reinterpret_cast<float2 *>(part_o + ((r * g.heads + h0 + gr + 8 * k) * g.splits + blockIdx.x) * (long long)g.rank4 +
+                                      c) = make_float2(o[i][2 * k], o[i][2 * k + 1]);
+    }
   }
 }
 
 // Joins the splits of LD_ROWS rows of one head and maps the weighted latents through W_uv; the CTAs of
 // grid.y share the head's value rows.
+// PIECES: pieces of 256 latent columns a row of W_uv has (at most).
+template <int PIECES>
 __global__ void __launch_bounds__(LD_THREADS)
 latent_join_kernel(LdShape g, const float *part_o, const float2 *part_ml, const bf16 *__restrict__ w_uv,
                    int w_ld, long long n_rows, bf16 *out, int out_ld) {
   extern __shared__ __align__(16) float ol[];  // [LD_ROWS][rank rounded up to 8] weighted latents, then [LD_ROWS][splits]
   pdl_launch_dependents();
-  pdl_wait();
   const int h = blockIdx.x, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
   const long long r0 = (long long)blockIdx.z * LD_ROWS;
   const int nr = (int)min((long long)LD_ROWS, n_rows - r0);
   const int r8 = (g.rank + 7) & ~7;
+  const int e_per = (g.vdim + gridDim.y - 1) / gridDim.y;
+  const int e0 = blockIdx.y * e_per + wid, e1 = min(g.vdim, (int)(blockIdx.y + 1) * e_per);
+  constexpr int PRE = 4 / PIECES;  // value rows per warp that are requested ahead of the wait
+  const bf16 *wv = w_uv + (long long)h * g.vdim * w_ld;  // rows end on a multiple of 8 with zeros behind the rank
+  auto piece = [&](int e, int i) {
+    const int c = (i * 32 + lane) * 8;
+    return e < e1 && c < r8 ? *reinterpret_cast<const uint4 *>(wv + (long long)e * w_ld + c) : make_uint4(0, 0, 0, 0);
+  };
+  uint4 pre[PRE][PIECES];
+#pragma unroll
+  for (int k = 0; k < PRE; ++k)
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) pre[k][i] = piece(e0 + 8 * k, i);
+  pdl_wait();
   float *fac = ol + LD_ROWS * r8;
   __shared__ int counts[LD_ROWS];
   if (wid < nr) {
@@ -509,15 +632,14 @@ latent_join_kernel(LdShape g, const float *part_o, const float2 *part_ml, const 
     *reinterpret_cast<float4 *>(ol + r * r8 + c) = a;
   }
   __syncthreads();
-  const int e_per = (g.vdim + gridDim.y - 1) / gridDim.y;
-  const int e1 = min(g.vdim, (int)(blockIdx.y + 1) * e_per);
-#pragma unroll 2
-  for (int e = blockIdx.y * e_per + wid; e < e1; e += LD_THREADS / 32) {
-    const bf16 *wr = w_uv + ((long long)h * g.vdim + e) * w_ld;
+  auto value = [&](int e, const uint4 (&row)[PIECES]) {
     float s[LD_ROWS] = {};
-    for (int c = lane * 8; c < r8; c += 256) {  // rows of W_uv end on a multiple of 8 with zeros behind the rank
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+      const int c = (i * 32 + lane) * 8;
+      if (c >= r8) break;
       float f[8];
-      unpack8(*reinterpret_cast<const uint4 *>(wr + c), f);
+      unpack8(row[i], f);
 #pragma unroll
       for (int r = 0; r < LD_ROWS; ++r) {
         if (r >= nr) break;
@@ -532,9 +654,21 @@ latent_join_kernel(LdShape g, const float *part_o, const float2 *part_ml, const 
       const float v = warp_sum(s[r]);
       if (lane == 0) out[(r0 + r) * out_ld + (long long)h * g.vdim + e] = __float2bfloat16_rn(v);
     }
+  };
+#pragma unroll
+  for (int k = 0; k < PRE; ++k)
+    if (e0 + 8 * k < e1) value(e0 + 8 * k, pre[k]);
+  for (int e = e0 + 8 * PRE; e < e1; e += 8) {
+    uint4 row[PIECES];
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) row[i] = piece(e, i);
+    value(e, row);
   }
 }
 
+// (A cluster's join reuses the areas: the weighted latents, at most 16 rows of rank rounded up to 8 floats,
+// over the queries, 32 rows of at least rank + 8 halves; a split's results, 16 rows of rank floats and 16
+// pairs, over the first tile, 64 rows of at least rank + 8 halves.)
 size_t chunk_smem(int rank, int stages) {
   const int pitch = ((rank + 15) & ~15) + 8;
   return (size_t)(stages * LD_KEYS + 2 * LD_HEADS) * pitch * 2 + (size_t)2 * LD_HEADS * (LD_KEYS + 8) * 2 +
@@ -549,9 +683,12 @@ int most_splits(int heads, int window, int s_cap, long long rows) {
   const long long want = (2 * 148 + groups - 1) / groups;
   return (int)(want < tiles ? want : tiles);
 }
+constexpr int LD_CLUSTER_TILES = 4;  // key tiles per CTA up to which a cluster beats more splits and a second launch
 void plan_splits(int heads, int window, int s_cap, long long rows, int *splits, int *span) {
   const int tiles = ((window < s_cap ? window : s_cap) + LD_KEYS - 1) / LD_KEYS;
-  const int want = most_splits(heads, window, s_cap, rows), per = (tiles + want - 1) / want;
+  int want = most_splits(heads, window, s_cap, rows);
+  if (want > LD_CLUSTER && tiles <= LD_CLUSTER * LD_CLUSTER_TILES) want = LD_CLUSTER;
+  const int per = (tiles + want - 1) / want;
   *span = per * LD_KEYS;
   *splits = (tiles + per - 1) / per;
 }
@@ -570,13 +707,13 @@ LdScratch ld_scratch(int heads, int rank, int splits, long long rows) {
 void launch_latent_store(const float *dkv, int dkv_ld, const float *gain, float eps, const LatentCache &cache,
                          void *packed, int packed_rows, int first, Precision type, const RowBatch &b, cudaStream_t st) {
   const int count = packed ? b.p0 + b.n - first : b.n;
-  const dim3 grid((unsigned)((count + 3) / 4), (unsigned)b.streams);
+  const dim3 grid((unsigned)((count + 7) / 8), (unsigned)b.streams);
   if (type == Precision::BF16)
-    launch_pdl(latent_store_kernel<bf16>, grid, dim3(128), 0, st, g_pdl_enabled, dkv, dkv_ld, gain, eps,
+    launch_pdl(latent_store_kernel<bf16>, grid, dim3(256), 0, st, g_pdl_enabled, dkv, dkv_ld, gain, eps,
                static_cast<bf16 *>(cache.rows), cache.cap, cache.ld, cache.rank, static_cast<bf16 *>(packed), packed_rows,
                first, b.n, b.p0, b.state, b.slot0);
   else
-    launch_pdl(latent_store_kernel<float>, grid, dim3(128), 0, st, g_pdl_enabled, dkv, dkv_ld, gain, eps,
+    launch_pdl(latent_store_kernel<float>, grid, dim3(256), 0, st, g_pdl_enabled, dkv, dkv_ld, gain, eps,
                static_cast<float *>(cache.rows), cache.cap, cache.ld, cache.rank, static_cast<float *>(packed), packed_rows,
                first, b.n, b.p0, b.state, b.slot0);
 }
@@ -633,34 +770,54 @@ int launch_latent_decode(const LatentAttention &a, const LatentFresh &fresh, flo
   float *po = scratch + n.q + n.ml;
   const bf16 *cache = static_cast<const bf16 *>(a.cache.rows);
   const unsigned row_groups = (unsigned)((rows + LD_ROWS - 1) / LD_ROWS);
-  const size_t q_smem = (size_t)LD_ROWS * a.dim * sizeof(float);
-  if (q_smem + 8 * LD_ROWS * LQ_COLS * 4 > 48 * 1024)
-    LB_CUDA(cudaFuncSetAttribute(latent_query_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)q_smem));
-  launch_pdl(latent_query_kernel,
-             dim3((unsigned)((g.rk + LQ_COLS - 1) / LQ_COLS), (unsigned)(a.heads + (fresh.dkv ? 1 : 0)), row_groups),
-             dim3(LD_THREADS), q_smem, st, g_pdl_enabled, g, static_cast<const bf16 *>(a.q), a.q_ld,
-             static_cast<const bf16 *>(a.w_uk), a.w_ld, a.scale * LOG2E, rows, qh, ql, fresh,
-             static_cast<bf16 *>(a.cache.rows), a.cache.cap, a.cache.ld);
+  auto query = [&](auto kernel, int per) {
+    const size_t q_smem = (size_t)per * a.dim * sizeof(float);
+    if (q_smem + (size_t)8 * per * LQ_COLS * 4 > 48 * 1024)
+      LB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)q_smem));
+    launch_pdl(kernel,
+               dim3((unsigned)((g.rk + LQ_COLS - 1) / LQ_COLS), (unsigned)(a.heads + (fresh.dkv ? 1 : 0)),
+                    (unsigned)((rows + per - 1) / per)),
+               dim3(LD_THREADS), q_smem, st, g_pdl_enabled, g, static_cast<const bf16 *>(a.q), a.q_ld,
+               static_cast<const bf16 *>(a.w_uk), a.w_ld, a.scale * LOG2E, rows, qh, ql, fresh,
+               static_cast<bf16 *>(a.cache.rows), a.cache.cap, a.cache.ld);
+  };
+  if (rows < LD_ROWS) query(latent_query_kernel<1>, 1);
+  else query(latent_query_kernel<LD_ROWS>, LD_ROWS);
   const int stages = g.span > LD_KEYS && chunk_smem(g.rank, 2) <= LD_SMEM_LIMIT ? 2 : 1;
   const size_t smem = chunk_smem(g.rank, stages);
+  const bool cluster = g.splits <= LD_CLUSTER;
   auto chunk = [&](auto kernel) {
     if (smem > 48 * 1024) LB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    launch_pdl(kernel, dim3((unsigned)g.splits, (unsigned)(g.heads16 / LD_HEADS), (unsigned)rows), dim3(LD_THREADS), smem, st,
-               g_pdl_enabled, g, (const bf16 *)qh, (const bf16 *)ql, cache, a.cache.cap, a.cache.ld, stages, po, ml);
+    launch_pdl_cluster_x(kernel, dim3((unsigned)g.splits, (unsigned)(g.heads16 / LD_HEADS), (unsigned)rows), dim3(LD_THREADS),
+                         smem, st, g_pdl_enabled, cluster ? (unsigned)g.splits : 1u, g, (const bf16 *)qh, (const bf16 *)ql,
+                         cache, a.cache.cap, a.cache.ld, stages, po, ml, static_cast<const bf16 *>(a.w_uv), a.w_ld,
+                         static_cast<bf16 *>(a.out), a.out_ld);
   };
-  if (g.rk <= 128) chunk(latent_chunk_kernel<2>);
-  else if (g.rk <= 256) chunk(latent_chunk_kernel<4>);
-  else if (g.rk <= 512) chunk(latent_chunk_kernel<8>);
-  else chunk(latent_chunk_kernel<16>);
+  if (cluster) {
+    if (g.rk <= 128) chunk(latent_chunk_kernel<2, true>);
+    else if (g.rk <= 256) chunk(latent_chunk_kernel<4, true>);
+    else if (g.rk <= 512) chunk(latent_chunk_kernel<8, true>);
+    else chunk(latent_chunk_kernel<16, true>);
+    return 2;
+  }
+  if (g.rk <= 128) chunk(latent_chunk_kernel<2, false>);
+  else if (g.rk <= 256) chunk(latent_chunk_kernel<4, false>);
+  else if (g.rk <= 512) chunk(latent_chunk_kernel<8, false>);
+  else chunk(latent_chunk_kernel<16, false>);
   int parts = (int)(2 * 148 / ((long long)row_groups * a.heads > 2 * 148 ? 2 * 148 : (long long)row_groups * a.heads));
   const int most = (a.vdim + 7) / 8;
   parts = parts < 1 ? 1 : parts > most ? most : parts > 8 ? 8 : parts;
   const size_t j_smem = (size_t)LD_ROWS * (((g.rank + 7) & ~7) + g.splits) * sizeof(float);
-  if (j_smem > 48 * 1024)
-    LB_CUDA(cudaFuncSetAttribute(latent_join_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)j_smem));
-  launch_pdl(latent_join_kernel, dim3((unsigned)a.heads, (unsigned)parts, row_groups), dim3(LD_THREADS), j_smem, st,
-             g_pdl_enabled, g, (const float *)po, (const float2 *)ml, static_cast<const bf16 *>(a.w_uv), a.w_ld, rows,
-             static_cast<bf16 *>(a.out), a.out_ld);
+  auto join = [&](auto kernel) {
+    if (j_smem > 48 * 1024)
+      LB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)j_smem));
+    launch_pdl(kernel, dim3((unsigned)a.heads, (unsigned)parts, row_groups), dim3(LD_THREADS), j_smem, st, g_pdl_enabled, g,
+               (const float *)po, (const float2 *)ml, static_cast<const bf16 *>(a.w_uv), a.w_ld, rows,
+               static_cast<bf16 *>(a.out), a.out_ld);
+  };
+  if (g.rank <= 256) join(latent_join_kernel<1>);
+  else if (g.rank <= 512) join(latent_join_kernel<2>);
+  else join(latent_join_kernel<4>);
   return 3;
 }
 

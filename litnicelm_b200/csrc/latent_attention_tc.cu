@@ -47,7 +47,7 @@ struct LpArgs {
   int out_ld;
 };
 
-__global__ void __launch_bounds__(LP_THREADS)
+__global__ void __launch_bounds__(LP_THREADS, 2)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_vt, LpArgs a, DevErr *err) {
   extern __shared__ unsigned char smem_raw[];
@@ -186,21 +186,25 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       // keys j0 + c seen by this row: c in [c_lo, c_hi]; whole tiles inside every row's window need no mask
       const int c_hi = qrel - j0, c_lo = qrel - a.window + 1 - j0;
       const bool inside = wq0 - j0 >= LP_BK - 1 && wq0 + 31 - a.window + 1 - j0 <= 0;
-      float mx = LP_NEG;
-#pragma unroll 1
-      for (int c0 = 0; c0 < LP_BK; c0 += 32) {
-        unsigned r[32];
-        tc_ld32(tmem_s + lanes + (unsigned)c0, r);
+      // the row's scores stay in registers; independent chains for the maximum and the sum
+      float s[LP_BK];
+      {
+        unsigned(&u)[4][32] = reinterpret_cast<unsigned(&)[4][32]>(s);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) tc_ld32(tmem_s + lanes + (unsigned)(c * 32), u[c]);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-        if (inside) {
-#pragma unroll
-          for (int j = 0; j < 32; ++j) mx = fmaxf(mx, __uint_as_float(r[j]) * a.factor);
-        } else {
-#pragma unroll
-          for (int j = 0; j < 32; ++j)
-            mx = fmaxf(mx, c0 + j <= c_hi && c0 + j >= c_lo ? __uint_as_float(r[j]) * a.factor : LP_NEG);
-        }
       }
+#pragma unroll
+      for (int j = 0; j < LP_BK; ++j) s[j] *= a.factor;
+      if (!inside) {
+#pragma unroll
+        for (int j = 0; j < LP_BK; ++j)
+          if (j > c_hi || j < c_lo) s[j] = 2.f * LP_NEG;  // weight zero against any reference maximum
+      }
+      float mq[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+      for (int j = 4; j < LP_BK; ++j) mq[j & 3] = fmaxf(mq[j & 3], s[j]);
+      const float mx = fmaxf(LP_NEG, fmaxf(fmaxf(mq[0], mq[1]), fmaxf(mq[2], mq[3])));
       const bool grow = mx > m + LP_SLACK;
       const float keep = grow ? lp_exp2(m - mx) : 1.f;
       if (grow) m = mx;
@@ -221,28 +225,21 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
           }
         }
       }
-      float ls = 0.f;
-#pragma unroll 1
+      float lq[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
       for (int c0 = 0; c0 < LP_BK; c0 += 32) {
-        unsigned r[32], pk[16];
-        tc_ld32(tmem_s + lanes + (unsigned)c0, r);
-        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        unsigned pk[16];
 #pragma unroll
         for (int j = 0; j < 32; j += 2) {
-          float e0 = lp_exp2(fmaf(__uint_as_float(r[j]), a.factor, -m));
-          float e1 = lp_exp2(fmaf(__uint_as_float(r[j + 1]), a.factor, -m));
-          if (!inside) {
-            if (c0 + j > c_hi || c0 + j < c_lo) e0 = 0.f;
-            if (c0 + j + 1 > c_hi || c0 + j + 1 < c_lo) e1 = 0.f;
-          }
-          ls += e0 + e1;
+          const float e0 = lp_exp2(s[c0 + j] - m), e1 = lp_exp2(s[c0 + j + 1] - m);
+          lq[j & 2] += e0;
+          lq[(j & 2) + 1] += e1;
           const __nv_bfloat162 v = __floats2bfloat162_rn(e0, e1);
           pk[j >> 1] = *reinterpret_cast<const unsigned *>(&v);
         }
-        // columns c0 / 2 .. + 15: scores there have been read by this warp already
-        tc_st16(tmem_s + lanes + (unsigned)(c0 >> 1), pk);
+        tc_st16(tmem_s + lanes + (unsigned)(c0 >> 1), pk);  // over the scores, which this warp has read
       }
-      l += ls;
+      l += (lq[0] + lq[1]) + (lq[2] + lq[3]);
       asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();

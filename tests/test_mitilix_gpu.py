@@ -123,6 +123,8 @@ ATT_TOL = {0: 3e-6, 1: 8e-3, 2: 8e-3, 3: 1.2e-2}
     (1, 260, 20, 1, 80, 144, 32, 128),    # two slabs of the head, wide values
     (1, 400, 131, 1, 256, 256, 64, 7),
     (1, 40, 40, 2, 32, 32, 512, 1),       # sees itself only
+    (1, 2300, 3, 3, 32, 48, 72, 2200),    # more splits of the window than a cluster has CTAs
+    (2, 700, 30, 18, 16, 16, 264, 650),   # several tiles per split, two groups of heads
 ])
 def test_latent_attention(engine, streams, t, n, heads, dim, vdim, rank, window):
     if engine == 2 and streams * n > 64:
