@@ -116,7 +116,7 @@ few_row_bf16_kernel(FewRowPair pair, int m, int ranks) {
           fr_mma(acc[i], wa[u].x, wb[u].x, wa[u].y, wb[u].y, v.x, v.y);
           fr_mma(acc[i], wa[u].z, wb[u].z, wa[u].w, wb[u].w, v.z, v.w);
         }
-    }
+      }
     }
     if (k0 + FR_WARPS * SPAN < k_end) load_w(k0 + FR_WARPS * SPAN);
   }

@@ -338,6 +338,14 @@ latent_chunk_kernel(LdShape g, const bf16 *q_hi, const bf16 *q_lo, const bf16 *c
   float *fac = sc + LD_HEADS * SP;                   // [16] factors of what has been summed so far
   bf16 *tiles = reinterpret_cast<bf16 *>(fac + LD_HEADS);     // [stages][LD_KEYS][pitch]
   pdl_launch_dependents();
+  if constexpr (CLUSTER) {  // the value rows this CTA maps its heads through depend on nothing: towards L2 now
+    const int nh = min(LD_HEADS, g.heads - (int)blockIdx.y * LD_HEADS);
+    for (int hh = blockIdx.x; hh < nh; hh += g.splits) {
+      const char *rows = reinterpret_cast<const char *>(w_uv + (long long)(blockIdx.y * LD_HEADS + hh) * g.vdim * w_ld);
+      for (int at = threadIdx.x * 128; at < g.vdim * w_ld * 2; at += LD_THREADS * 128)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(rows + at));
+    }
+  }
   pdl_wait();
   const long long r = blockIdx.z;
   int b;
