@@ -272,7 +272,8 @@ void launch_layernorm_dense(const float *x, const float *gamma, const float *bet
 
 // gemv.cu: out[m, n] = x[m, :] . W[:, n] for m <= 8 rows; W row-major [k, n].
 // scratch must hold gemv_scratch_floats(m, n, k) floats when the launcher
-// decides to split k across CTAs. x must hold 1, 2, 4 or 8 rows (m rounded up).
+// decides to split k across CTAs. x and out must hold 1, 2, 4 or 8 rows (m rounded up;
+// the rows behind m are read and written).
 // err (optional) receives DEVERR_WAIT_TIMEOUT if a bounded wait of the
 // streaming kernel runs out. Returns the number of kernels launched.
 size_t gemv_scratch_floats(int m, int n, int k);

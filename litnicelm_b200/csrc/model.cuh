@@ -76,7 +76,8 @@ class DecoderModel {
   // number of kernels launched.
   virtual int enqueue_rows(const RowBatch &batch, cudaStream_t st, DevErr *err) = 0;
   // Logits [n_rows, vocab] of rows of the batch just enqueued: the rows listed at rows_dev (device
-  // memory), or, with rows_dev == nullptr, the last row of every stream.
+  // memory), or, with rows_dev == nullptr, the last row of every stream. logits has room for n_rows
+  // rounded up to a multiple of 8.
   virtual int enqueue_head(const RowBatch &batch, const int *rows_dev, int n_rows, float *logits, cudaStream_t st,
                            DevErr *err) = 0;
   // Contexts of one bucket replay the same captured step: its upper bound for a context of s.

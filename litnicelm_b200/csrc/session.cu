@@ -919,6 +919,7 @@ void model_decode_step(litnice_b200_session *s, int B, int s_cap, int sl, const 
 }
 
 void ensure_logits_all(litnice_b200_session *s, long long rows) {
+  rows = (rows + 7) / 8 * 8;  // the float few-row product writes its row count rounded up to 1, 2, 4 or 8
   if (s->logits_all_rows >= rows) return;
   LB_CUDA(cudaStreamSynchronize(s->st));
   if (s->logits_all) cudaFree(s->logits_all);
