@@ -27,7 +27,7 @@
 // (litnice_b200_session_create_model) instead of a litnicelm checkpoint; it has no
 // tokenizer, so prompts are token ids and text is printed as ids. `trace` replays
 // given token ids: one JSON step per line of standard input,
-//   {"step": 0, "entries": [{"id": "a", "tokens": [5, 17], "want": [0, 1]}], "end": ["a"]}
+//   {"step": 0, "entries": [{"id": "a", "tokens": [11, 42], "want": [0, 1]}], "end": ["a"]}
 // feeds each entry's tokens to its sequence, writes the logits of the wanted places to
 // DIR/<step>.f32 (little-endian floats, [wanted, vocab]) and answers "done <step>".
 #include <dlfcn.h>

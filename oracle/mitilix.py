@@ -1,4 +1,4 @@
-"""Plain, slow implementation of the Mitilix decoder in numpy: the checker of the CUDA path.
+"""Plain, slow implementation of the Mitilix decoder in numpy, for the tests of the CUDA path.
 
 One function per mechanism, written from the equations in double precision; nothing here is
 shared with the product path. Weights are a dict name -> array (linear weights [out, in]).
