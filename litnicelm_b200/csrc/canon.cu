@@ -247,7 +247,7 @@ rms_canon_vec_kernel(const float *x, int d, float gain, float eps, float *histor
 
 template <typename T>
 __global__ void __launch_bounds__(CN_THREADS)
-rms_rows_kernel(const float *x, int d, float gain, float eps, const int *rows_list,
+rms_rows_kernel(const float *x, int d, RmsWeight weight, float eps, const int *rows_list,
                 int n_per_stream, T *__restrict__ out, int ld) {
   __shared__ float part[CN_THREADS / 32];
   pdl_launch_dependents();
@@ -264,8 +264,8 @@ rms_rows_kernel(const float *x, int d, float gain, float eps, const int *rows_li
   s = 0.f;
 #pragma unroll
   for (int i = 0; i < CN_THREADS / 32; ++i) s += part[i];
-  const float inv = 1.0f / sqrtf(s / (float)d + eps) * gain;
-  for (int c = threadIdx.x; c < d; c += CN_THREADS) out[(long long)r * ld + c] = from_float<T>(row[c] * inv);
+  const float inv = 1.0f / sqrtf(s / (float)d + eps);
+  for (int c = threadIdx.x; c < d; c += CN_THREADS) out[(long long)r * ld + c] = from_float<T>(row[c] * inv * weight.at(c));
 }
 
 template <typename T>
@@ -326,13 +326,13 @@ void launch_rms_canon(const float *x, int d, float gain, float eps, int taps, fl
   else launch_canon_t<float>(x, d, gain, eps, taps, history, cv, b, st);
 }
 
-void launch_rms_rows(const float *x, int d, float gain, float eps, const int *rows_dev, int n_rows, int n_per_stream,
+void launch_rms_rows(const float *x, int d, const RmsWeight &weight, float eps, const int *rows_dev, int n_rows, int n_per_stream,
                      void *out, int ld, Precision type, cudaStream_t st) {
   if (type == Precision::BF16)
-    launch_pdl(rms_rows_kernel<__nv_bfloat16>, dim3((unsigned)n_rows), dim3(CN_THREADS), 0, st, g_pdl_enabled, x, d, gain,
+    launch_pdl(rms_rows_kernel<__nv_bfloat16>, dim3((unsigned)n_rows), dim3(CN_THREADS), 0, st, g_pdl_enabled, x, d, weight,
                eps, rows_dev, n_per_stream, static_cast<__nv_bfloat16 *>(out), ld);
   else
-    launch_pdl(rms_rows_kernel<float>, dim3((unsigned)n_rows), dim3(CN_THREADS), 0, st, g_pdl_enabled, x, d, gain, eps,
+    launch_pdl(rms_rows_kernel<float>, dim3((unsigned)n_rows), dim3(CN_THREADS), 0, st, g_pdl_enabled, x, d, weight, eps,
                rows_dev, n_per_stream, static_cast<float *>(out), ld);
 }
 

@@ -1,0 +1,628 @@
+// The gated delta rule of many new rows on bfloat16, in chunks of 64 tokens.
+//
+// Inside a chunk, with G_i the sum of the logarithms of the decays up to token i, r_i = 1 / |k'_i|,
+// r'_i = dim^-1/2 / |q'_i| (k', q' the convolved vectors as stored) and S the state before the chunk, the rule's
+// updates u_i solve a unit lower triangular system:
+//   L_ij = beta_i r_i r_j e^(G_i - G_j) (k'_i . k'_j)  (j < i),   (I + L) U = diag(beta) (V - diag(e^G_i r_i) K' S)
+//   A_ij = r'_i r_j e^(G_i - G_j) (q'_i . k'_j)        (j <= i),  O = diag(e^G_i r'_i) Q' S + A U
+//   S <- e^G_last S + (diag(e^(G_last - G_j) r_j) K')^T U
+// Exponents are never positive, and the vectors' norms stay out of the matrix operands, which are the stored
+// bfloat16 values themselves. Everything else that enters a product (the state, (I + L)^-1 diag(beta), A, the
+// right-hand side, U) is 32-bit and enters as two bfloat16 terms.
+//
+//   delta_prepare_kernel   per chunk and key head: K'K'^T and Q'K'^T, then per head L, its inverse by blocks of
+//                          32, A, and the factors of a token; no chunk depends on another
+//   delta_scan_kernel      per stream, head and tile of value columns: the chunks in order. A warp owns 16 value
+//                          columns and keeps their part of S^T in registers as accumulators of mma.sync tiles,
+//                          whose layout is that of the next product's left operand: the chain
+//                          S^T K'^T -> right-hand side -> U^T -> O^T, S^T runs without leaving the warp, on tiles
+//                          of K', Q', V and the chunk's matrices that all warps share (cp.async, two stages).
+//                          Where the CTA holds a whole head the output's norm and gate follow at once.
+// (A register-resident chain on mma.sync rather than tcgen05: each product's result is the next one's operand
+// after an elementwise step, and tensor memory would put a store, a fence and a barrier between any two.)
+#include "delta.cuh"
+
+namespace lb {
+
+namespace {
+
+typedef __nv_bfloat16 bf16;
+
+constexpr int CH = 64;           // tokens per chunk
+constexpr int MP = CH + 8;       // pitch of the chunk's matrices in shared memory
+constexpr int PREP_THREADS = 128;
+constexpr int TP = 68;           // pitch of the float matrices
+
+__device__ __forceinline__ unsigned smem_addr(const void *p) { return (unsigned)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldmatrix4(unsigned (&r)[4], const bf16 *p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_addr(p)));
+}
+__device__ __forceinline__ void ldmatrix4_trans(unsigned (&r)[4], const bf16 *p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_addr(p)));
+}
+__device__ __forceinline__ void mma(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// 16 bytes to shared memory in the background; false stores zeros.
+__device__ __forceinline__ void copy16(void *dst, const void *src, bool in) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void copy_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+__device__ __forceinline__ unsigned pack(float a, float b) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const unsigned *>(&v);
+}
+__device__ __forceinline__ float low_half(unsigned u) { return __uint_as_float(u << 16); }
+__device__ __forceinline__ float high_half(unsigned u) { return __uint_as_float(u & 0xffff0000u); }
+// Two floats as two terms of two packed bfloat16 each.
+__device__ __forceinline__ void split(float a, float b, unsigned &hi, unsigned &lo) {
+  hi = pack(a, b);
+  lo = pack(a - low_half(hi), b - high_half(hi));
+}
+// Left operand (16 x 16) from two neighbouring accumulator tiles of 16 x 8.
+__device__ __forceinline__ void operand(const float (&c0)[4], const float (&c1)[4], unsigned (&hi)[4], unsigned (&lo)[4]) {
+  split(c0[0], c0[1], hi[0], lo[0]);
+  split(c0[2], c0[3], hi[1], lo[1]);
+  split(c1[0], c1[1], hi[2], lo[2]);
+  split(c1[2], c1[3], hi[3], lo[3]);
+}
+
+struct ChunkArgs {
+  int heads, groups, dim, vdim, channels, n, chunks;
+  float q_scale;
+  const float *a_log, *dt_bias;
+  const float *ba;
+  int ba_ld;
+};
+
+// Matrices of a chunk and head: [inverse high, low, A high, low][64][64], only blocks of 16 columns that start at or
+// below the diagonal of their 16 rows are written and read.
+constexpr int MAT = CH * CH;
+// Factors of a token: e^G r, e^G r', e^(G_last - G) r, e^G_last.
+__device__ __forceinline__ long long chunk_at(const ChunkArgs &a, int b, int h, int chunk) {
+  return ((long long)b * a.heads + h) * a.chunks + chunk;
+}
+
+__global__ void __launch_bounds__(PREP_THREADS)
+delta_prepare_kernel(ChunkArgs a, const bf16 *conv, bf16 *mats, float4 *factors) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int pitch = a.dim + 8;
+  bf16 *ks = reinterpret_cast<bf16 *>(raw), *qs = ks + CH * pitch;
+  float *ls = reinterpret_cast<float *>(qs + CH * pitch);  // [64][TP] L
+  float *ts = ls + CH * TP;                                // [64][TP] its inverse
+  __shared__ double gs[CH];
+  __shared__ float rk[CH], rq[CH], bs[CH];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, g = lane >> 2, t2 = (lane & 3) * 2;
+  const int chunk = blockIdx.x, grp = blockIdx.y, b = blockIdx.z;
+  const int t0 = chunk * CH, nt = min(CH, a.n - t0);
+  const long long r0 = (long long)b * a.n + t0;
+  const bf16 *src = conv + r0 * a.channels + grp * a.dim;
+  const int pieces = a.dim >> 3;
+  for (int i = tid; i < CH * pieces; i += PREP_THREADS) {
+    const int t = i / pieces, c = (i - t * pieces) * 8;
+    const bf16 *row = t < nt ? src + (long long)t * a.channels + c : src;
+    copy16(qs + t * pitch + c, row, t < nt);
+    copy16(ks + t * pitch + c, row + a.groups * a.dim, t < nt);
+  }
+  copy_commit();
+  copy_wait_all();
+  __syncthreads();
+  {  // one thread per row and kind
+    const int t = tid & 63;
+    const bf16 *row = (tid < 64 ? ks : qs) + t * pitch;
+    float s = 0.f;
+    for (int c = 0; c < a.dim; c += 8) {
+      const uint4 u = *reinterpret_cast<const uint4 *>(row + c);
+      const unsigned w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s += low_half(w[i]) * low_half(w[i]) + high_half(w[i]) * high_half(w[i]);
+    }
+    if (tid < 64) rk[t] = 1.0f / sqrtf(s + DELTA_UNIT_EPS);
+    else rq[t] = a.q_scale / sqrtf(s + DELTA_UNIT_EPS);
+  }
+  // products of the warp's 16 rows with the tokens up to its last row
+  const int w0 = wid * 16;
+  float kk[8][4], qk[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) kk[i][j] = qk[i][j] = 0.f;
+  const int ar = w0 + (lane & 15), ac = (lane >> 4) * 8;                        // left operand's row and column
+  const int br = (lane & 7) + ((lane >> 4) << 3), bc = ((lane >> 3) & 1) * 8;  // right operand: two tiles of 8 tokens
+  for (int c = 0; c < a.dim; c += 16) {
+    unsigned ak[4], aq[4];
+    ldmatrix4(ak, ks + ar * pitch + c + ac);
+    ldmatrix4(aq, qs + ar * pitch + c + ac);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (j > wid) break;
+      unsigned bk[4];
+      ldmatrix4(bk, ks + (j * 16 + br) * pitch + c + bc);
+      mma(kk[2 * j], ak, bk[0], bk[1]);
+      mma(kk[2 * j + 1], ak, bk[2], bk[3]);
+      mma(qk[2 * j], aq, bk[0], bk[1]);
+      mma(qk[2 * j + 1], aq, bk[2], bk[3]);
+    }
+  }
+  const int per = a.heads / a.groups;
+  for (int hh = 0; hh < per; ++hh) {
+    const int h = grp * per + hh;
+    const long long at = chunk_at(a, b, h, chunk);
+    __syncthreads();  // norms are there; the previous head is done with ls, ts and the factors
+    if (wid == 0) {  // sums of the decays' logarithms, two tokens per lane
+      double x[2];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = lane * 2 + i;
+        const float *row = a.ba + (r0 + t) * a.ba_ld + h;
+        x[i] = t < nt ? (double)delta_log_decay(row[a.heads], a.a_log[h], a.dt_bias[h]) : 0.0;
+        bs[t] = t < nt ? sigmoid_f32(row[0]) : 0.f;
+      }
+      double sum = x[0] + x[1];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const double y = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += y;
+      }
+      gs[lane * 2] = sum - x[1];
+      gs[lane * 2 + 1] = sum;
+    }
+    __syncthreads();
+    const double last = gs[CH - 1];
+    if (tid < CH) {
+      const float e = expf((float)gs[tid]);
+      factors[at * CH + tid] = make_float4(e * rk[tid], e * rq[tid], expf((float)(last - gs[tid])) * rk[tid], expf((float)last));
+    }
+    bf16 *mat = mats + at * 4 * MAT;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (j > 2 * wid + 1) break;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int i = w0 + g + half * 8;
+        float e[2], av[2];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          const int col = j * 8 + t2 + k;
+          e[k] = col <= i ? expf((float)(gs[i] - gs[col])) * rk[col] : 0.f;
+          av[k] = e[k] * rq[i] * qk[j][half * 2 + k];
+          ls[i * TP + col] = col < i ? e[k] * bs[i] * rk[i] * kk[j][half * 2 + k] : 0.f;
+        }
+        unsigned hi, lo;
+        split(av[0], av[1], hi, lo);
+        *reinterpret_cast<unsigned *>(mat + 2 * MAT + i * CH + j * 8 + t2) = hi;
+        *reinterpret_cast<unsigned *>(mat + 3 * MAT + i * CH + j * 8 + t2) = lo;
+      }
+    }
+    __syncthreads();
+    // inverse of I + L: the two diagonal blocks of 32 by forward substitution, one column per lane
+    if (wid < 2) {
+      const float *lb = ls + wid * 32 * TP + wid * 32;
+      float x[32];
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        float s = i == lane ? 1.f : 0.f;
+#pragma unroll
+        for (int j = 0; j < i; ++j) s = fmaf(-lb[i * TP + j], x[j], s);
+        x[i] = s;
+      }
+#pragma unroll
+      for (int i = 0; i < 32; ++i) ts[(wid * 32 + i) * TP + wid * 32 + lane] = x[i];
+    }
+    __syncthreads();
+    {  // the block below them: -(second inverse) L21 (first inverse); the upper right block holds L21 (first inverse)
+      const int r = tid >> 2, c = (tid & 3) * 8;
+      float m[8] = {};
+      for (int j = 0; j < 32; ++j) {
+        const float l = ls[(32 + r) * TP + j];
+        const float4 x = *reinterpret_cast<const float4 *>(ts + j * TP + c), y = *reinterpret_cast<const float4 *>(ts + j * TP + c + 4);
+        m[0] = fmaf(l, x.x, m[0]);
+        m[1] = fmaf(l, x.y, m[1]);
+        m[2] = fmaf(l, x.z, m[2]);
+        m[3] = fmaf(l, x.w, m[3]);
+        m[4] = fmaf(l, y.x, m[4]);
+        m[5] = fmaf(l, y.y, m[5]);
+        m[6] = fmaf(l, y.z, m[6]);
+        m[7] = fmaf(l, y.w, m[7]);
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ts[r * TP + 32 + c + i] = m[i];
+      __syncthreads();
+      float n[8] = {};
+      for (int j = 0; j < 32; ++j) {
+        const float l = -ts[(32 + r) * TP + 32 + j];
+        const float *row = ts + j * TP + 32 + c;
+        const float4 x = *reinterpret_cast<const float4 *>(row), y = *reinterpret_cast<const float4 *>(row + 4);
+        n[0] = fmaf(l, x.x, n[0]);
+        n[1] = fmaf(l, x.y, n[1]);
+        n[2] = fmaf(l, x.z, n[2]);
+        n[3] = fmaf(l, x.w, n[3]);
+        n[4] = fmaf(l, y.x, n[4]);
+        n[5] = fmaf(l, y.y, n[5]);
+        n[6] = fmaf(l, y.z, n[6]);
+        n[7] = fmaf(l, y.w, n[7]);
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ts[(32 + r) * TP + c + i] = n[i];
+    }
+    __syncthreads();
+    for (int i = tid; i < CH * (CH / 8); i += PREP_THREADS) {
+      const int r = i >> 3, c = (i & 7) * 8;
+      if (c >= (r / 16 + 1) * 16) continue;
+      unsigned hi[4], lo[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const int c0 = c + 2 * k, c1 = c0 + 1;
+        split(c0 <= r ? ts[r * TP + c0] * bs[c0] : 0.f, c1 <= r ? ts[r * TP + c1] * bs[c1] : 0.f, hi[k], lo[k]);
+      }
+      *reinterpret_cast<uint4 *>(mat + r * CH + c) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4 *>(mat + MAT + r * CH + c) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+  }
+}
+
+struct ScanArgs {
+  ChunkArgs c;
+  int p0, slot0, stages;
+  float *state, *o;
+  const bf16 *gate;
+  int in_ld, out_ld, normed;
+  float count, eps;
+  const float *norm;
+  bf16 *out;
+};
+
+// Shared memory of a stage, in bfloat16 elements (the token factors, 64 float4, behind them).
+__host__ __device__ __forceinline__ int stage_elems(int dim, int vt) {
+  return 2 * CH * (dim + 8) + CH * (vt + 8) + 4 * CH * MP + CH * 8;
+}
+
+// NT: tiles of 8 state rows (dim / 8 at most); WARPS: 16 value columns each. TWO_PASS: the products of the state
+// with keys and with queries one after the other (fewer registers).
+template <int NT, int WARPS, bool TWO_PASS>
+__global__ void __launch_bounds__(WARPS * 32)
+delta_scan_kernel(ScanArgs s, const bf16 *conv, const bf16 *mats, const float4 *factors) {
+  constexpr int THREADS = WARPS * 32, VT = WARPS * 16, SP = VT + 4;
+  extern __shared__ __align__(16) unsigned char raw[];
+  const ChunkArgs &a = s.c;
+  const int pitch = a.dim + 8, vp = VT + 8, elems = stage_elems(a.dim, VT);
+  bf16 *stages = reinterpret_cast<bf16 *>(raw);
+  float *stage_o = reinterpret_cast<float *>(stages + (size_t)s.stages * elems);  // [64][SP] outputs of the chunk
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, g = lane >> 2, t2 = (lane & 3) * 2;
+  const int tiles = (a.vdim + VT - 1) / VT;
+  const int h = blockIdx.x / tiles, vt = (blockIdx.x - h * tiles) * VT, b = blockIdx.y;
+  const int grp = h / (a.heads / a.groups);
+  const int cols = min(VT, a.vdim - vt);
+  const bf16 *base = conv + (long long)b * a.n * a.channels;
+  const int q_at = grp * a.dim, k_at = (a.groups + grp) * a.dim, v_at = 2 * a.groups * a.dim + h * a.vdim + vt;
+  auto load = [&](int chunk) {
+    bf16 *ks = stages + (size_t)(chunk % s.stages) * elems, *qs = ks + CH * pitch, *vs = qs + CH * pitch, *ms = vs + CH * vp;
+    float4 *fs = reinterpret_cast<float4 *>(ms + 4 * CH * MP);
+    const int t0 = chunk * CH, nt = min(CH, a.n - t0), pieces = a.dim >> 3;
+    const bf16 *rows = base + (long long)t0 * a.channels;
+    for (int i = tid; i < CH * pieces; i += THREADS) {
+      const int t = i / pieces, c = (i - t * pieces) * 8;
+      const bf16 *row = t < nt ? rows + (long long)t * a.channels : rows;
+      copy16(ks + t * pitch + c, row + k_at + c, t < nt);
+      copy16(qs + t * pitch + c, row + q_at + c, t < nt);
+    }
+    for (int i = tid; i < CH * (VT / 8); i += THREADS) {
+      const int t = i / (VT / 8), c = (i - t * (VT / 8)) * 8;
+      const bool in = t < nt && c < cols;
+      copy16(vs + t * vp + c, in ? rows + (long long)t * a.channels + v_at + c : rows, in);
+    }
+    const long long at = chunk_at(a, b, h, chunk);
+    for (int i = tid; i < 4 * CH * 8; i += THREADS) {
+      const int m = i >> 9, r = (i >> 3) & 63, c = (i & 7) * 8;
+      if (c < (r / 16 + 1) * 16) copy16(ms + (m * CH + r) * MP + c, mats + (at * 4 + m) * MAT + r * CH + c, true);
+    }
+    for (int i = tid; i < CH; i += THREADS) copy16(fs + i, factors + at * CH + i, true);
+    copy_commit();
+  };
+  load(0);
+  // S^T: this warp's 16 value columns by all state rows; element (v, d) of tile d / 8
+  const int v0 = vt + wid * 16 + g;
+  float *S = s.state + ((long long)(s.slot0 + b) * a.heads + h) * a.dim * a.vdim;
+  float st[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int d = i * 8 + t2 + (j & 1), v = v0 + (j >> 1) * 8;
+      st[i][j] = s.p0 > 0 && d < a.dim && v < a.vdim ? S[(long long)d * a.vdim + v] : 0.f;
+    }
+  const int br = (lane & 7) + ((lane >> 4) << 3), bc = ((lane >> 3) & 1) * 8;  // right operand, index rows
+  const int tr = (lane & 7) + ((lane >> 3) & 1) * 8, tc = (lane >> 4) * 8;     // right operand, k rows (transposed on load)
+  for (int chunk = 0; chunk < a.chunks; ++chunk) {
+    copy_wait_all();
+    __syncthreads();
+    if (s.stages > 1 && chunk + 1 < a.chunks) load(chunk + 1);
+    const bf16 *ks = stages + (size_t)(chunk % s.stages) * elems, *qs = ks + CH * pitch, *vs = qs + CH * pitch,
+               *ms = vs + CH * vp;
+    const float4 *fs = reinterpret_cast<const float4 *>(ms + 4 * CH * MP);
+    float pk[8][4], pq[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) pk[i][j] = pq[i][j] = 0.f;
+    // S^T K'^T (and S^T Q'^T)
+#pragma unroll
+    for (int kt = 0; kt < NT / 2; ++kt) {
+      if (kt * 16 < a.dim) {
+        unsigned hi[4], lo[4];
+        operand(st[2 * kt], st[2 * kt + 1], hi, lo);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          unsigned x[4];
+          ldmatrix4(x, ks + (j * 16 + br) * pitch + kt * 16 + bc);
+          mma(pk[2 * j], lo, x[0], x[1]);
+          mma(pk[2 * j + 1], lo, x[2], x[3]);
+          mma(pk[2 * j], hi, x[0], x[1]);
+          mma(pk[2 * j + 1], hi, x[2], x[3]);
+          if (!TWO_PASS) {
+            ldmatrix4(x, qs + (j * 16 + br) * pitch + kt * 16 + bc);
+            mma(pq[2 * j], lo, x[0], x[1]);
+            mma(pq[2 * j + 1], lo, x[2], x[3]);
+            mma(pq[2 * j], hi, x[0], x[1]);
+            mma(pq[2 * j + 1], hi, x[2], x[3]);
+          }
+        }
+      }
+    }
+    // right-hand side V^T - e^G r (S^T K'^T)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      unsigned x[4];
+      ldmatrix4_trans(x, vs + (j * 16 + br) * vp + wid * 16 + bc);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = j * 16 + i * 8 + t2;
+        const float f0 = fs[t].x, f1 = fs[t + 1].x;
+        float(&p)[4] = pk[2 * j + i];
+        p[0] = low_half(x[2 * i]) - f0 * p[0];
+        p[1] = high_half(x[2 * i]) - f1 * p[1];
+        p[2] = low_half(x[2 * i + 1]) - f0 * p[2];
+        p[3] = high_half(x[2 * i + 1]) - f1 * p[3];
+      }
+    }
+    // U^T = (right-hand side)^T ((I + L)^-1 diag(beta))^T
+    float u[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) u[i][j] = 0.f;
+#pragma unroll
+    for (int kt = 0; kt < 4; ++kt) {
+      unsigned hi[4], lo[4];
+      operand(pk[2 * kt], pk[2 * kt + 1], hi, lo);
+#pragma unroll
+      for (int j = kt; j < 4; ++j) {
+        unsigned x[4], y[4];
+        ldmatrix4(x, ms + (j * 16 + br) * MP + kt * 16 + bc);
+        ldmatrix4(y, ms + (CH + j * 16 + br) * MP + kt * 16 + bc);
+        mma(u[2 * j], lo, x[0], x[1]);
+        mma(u[2 * j + 1], lo, x[2], x[3]);
+        mma(u[2 * j], hi, y[0], y[1]);
+        mma(u[2 * j + 1], hi, y[2], y[3]);
+        mma(u[2 * j], hi, x[0], x[1]);
+        mma(u[2 * j + 1], hi, x[2], x[3]);
+      }
+    }
+    if (TWO_PASS) {
+#pragma unroll
+      for (int kt = 0; kt < NT / 2; ++kt) {
+        if (kt * 16 < a.dim) {
+          unsigned hi[4], lo[4];
+          operand(st[2 * kt], st[2 * kt + 1], hi, lo);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            unsigned x[4];
+            ldmatrix4(x, qs + (j * 16 + br) * pitch + kt * 16 + bc);
+            mma(pq[2 * j], lo, x[0], x[1]);
+            mma(pq[2 * j + 1], lo, x[2], x[3]);
+            mma(pq[2 * j], hi, x[0], x[1]);
+            mma(pq[2 * j + 1], hi, x[2], x[3]);
+          }
+        }
+      }
+    }
+    // O^T = e^G r' (S^T Q'^T) + U^T A^T
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float f0 = fs[i * 8 + t2].y, f1 = fs[i * 8 + t2 + 1].y;
+      pq[i][0] *= f0;
+      pq[i][1] *= f1;
+      pq[i][2] *= f0;
+      pq[i][3] *= f1;
+    }
+#pragma unroll
+    for (int kt = 0; kt < 4; ++kt) {
+      unsigned hi[4], lo[4];
+      operand(u[2 * kt], u[2 * kt + 1], hi, lo);
+#pragma unroll
+      for (int j = kt; j < 4; ++j) {
+        unsigned x[4], y[4];
+        ldmatrix4(x, ms + (2 * CH + j * 16 + br) * MP + kt * 16 + bc);
+        ldmatrix4(y, ms + (3 * CH + j * 16 + br) * MP + kt * 16 + bc);
+        mma(pq[2 * j], lo, x[0], x[1]);
+        mma(pq[2 * j + 1], lo, x[2], x[3]);
+        mma(pq[2 * j], hi, y[0], y[1]);
+        mma(pq[2 * j + 1], hi, y[2], y[3]);
+        mma(pq[2 * j], hi, x[0], x[1]);
+        mma(pq[2 * j + 1], hi, x[2], x[3]);
+      }
+    }
+    // S^T <- e^G_last S^T + (U^T diag(e^(G_last - G) r)) K'
+    const float keep = fs[0].w;
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) st[i][j] *= keep;
+#pragma unroll
+    for (int kt = 0; kt < 4; ++kt) {
+#pragma unroll
+      for (int i = 2 * kt; i < 2 * kt + 2; ++i) {
+        const float f0 = fs[i * 8 + t2].z, f1 = fs[i * 8 + t2 + 1].z;
+        u[i][0] *= f0;
+        u[i][1] *= f1;
+        u[i][2] *= f0;
+        u[i][3] *= f1;
+      }
+      unsigned hi[4], lo[4];
+      operand(u[2 * kt], u[2 * kt + 1], hi, lo);
+#pragma unroll
+      for (int i = 0; i < NT / 2; ++i) {
+        if (i * 16 < a.dim) {
+          unsigned x[4];
+          ldmatrix4_trans(x, ks + (kt * 16 + tr) * pitch + i * 16 + tc);
+          mma(st[2 * i], lo, x[0], x[1]);
+          mma(st[2 * i + 1], lo, x[2], x[3]);
+          mma(st[2 * i], hi, x[0], x[1]);
+          mma(st[2 * i + 1], hi, x[2], x[3]);
+        }
+      }
+    }
+    // the chunk's outputs as whole rows
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) stage_o[(i * 8 + t2 + (j & 1)) * SP + wid * 16 + g + (j >> 1) * 8] = pq[i][j];
+    __syncthreads();
+    const int t0 = chunk * CH, nt = min(CH, a.n - t0);
+    constexpr int LANES = VT / 8;  // per row, eight columns each
+#pragma unroll
+    for (int i = tid; i < CH * LANES; i += THREADS) {
+      const int t = i / LANES, c = (i - t * LANES) * 8;
+      const float4 x = *reinterpret_cast<const float4 *>(stage_o + t * SP + c);
+      const float4 y = *reinterpret_cast<const float4 *>(stage_o + t * SP + c + 4);
+      const long long r = (long long)b * a.n + t0 + t;
+      if (!s.normed) {
+        if (t < nt && c < cols) {
+          float *o = s.o + (r * a.heads + h) * a.vdim + vt + c;
+          *reinterpret_cast<float4 *>(o) = x;
+          *reinterpret_cast<float4 *>(o + 4) = y;
+        }
+        continue;
+      }
+      float q = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w + y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+#pragma unroll
+      for (int o = LANES / 2; o > 0; o >>= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
+      if (t >= nt || c >= cols) continue;
+      const float inv = 1.0f / sqrtf(q / s.count + s.eps);
+      const uint4 z = *reinterpret_cast<const uint4 *>(s.gate + r * s.in_ld + h * a.vdim + c);
+      const float4 w0 = *reinterpret_cast<const float4 *>(s.norm + c), w1 = *reinterpret_cast<const float4 *>(s.norm + c + 4);
+      *reinterpret_cast<uint4 *>(s.out + r * s.out_ld + h * a.vdim + c) =
+          make_uint4(pack(x.x * inv * w0.x * silu_f32(low_half(z.x)), x.y * inv * w0.y * silu_f32(high_half(z.x))),
+                     pack(x.z * inv * w0.z * silu_f32(low_half(z.y)), x.w * inv * w0.w * silu_f32(high_half(z.y))),
+                     pack(y.x * inv * w1.x * silu_f32(low_half(z.z)), y.y * inv * w1.y * silu_f32(high_half(z.z))),
+                     pack(y.z * inv * w1.z * silu_f32(low_half(z.w)), y.w * inv * w1.w * silu_f32(high_half(z.w))));
+    }
+    if (s.stages == 1 && chunk + 1 < a.chunks) load(chunk + 1);  // every warp is past this chunk's tiles
+  }
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int d = i * 8 + t2 + (j & 1), v = v0 + (j >> 1) * 8;
+      if (d < a.dim && v < a.vdim) S[(long long)d * a.vdim + v] = st[i][j];
+    }
+}
+
+struct Parts {
+  size_t mats, factors;
+};
+Parts parts(const DeltaMixer &m, long long rows, int streams) {
+  const size_t all = (size_t)(rows / CH + streams) * m.heads;  // however the rows are shared among the streams
+  return {all * 4 * MAT * 2, all * CH * 16};
+}
+
+constexpr size_t SMEM_LIMIT = 227 * 1024;
+
+}  // namespace
+
+bool delta_chunk_supports(const DeltaMixer &m) { return m.dim <= 256; }
+
+size_t delta_chunk_bytes(const DeltaMixer &m, long long rows, int streams) {
+  const Parts p = parts(m, rows, streams);
+  return p.mats + p.factors;
+}
+
+int launch_delta_chunks(const DeltaMixer &m, const void *conv, float *o, void *scratch, const RowBatch &b, bool *normed,
+                        cudaStream_t st) {
+  const Parts part = parts(m, b.rows(), b.streams);
+  bf16 *mats = static_cast<bf16 *>(scratch);
+  float4 *factors = reinterpret_cast<float4 *>(static_cast<char *>(scratch) + part.mats);
+  const bf16 *rows = static_cast<const bf16 *>(conv);
+  ChunkArgs c{};
+  c.heads = m.heads;
+  c.groups = m.groups;
+  c.dim = m.dim;
+  c.vdim = m.vdim;
+  c.channels = m.conv_channels();
+  c.n = b.n;
+  c.chunks = (b.n + CH - 1) / CH;
+  c.q_scale = 1.0f / sqrtf((float)m.true_dim);
+  c.a_log = m.a_log;
+  c.dt_bias = m.dt_bias;
+  c.ba = m.ba;
+  c.ba_ld = m.ba_ld;
+  const size_t prep_smem = (size_t)2 * CH * (m.dim + 8) * 2 + (size_t)2 * CH * TP * 4;
+  LB_CUDA(cudaFuncSetAttribute(delta_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem));
+  launch_pdl(delta_prepare_kernel, dim3((unsigned)c.chunks, (unsigned)m.groups, (unsigned)b.streams), dim3(PREP_THREADS),
+             prep_smem, st, g_pdl_enabled, c, rows, mats, factors);
+  ScanArgs s{};
+  s.c = c;
+  s.p0 = b.p0;
+  s.slot0 = b.slot0;
+  s.state = m.state;
+  s.o = o;
+  s.gate = static_cast<const bf16 *>(m.in) + c.channels;
+  s.in_ld = m.in_ld;
+  s.out_ld = m.out_ld;
+  s.count = (float)m.true_vdim;
+  s.eps = m.eps;
+  s.norm = m.norm;
+  s.out = static_cast<bf16 *>(m.out);
+  // the widest tile of value columns that still gives about half the SMs a CTA
+  const long long lanes = (long long)b.streams * m.heads;
+  int vt = m.dim > 128 ? 64 : 128;
+  while (vt > 32 && (vt / 2 >= m.vdim || lanes * ((m.vdim + vt - 1) / vt) < 74)) vt /= 2;
+  s.normed = vt >= m.vdim;
+  *normed = s.normed != 0;
+  auto scan = [&](auto kernel, int warps) {
+    const size_t stage = (size_t)stage_elems(m.dim, vt) * 2, extra = (size_t)CH * (vt + 4) * 4;
+    s.stages = 2 * stage + extra <= SMEM_LIMIT ? 2 : 1;
+    const size_t smem = s.stages * stage + extra;
+    LB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    launch_pdl(kernel, dim3((unsigned)(m.heads * ((m.vdim + vt - 1) / vt)), (unsigned)b.streams), dim3((unsigned)(warps * 32)),
+               smem, st, g_pdl_enabled, s, rows, (const bf16 *)mats, (const float4 *)factors);
+  };
+  if (m.dim <= 64) {
+    if (vt == 128) scan(delta_scan_kernel<8, 8, false>, 8);
+    else if (vt == 64) scan(delta_scan_kernel<8, 4, false>, 4);
+    else scan(delta_scan_kernel<8, 2, false>, 2);
+  } else if (m.dim <= 128) {
+    if (vt == 128) scan(delta_scan_kernel<16, 8, false>, 8);
+    else if (vt == 64) scan(delta_scan_kernel<16, 4, false>, 4);
+    else scan(delta_scan_kernel<16, 2, false>, 2);
+  } else {
+    if (vt == 64) scan(delta_scan_kernel<32, 4, true>, 4);
+    else scan(delta_scan_kernel<32, 2, true>, 2);
+  }
+  return 2;
+}
+
+}  // namespace lb

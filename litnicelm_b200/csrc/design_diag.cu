@@ -121,7 +121,7 @@ int litnice_b200_bf16_product_host(int32_t engine, const float *a, int32_t m, in
     p.n_half = n_half;
     p.half_out = dev.alloc((size_t)m * up8(n_half ? n_half : 1) * 2);
     p.half_ld = up8(n_half ? n_half : 1);
-    p.gelu = gelu;
+    p.act = gelu;
     p.float_ld = nf > 0 ? nf : 1;
     p.accumulate = accumulate;
     std::vector<float> part((size_t)m * (nf > 0 ? nf : 1));

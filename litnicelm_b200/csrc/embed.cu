@@ -127,10 +127,11 @@ __global__ void advance_state_kernel(LoopState *state) {
   state->step += 1;
 }
 
-// The rows of a batch (new positions only): x[r, :] = table[ids[slot, p]] + pos[p], in 32-bit.
+// The rows of a batch (new positions only): x[r, :] = table[ids[slot, p]] * scale + pos[p], in 32-bit
+// (pos == nullptr: no position vectors).
 template <typename T>
-__global__ void embed_rows_kernel(const T *__restrict__ table, const T *__restrict__ pos, const int *ids,
-                                  int ids_ld, const LoopState *state, int p0_host, int n, int slot0, int d, int vocab,
+__global__ void embed_rows_kernel(const T *__restrict__ table, const T *__restrict__ pos, float scale,
+                                  const int *ids, int ids_ld, const LoopState *state, int p0_host, int n, int slot0, int d, int vocab,
                                   float *x, DevErr *err) {
   pdl_launch_dependents();
   pdl_wait();
@@ -144,26 +145,25 @@ __global__ void embed_rows_kernel(const T *__restrict__ table, const T *__restri
     }
     id = 0;
   }
-  const T *tp = table + (long long)id * d, *pp = pos + (long long)p * d;
+  const T *tp = table + (long long)id * d, *pp = pos ? pos + (long long)p * d : nullptr;
   float *xp = x + ((long long)b * n + t) * d;
   if ((d & 3) == 0) {
-    for (int c = threadIdx.x * 4; c < d; c += blockDim.x * 4) {
-      float4 v;
+    auto load4 = [](const T *q) {
       if (sizeof(T) == 2) {  // two bfloat16 per word
-        const uint2 a = *reinterpret_cast<const uint2 *>(tp + c), q = *reinterpret_cast<const uint2 *>(pp + c);
-        v = make_float4(__uint_as_float(a.x << 16) + __uint_as_float(q.x << 16),
-                        __uint_as_float(a.x & 0xffff0000u) + __uint_as_float(q.x & 0xffff0000u),
-                        __uint_as_float(a.y << 16) + __uint_as_float(q.y << 16),
-                        __uint_as_float(a.y & 0xffff0000u) + __uint_as_float(q.y & 0xffff0000u));
-      } else {
-        const float4 a = *reinterpret_cast<const float4 *>(tp + c), q = *reinterpret_cast<const float4 *>(pp + c);
-        v = make_float4(a.x + q.x, a.y + q.y, a.z + q.z, a.w + q.w);
+        const uint2 a = *reinterpret_cast<const uint2 *>(q);
+        return make_float4(__uint_as_float(a.x << 16), __uint_as_float(a.x & 0xffff0000u), __uint_as_float(a.y << 16),
+                           __uint_as_float(a.y & 0xffff0000u));
       }
-      *reinterpret_cast<float4 *>(xp + c) = v;
+      return *reinterpret_cast<const float4 *>(q);
+    };
+    for (int c = threadIdx.x * 4; c < d; c += blockDim.x * 4) {
+      const float4 a = load4(tp + c), q = pp ? load4(pp + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      *reinterpret_cast<float4 *>(xp + c) =
+          make_float4(fmaf(a.x, scale, q.x), fmaf(a.y, scale, q.y), fmaf(a.z, scale, q.z), fmaf(a.w, scale, q.w));
     }
     return;
   }
-  for (int c = threadIdx.x; c < d; c += blockDim.x) xp[c] = (float)tp[c] + (float)pp[c];
+  for (int c = threadIdx.x; c < d; c += blockDim.x) xp[c] = fmaf((float)tp[c], scale, pp ? (float)pp[c] : 0.f);
 }
 
 }  // namespace
@@ -190,16 +190,16 @@ void launch_advance_state(LoopState *state, cudaStream_t st) {
   launch_pdl(advance_state_kernel, dim3(1), dim3(1), 0, st, g_pdl_enabled, state);
 }
 
-void launch_embed_rows(const void *table, const void *pos, Precision type, const RowBatch &b, int d, int vocab, float *x,
+void launch_embed_rows(const void *table, const void *pos, float scale, Precision type, const RowBatch &b, int d, int vocab, float *x,
                        cudaStream_t st, DevErr *err) {
   const dim3 grid((unsigned)b.n, (unsigned)b.streams);
   if (type == Precision::BF16)
     launch_pdl(embed_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, g_pdl_enabled,
-               static_cast<const __nv_bfloat16 *>(table), static_cast<const __nv_bfloat16 *>(pos), b.ids, b.ids_ld, b.state,
+               static_cast<const __nv_bfloat16 *>(table), static_cast<const __nv_bfloat16 *>(pos), scale, b.ids, b.ids_ld, b.state,
                b.p0, b.n, b.slot0, d, vocab, x, err);
   else
     launch_pdl(embed_rows_kernel<float>, grid, dim3(256), 0, st, g_pdl_enabled, static_cast<const float *>(table),
-               static_cast<const float *>(pos), b.ids, b.ids_ld, b.state, b.p0, b.n, b.slot0, d, vocab, x, err);
+               static_cast<const float *>(pos), scale, b.ids, b.ids_ld, b.state, b.p0, b.n, b.slot0, d, vocab, x, err);
 }
 
 }  // namespace lb

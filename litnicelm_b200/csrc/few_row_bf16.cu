@@ -9,6 +9,7 @@
 // of W per warp and row. Up to two products with inputs of their own share a launch. Where the columns
 // alone give too few CTAs, k is cut over the CTAs of a thread-block cluster, whose sums meet in the shared
 // memory of the rank that stores them (rank order, so results do not depend on scheduling).
+#include "activation.cuh"
 #include "model.cuh"
 #include "tc_ptx.cuh"
 
@@ -142,10 +143,7 @@ few_row_bf16_kernel(FewRowPair pair, int m, int ranks) {
     e_begin = min(TILE, (int)blockIdx.z * share);
     e_end = min(TILE, e_begin + share);
   }
-  for (int e = e_begin + threadIdx.x; e < e_end; e += FR_WARPS * 32) {
-    const int c = e & (FR_COLS - 1), row = e / FR_COLS;
-    const int col = n0 + c;
-    if (row >= m || col >= p.n) continue;
+  auto total = [&](int c, int row) {
     float v = 0.f;
     if (ranks > 1) {
       const unsigned at = smem_u32(&red[0][row >> 3][c][row & 7]);
@@ -154,9 +152,21 @@ few_row_bf16_kernel(FewRowPair pair, int m, int ranks) {
 #pragma unroll
       for (int q = 0; q < FR_WARPS; ++q) v += red[q][row >> 3][c][row & 7];
     }
+    return v;
+  };
+  for (int e = e_begin + threadIdx.x; e < e_end; e += FR_WARPS * 32) {
+    const int c = e & (FR_COLS - 1), row = e / FR_COLS;
+    const int col = n0 + c;
+    if (row >= m || col >= p.n) continue;
+    if (p.gated && col < p.n_half) {  // a pair's columns are neighbours in one share: its even one finishes both
+      if (c & 1) continue;
+      const float z = activate(total(c, row), p.act) * total(c + 1, row);
+      static_cast<bf16 *>(p.half_out)[(long long)row * p.half_ld + (col >> 1)] = __float2bfloat16_rn(z);
+      continue;
+    }
+    const float v = total(c, row);
     if (col < p.n_half) {
-      if (p.gelu) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
-      static_cast<bf16 *>(p.half_out)[(long long)row * p.half_ld + col] = __float2bfloat16_rn(v);
+      static_cast<bf16 *>(p.half_out)[(long long)row * p.half_ld + col] = __float2bfloat16_rn(activate(v, p.act));
     } else {
       float *o = p.float_out + (long long)row * p.float_ld + (col - p.n_half);
       *o = p.accumulate ? *o + v : v;

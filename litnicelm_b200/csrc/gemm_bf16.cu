@@ -10,6 +10,7 @@
 // Rows and columns outside the operands load as zeros (k need not be a multiple of 64) and are not
 // stored. Every mbarrier wait is bounded; a wait that runs out sets the error word and ends the kernel
 // after its copies have landed and tensor memory is freed. No clusters, no multicast.
+#include "activation.cuh"
 #include "model.cuh"
 #include "gemm_tc.cuh"
 #include "tc_ptx.cuh"
@@ -194,13 +195,12 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
           const int rr = i * 4 + sub, row = row0 + rr;
           if (row >= m || col >= p.n) continue;
           float4 v = *reinterpret_cast<const float4 *>(patch + rr * GB_PATCH_LD + c4);
-          if (whole && to_half && half_vec) {
-            if (p.gelu) {
-              v.x = 0.5f * v.x * (1.0f + erff(v.x * 0.70710678118654752f));
-              v.y = 0.5f * v.y * (1.0f + erff(v.y * 0.70710678118654752f));
-              v.z = 0.5f * v.z * (1.0f + erff(v.z * 0.70710678118654752f));
-              v.w = 0.5f * v.w * (1.0f + erff(v.w * 0.70710678118654752f));
-            }
+          if (whole && to_half && p.gated) {  // two pairs
+            const __nv_bfloat162 a = __floats2bfloat162_rn(activate(v.x, p.act) * v.y, activate(v.z, p.act) * v.w);
+            *reinterpret_cast<__nv_bfloat162 *>(static_cast<bf16 *>(p.half_out) + (long long)row * p.half_ld + (col >> 1)) = a;
+          } else if (whole && to_half && half_vec) {
+            if (p.act != ACT_NONE)
+              v = make_float4(activate(v.x, p.act), activate(v.y, p.act), activate(v.z, p.act), activate(v.w, p.act));
             const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
             uint2 o;
             o.x = *reinterpret_cast<const unsigned *>(&a);
@@ -219,8 +219,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
             for (int j = 0; j < 4; ++j) {
               if (col + j >= p.n) continue;
               if (col + j < p.n_half) {
-                const float z = p.gelu ? 0.5f * e[j] * (1.0f + erff(e[j] * 0.70710678118654752f)) : e[j];
-                static_cast<bf16 *>(p.half_out)[(long long)row * p.half_ld + col + j] = __float2bfloat16_rn(z);
+                if (p.gated) {
+                  if ((j & 1) == 0)  // n_half is even
+                    static_cast<bf16 *>(p.half_out)[(long long)row * p.half_ld + ((col + j) >> 1)] =
+                        __float2bfloat16_rn(activate(e[j], p.act) * e[j + 1]);
+                } else {
+                  static_cast<bf16 *>(p.half_out)[(long long)row * p.half_ld + col + j] =
+                      __float2bfloat16_rn(activate(e[j], p.act));
+                }
               } else {
                 float *o = p.float_out + (long long)row * p.float_ld + (col + j - p.n_half);
                 *o = p.accumulate ? *o + e[j] : e[j];
@@ -268,6 +274,7 @@ void launch_bn(const Bf16Product &p, int m, cudaStream_t st, DevErr *err) {
 
 void launch_gemm_bf16(const Bf16Product &p, int m, cudaStream_t st, DevErr *err) {
   if (m < 1 || p.n < 1 || p.k < 1) throw std::invalid_argument("launch_gemm_bf16: empty product");
+  if (p.gated && ((p.n_half | p.half_ld) & 1) != 0) throw std::invalid_argument("launch_gemm_bf16: a gated product needs pairs");
   // the widest tile that still gives most SMs one
   const long long mt = (m + TC_BM - 1) / TC_BM;
   const long long sms = device_sms();

@@ -8,7 +8,7 @@
 // latents once for all heads and expands no key or value.
 //
 //   latent_store_kernel          RMS norm of the new rows' W_dkv h into the cache, and the window's rows
-//                                side by side for the expanding kernels (latent_attention_tc.cu)
+//                                side by side for the expanding kernels (prefill_attention_tc.cu)
 //   latent_attention_rows_kernel any size, one CTA per row and head, float or bfloat16 storage
 //   latent_query / latent_chunk / latent_join   few rows on bfloat16: the absorbed query per head (and the
 //                                new latents into the cache, by CTAs of their own); splits of the window

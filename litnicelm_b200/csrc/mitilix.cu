@@ -16,7 +16,7 @@
 //               latents for the tensor-core attention (V directly transposed, as W_uv c^T)
 // 32-bit runs the framework's float products and the CUDA-core attention.
 #include "model.cuh"
-#include "gemm_tc.cuh"
+#include "model_common.cuh"
 
 #include <cmath>
 #include <cstring>
@@ -24,44 +24,6 @@
 namespace lb {
 
 namespace {
-
-int up8(int v) { return (v + 7) & ~7; }
-int up16(int v) { return (v + 15) & ~15; }
-
-struct DevBuf {
-  void *p = nullptr;
-  size_t bytes = 0;
-  DevBuf() = default;
-  DevBuf(const DevBuf &) = delete;
-  DevBuf &operator=(const DevBuf &) = delete;
-  DevBuf(DevBuf &&o) noexcept : p(o.p), bytes(o.bytes) {
-    o.p = nullptr;
-    o.bytes = 0;
-  }
-  ~DevBuf() {
-    if (p) cudaFree(p);
-  }
-  // At least `need` bytes, zeroed when new; true when the buffer moved (its content is gone).
-  bool ensure(size_t need, cudaStream_t st) {
-    if (need <= bytes) return false;
-    if (p) {
-      LB_CUDA(cudaStreamSynchronize(st));
-      cudaFree(p);
-      p = nullptr;
-      bytes = 0;
-    }
-    need = (need + 255) & ~(size_t)255;
-    if (cudaMalloc(&p, need) != cudaSuccess) {
-      p = nullptr;
-      (void)cudaGetLastError();
-      throw std::bad_alloc();
-    }
-    bytes = need;
-    LB_CUDA(cudaMemsetAsync(p, 0, need, st));
-    return true;
-  }
-  float *f() const { return static_cast<float *>(p); }
-};
 
 struct Layer {
   int heads = 0, dim = 0, vdim = 0, rank = 0, window = 0, kv_from = -1, ff = 0;
@@ -76,17 +38,6 @@ struct Layer {
   int o_cols() const { return heads * vdim; }
   bool own() const { return kv_from < 0; }
 };
-
-MatView dense(const float *p, long long rows, long long cols) {
-  MatView v{};
-  v.data = reinterpret_cast<char *>(const_cast<float *>(p));
-  v.batch = 1;
-  v.rows = rows;
-  v.cols = cols;
-  v.rs = cols * 4;
-  v.cs = 4;
-  return v;
-}
 
 class Mitilix final : public DecoderModel {
  public:
@@ -233,10 +184,10 @@ class Mitilix final : public DecoderModel {
       const int ns = streams > slots_ ? streams : slots_, nc = cap > cap_ ? cap : cap_;
       for (Layer &l : layers_) {
         const size_t hist = (size_t)(taps_ - 1) * width_ * 4;
-        if (ns > slots_ && hist > 0) grow(l.history, hist, slots_, hist, ns, hist, st);
+        if (ns > slots_ && hist > 0) l.history.grow(hist, slots_, hist, ns, hist, st);
         if (!l.own()) continue;
         const size_t row = (size_t)cache_ld(l) * es;
-        grow(l.cache, row * cap_, slots_, row * cap_, ns, row * nc, st);
+        l.cache.grow(row * cap_, slots_, row * cap_, ns, row * nc, st);
       }
       slots_ = ns;
       cap_ = nc;
@@ -276,7 +227,7 @@ class Mitilix final : public DecoderModel {
 
   int enqueue_rows(const RowBatch &b, cudaStream_t st, DevErr *err) override {
     launches_ = 0;
-    launch_embed_rows(embed_.p, pos_.p, prec_, b, width_, vocab_, x_.f(), st, err);
+    launch_embed_rows(embed_.p, pos_.p, 1.0f, prec_, b, width_, vocab_, x_.f(), st, err);
     ++launches_;
     packed_from_ = packed_first_ = -1;
     for (size_t i = 0; i < layers_.size(); ++i) {
@@ -290,7 +241,7 @@ class Mitilix final : public DecoderModel {
                    DevErr *err) override {
     launches_ = 0;
     const int ld = prec_ == Precision::BF16 ? up8(width_) : width_;
-    launch_rms_rows(x_.f(), width_, final_gain_, eps_, rows_dev, n_rows, b.n, xl_.p, ld, prec_, st);
+    launch_rms_rows(x_.f(), width_, RmsWeight{nullptr, final_gain_}, eps_, rows_dev, n_rows, b.n, xl_.p, ld, prec_, st);
     ++launches_;
     if (prec_ == Precision::BF16) {
       Bf16Product p;
@@ -311,17 +262,6 @@ class Mitilix final : public DecoderModel {
 
  private:
   int cache_ld(const Layer &l) const { return prec_ == Precision::BF16 ? up8(l.rank) : (l.rank + 3) & ~3; }
-
-  // A [slots][bytes] buffer to more or longer slots, what it holds kept.
-  void grow(DevBuf &buf, size_t old_bytes, int old_slots, size_t old_pitch, int slots, size_t pitch, cudaStream_t st) {
-    DevBuf next;
-    next.ensure(pitch * slots, st);
-    if (buf.p && old_bytes > 0 && old_slots > 0)
-      LB_CUDA(cudaMemcpy2DAsync(next.p, pitch, buf.p, old_pitch, old_bytes, (size_t)old_slots, cudaMemcpyDeviceToDevice, st));
-    LB_CUDA(cudaStreamSynchronize(st));
-    std::swap(buf.p, next.p);
-    std::swap(buf.bytes, next.bytes);
-  }
 
   const Layer &source(int i) const {
     const Layer &l = layers_[(size_t)i];
@@ -351,13 +291,7 @@ class Mitilix final : public DecoderModel {
   }
 
   void product_bf16(const Bf16Product *p, int count, int m, cudaStream_t st, DevErr *err) {
-    if (m <= FEW_ROWS_MAX) {
-      launch_few_row_bf16(p, count, m, st);
-      ++launches_;
-      return;
-    }
-    for (int i = 0; i < count; ++i) launch_gemm_bf16(p[i], m, st, err);
-    launches_ += count;
+    launches_ += products_bf16(p, count, m, st, err);
   }
 
   void layer_bf16(int i, const RowBatch &b, cudaStream_t st, DevErr *err) {
@@ -383,7 +317,7 @@ class Mitilix final : public DecoderModel {
     in[1].w = l.up.p;
     in[1].k = D;
     in[1].n = in[1].n_half = l.ff;
-    in[1].gelu = 1;
+    in[1].act = ACT_GELU_ERF;
     in[1].half_out = static_cast<uint16_t *>(mix_.p) + O8;
     in[1].half_ld = mix_ld;
     product_bf16(in, l.ff ? 2 : 1, m, st, err);
@@ -451,17 +385,9 @@ class Mitilix final : public DecoderModel {
     product_bf16(&out, 1, m, st, err);
   }
 
-  // out[m, n] = a[m, k] w[k, n] (+ residual) on the float products of the framework.
   void product_f32(const float *a, int m, int k, const float *w, int n, const float *residual, float *out,
                    cudaStream_t st, DevErr *err) {
-    if (m <= 8) {
-      launches_ += launch_gemv(a, m, w, k, n, nullptr, out, scratch_.f(), st, err, residual);
-      return;
-    }
-    GemmEpilogue ep;
-    ep.residual = residual;
-    launch_gemm_simt(dense(a, m, k), dense(w, k, n), dense(out, m, n), m, n, k, ep, st);
-    ++launches_;
+    launches_ += lb::product_f32(a, m, k, w, n, residual, out, scratch_.f(), st, err);
   }
 
   void layer_f32(int i, const RowBatch &b, cudaStream_t st, DevErr *err) {
@@ -482,7 +408,7 @@ class Mitilix final : public DecoderModel {
     product_f32(mix_.f(), m, l.o_cols(), l.o_t.f(), D, x_.f(), x_.f(), st, err);
     if (l.ff) {
       product_f32(a2_.f(), m, D, l.up_t.f(), l.ff, nullptr, hidden_.f(), st, err);
-      launch_gelu_f32(hidden_.f(), (long long)m * l.ff, st);
+      launch_activation_f32(hidden_.f(), nullptr, (long long)m * l.ff, ACT_GELU_ERF, st);
       ++launches_;
       product_f32(hidden_.f(), m, l.ff, l.down_t.f(), D, x_.f(), x_.f(), st, err);
     }

@@ -67,6 +67,7 @@ class DecoderModel {
   virtual int n_layers() const = 0;
   virtual int width() const = 0;
   virtual int vocab() const = 0;
+  // Positions the design has vectors for; 0: no bound of its own.
   virtual int max_positions() const = 0;
   virtual void load(const TensorFile &file, cudaStream_t st, DevErr *err) = 0;
   // Room for `streams` slots of `cap` positions each (what the slots hold is kept) and for steps of
@@ -95,8 +96,8 @@ std::string read_text_file(const std::string &path);
 // Inside these kernels only weights are __restrict__ const: such loads count as invariant and may be
 // scheduled ahead of the wait for the preceding kernel (pdl_wait), which wrote every other input.
 
-// embed.cu: x[r, :] = table[ids] + pos[p] for the rows of a batch; tables bfloat16 or float.
-void launch_embed_rows(const void *table, const void *pos, Precision type, const RowBatch &b, int d, int vocab, float *x,
+// embed.cu: x[r, :] = table[ids] * scale + pos[p] for the rows of a batch (pos may be null); tables bfloat16 or float.
+void launch_embed_rows(const void *table, const void *pos, float scale, Precision type, const RowBatch &b, int d, int vocab, float *x,
                        cudaStream_t st, DevErr *err);
 
 // canon.cu: h = x / sqrt(mean(x^2) + eps) * gain (one gain for all coordinates), then for each of up
@@ -109,8 +110,14 @@ struct CanonConv {
 };
 void launch_rms_canon(const float *x, int d, float gain, float eps, int taps, float *history, const CanonConv *conv,
                       int n_conv, Precision type, const RowBatch &b, cudaStream_t st);
-// canon.cu: the scalar-gain RMS norm alone, of listed rows (rows_dev) or of every stream's last row.
-void launch_rms_rows(const float *x, int d, float gain, float eps, const int *rows_dev, int n_rows, int n_per_stream,
+// Gain of an RMS norm: base + w[c], or base alone for all coordinates. Weights stored around zero take base 1.
+struct RmsWeight {
+  const float *w = nullptr;
+  float base = 0.f;
+  __device__ __forceinline__ float at(int c) const { return w ? base + w[c] : base; }
+};
+// canon.cu: RMS norm of listed rows (rows_dev) or of every stream's last row.
+void launch_rms_rows(const float *x, int d, const RmsWeight &weight, float eps, const int *rows_dev, int n_rows, int n_per_stream,
                      void *out, int ld, Precision type, cudaStream_t st);
 
 // latent_attention.cu. A latent cache is [slots][cap][ld] (bfloat16 or float): one compressed row per
@@ -156,12 +163,97 @@ size_t latent_decode_scratch_floats(int heads, int rank, int window, int s_cap, 
 int launch_latent_decode(const LatentAttention &a, const LatentFresh &fresh, float *scratch, const RowBatch &b,
                          cudaStream_t st);
 
-// latent_attention_tc.cu: many new rows on bfloat16 tensor cores over expanded keys and values:
+// prefill_attention_tc.cu: many new rows on bfloat16 tensor cores over expanded keys and values:
 // k [streams * key_rows, k_ld] row-major, vt [heads * vdim, vt_ld] with one column per key; key row j
 // of a stream is position first + j.
 bool latent_prefill_supports(int dim, int vdim);
 void launch_latent_prefill(const LatentAttention &a, const void *k, int k_ld, const void *vt, int vt_ld, int key_rows,
                            int first, const RowBatch &b, cudaStream_t st, DevErr *err);
+
+// residual_norm.cu: the norms around a sublayer in one pass over the residual stream x [rows, d]:
+//   x <- x + rms(y) * after      (y == nullptr: x stays)
+//   h  = rms(x) * before         (h == nullptr: not asked for)
+// y [rows, d] float, h [rows, h_ld] bfloat16 or float.
+void launch_residual_norm(float *x, const float *y, const RmsWeight &after, void *h, int h_ld, const RmsWeight &before, int d,
+                          long long rows, float eps, Precision type, cudaStream_t st);
+
+// Which keys a query at position p sees besides j <= p: the last `size` positions, or those of its own chunk of
+// `size` positions counted from 0.
+enum class SpanKind : int { WINDOW = 0, CHUNK = 1 };
+struct KeySpan {
+  SpanKind kind = SpanKind::WINDOW;
+  int size = 1;
+  // First key of the query at p (may be negative for a window).
+  __host__ __device__ __forceinline__ int first(int p) const {
+    return kind == SpanKind::CHUNK ? p - p % size : p - size + 1;
+  }
+};
+
+// Rotary positions: dimension i of a head turns together with i + dims / 2 by p * turns[i] half turns (turns: angle
+// per position over pi, double), both results times `amplitude`; dimensions from dims on pass.
+struct Rotation {
+  int dims = 0;
+  const double *turns = nullptr;  // [dims / 2], device
+  float amplitude = 1.f;
+};
+
+// grouped_attention.cu: softmax attention whose query heads share key and value heads. Heads are padded to
+// multiples of 16 elements with zeros everywhere (dim, vdim: padded sizes); caches are [slots][cap][groups * dim] and
+// [slots][cap][groups * vdim].
+struct GroupedAttention {
+  int heads, groups, dim, vdim;
+  float scale;
+  KeySpan span;
+  const void *q;   // [rows, q_ld]
+  int q_ld;
+  void *k_cache, *v_cache;
+  int cap, slots;
+  void *out;       // [rows, out_ld], heads side by side, vdim each
+  int out_ld;
+};
+// Queries and keys: RMS norm over all heads of a row at once (weights [heads * dim] and [groups * dim], true_dim of each
+// dim counted), rotation, queries to q, keys and values to the caches. src rows: [queries | keys | values], ld apart.
+void launch_qk_norm_rotate(const void *src, int ld, const float *q_weight, const float *k_weight, float eps, int true_dim,
+                           const Rotation &rot, const GroupedAttention &a, void *q, Precision type, const RowBatch &b,
+                           cudaStream_t st);
+// Any number of rows, 32-bit arithmetic on CUDA cores; keys split over a cluster's CTAs where rows are few.
+void launch_grouped_attention_rows(const GroupedAttention &a, Precision type, const RowBatch &b, cudaStream_t st);
+// prefill_attention_tc.cu: many new rows on bfloat16 tensor cores, keys and values as they lie in the caches.
+bool grouped_prefill_supports(int dim, int vdim);
+void launch_grouped_prefill(const GroupedAttention &a, const RowBatch &b, cudaStream_t st, DevErr *err);
+
+// delta.cu, delta_chunk.cu: the gated delta rule. Per head, with unit vectors q, k and the state S [dim, vdim]:
+//   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+// after a short causal convolution and SiLU on q, k and v; o is normalised per head and gated. dim and vdim are
+// padded to multiples of 16 with zeros. Columns of a projected row: [q | k | v | gate], groups * dim twice and
+// heads * vdim twice, and beside them [beta | decay] in float.
+struct DeltaMixer {
+  int heads, groups, dim, vdim;   // padded sizes
+  int true_dim, true_vdim;        // q scale, and what the output's norm counts
+  int taps;
+  float eps;
+  const float *conv;              // [taps][conv_channels]
+  const float *a_log, *dt_bias;   // [heads]
+  const float *norm;              // [vdim]
+  float *state;                   // [slots][heads][dim][vdim]
+  void *history;                  // [slots][taps][conv_channels]: inputs of the convolution, position % taps
+  const void *in;                 // [rows, in_ld] bfloat16 or float
+  int in_ld;
+  const float *ba;                // [rows, ba_ld]
+  int ba_ld;
+  void *out;                      // [rows, out_ld]
+  int out_ld;
+  int conv_channels() const { return 2 * groups * dim + heads * vdim; }
+};
+// What launch_delta needs besides: convolved rows [rows][conv_channels], outputs before the norm
+// [rows][heads * vdim] float, and the chunked form's matrices.
+size_t delta_scratch_bytes(const DeltaMixer &m, long long rows, int streams, Precision type);
+// The new rows' recurrence and gated norm, state and history advanced; returns the kernels launched.
+int launch_delta(const DeltaMixer &m, void *scratch, Precision type, const RowBatch &b, cudaStream_t st);
+bool delta_supports(int dim, int vdim);
+
+// Activations of the products and of launch_activation_f32: GELU in its error-function and tanh forms.
+enum Activation : int { ACT_NONE = 0, ACT_GELU_ERF = 1, ACT_GELU_TANH = 2 };
 
 // Matrix products on bfloat16 with 32-bit accumulation: C[m, n] = A[m, k] W[n, k]^T.
 struct Bf16Product {
@@ -170,12 +262,14 @@ struct Bf16Product {
   const void *w = nullptr;  // [n, w_ld] bfloat16; w_ld % 8 == 0
   int w_ld = 0;
   int n = 0, k = 0;
-  // result: columns below n_half go to half_out (bfloat16, through GELU when gelu is set), the others
-  // to float_out[:, column - n_half] (added to what it holds when accumulate is set)
+  // result: columns below n_half go to half_out (bfloat16, through the activation), the others to
+  // float_out[:, column - n_half] (added to what it holds when accumulate is set)
   int n_half = 0;
   void *half_out = nullptr;
   int half_ld = 0;
-  int gelu = 0;
+  int act = ACT_NONE;
+  // gated: columns 2 j and 2 j + 1 below n_half are a gate and its factor, half_out[:, j] = act(c_2j) * c_2j+1
+  int gated = 0;
   float *float_out = nullptr;
   int float_ld = 0;
   int accumulate = 0;
@@ -192,7 +286,16 @@ void launch_pack_bf16(const void *src, long long rows, int cols, void *dst, long
 // The same to float, optionally transposed: dst[c * ld + r].
 void launch_expand_f32(const void *src, long long rows, int cols, float *dst, long long ld, bool transpose,
                        cudaStream_t st, DevErr *err);
-// x <- gelu(x) (erf form) on a dense float array.
-void launch_gelu_f32(float *x, long long count, cudaStream_t st);
+// dst[offset + r' * row_stride + c' * col_stride] = src[r * cols + c] (bfloat16, or float for Precision::F32) with
+// r' = r / row_group * row_pad + r % row_group, and c' alike (group 0: r' = r): rows or columns in padded groups,
+// transposed, interleaved.
+struct WeightPlace {
+  long long offset = 0, row_stride = 0, col_stride = 1;
+  int row_group = 0, row_pad = 0, col_group = 0, col_pad = 0;
+};
+void launch_place(const void *src, long long rows, int cols, void *dst, Precision type, const WeightPlace &at,
+                  cudaStream_t st, DevErr *err);
+// x <- act(x), or act(x) * factor, on dense float arrays.
+void launch_activation_f32(float *x, const float *factor, long long count, Activation act, cudaStream_t st);
 
 }  // namespace lb

@@ -7,6 +7,7 @@
 
 namespace lb {
 
+std::unique_ptr<DecoderModel> make_gobesun(const Json &config, Precision precision);
 std::unique_ptr<DecoderModel> make_mitilix(const Json &config, Precision precision);
 
 namespace {
@@ -17,6 +18,7 @@ struct Design {
 };
 const Design kDesigns[] = {
     {"Mitilix", &make_mitilix},
+    {"Gobesun", &make_gobesun},
 };
 
 }  // namespace

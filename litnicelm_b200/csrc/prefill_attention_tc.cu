@@ -1,12 +1,17 @@
-// Sliding-window attention of many new rows on the sm_100a tensor cores (tcgen05 + TMEM + TMA),
-// bfloat16 operands and 32-bit scores, weights and sums, over keys and values expanded from the
-// window's latents (k row-major, v transposed: both K-major operands as they lie).
+// Attention of many new rows on the sm_100a tensor cores (tcgen05 + TMEM + TMA), bfloat16 operands and
+// 32-bit scores, weights and sums; a query sees the keys of its KeySpan (a sliding window or its chunk).
+// Keys are row-major. Values come in one of two forms:
+//   V_ROWS false   transposed (one row per value column, one column per key): a K-major operand as it
+//                  lies; keys and values expanded from a window's latents
+//   V_ROWS true    row-major like the keys, straight from a cache: an operand with its columns
+//                  contiguous (64 columns per slab, eight keys per swizzle atom); query heads may share
+//                  key and value heads
 //
-// One CTA per 128 queries of one head and stream walks the key tiles (128 keys) its window touches:
+// One CTA per 128 queries of one head and stream walks the key tiles (128 keys) its rows see:
 //   S = Q K^T      A = Q tile, B = K tile, into 128 columns of tensor memory
 //   P              four warps, one thread per query row: maximum, weights 2^(s - m), stored as
 //                  bfloat16 pairs over the scores' own columns (two keys per column)
-//   O += P V       A = P from tensor memory, B = V^T tile
+//   O += P V       A = P from tensor memory, B = V tile
 // The reference maximum of a row follows its running maximum only when that has grown by more than
 // 2^8: until then the accumulated O and the sum stay as they are (weights up to 2^8 are exact enough
 // in either format), so most tiles need no pass over O.
@@ -39,24 +44,30 @@ __device__ __forceinline__ float lp_exp2(float x) {
 
 struct LpArgs {
   int dim, vdim, n, n_rows;   // n new rows per stream
-  int q0_rel;                 // position of a stream's first new row minus `first`: its place among the key rows
+  int group;                  // query heads per key head
+  int pos0;                   // position of a stream's first new row
+  int first;                  // position of a stream's key row 0
+  int key_base;               // key row 0 of stream 0 in the maps
   int key_rows, n_keys;       // key rows per stream as laid out, and those that exist
-  int window;
+  KeySpan span;
   float factor;               // scale * log2(e)
   bf16 *out;
   int out_ld;
 };
 
+template <bool V_ROWS>
 __global__ void __launch_bounds__(LP_THREADS, 2)
-latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                      const __grid_constant__ CUtensorMap map_vt, LpArgs a, DevErr *err) {
+prefill_attention_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                      const __grid_constant__ CUtensorMap map_v, LpArgs a, DevErr *err) {
   extern __shared__ unsigned char smem_raw[];
   const unsigned base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   unsigned char *base_ptr = smem_raw + (base - smem_u32(smem_raw));
   const int dslabs = (a.dim + 63) >> 6;
   const unsigned q_off = base, k_off = base + (unsigned)(dslabs * LP_SLAB), v_off = k_off + (unsigned)(dslabs * LP_SLAB);
-  const unsigned vslab = (unsigned)a.vdim * 128u;
-  const unsigned bars = v_off + 2u * vslab;
+  // the V tile: two slabs of 64 keys by vdim rows, or slabs of 64 columns by 128 key rows
+  const unsigned vslab = V_ROWS ? (unsigned)LP_SLAB : (unsigned)a.vdim * 128u;
+  const int vslabs = V_ROWS ? (a.vdim + 63) >> 6 : 2;
+  const unsigned bars = v_off + (unsigned)vslabs * vslab;
   unsigned char *bar_ptr = base_ptr + (bars - base);
   const unsigned q_full = bars, k_full = bars + 8, v_full = bars + 16, k_free = bars + 24, s_full = bars + 32,
                  p_ready = bars + 40, o_full = bars + 48;
@@ -65,9 +76,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, b = blockIdx.z, t0 = blockIdx.x * LP_BQ;
   const unsigned cols = a.vdim <= 128 ? 256u : 512u;
-  // key rows this tile of queries sees: [lo, hi], tiles from lo rounded down to a 16-byte boundary of V^T's rows
-  const int qrel0 = a.q0_rel + t0;
-  const int lo = max(0, qrel0 - a.window + 1) & ~7;
+  // key rows this tile of queries sees: [lo, hi]; lo rounded down to a 16-byte boundary of V^T's rows
+  const int qrel0 = a.pos0 - a.first + t0;
+  const int lo = max(0, a.span.first(a.pos0 + t0) - a.first) & ~(V_ROWS ? 0 : 7);
+  const int kcol = h / a.group * a.dim, vcol = h / a.group * a.vdim, key0 = a.key_base + b * a.key_rows;
   const int hi = min(qrel0 + LP_BQ, a.n_keys) - 1;
   const int tiles = (hi - lo) / LP_BK + 1;
 
@@ -106,15 +118,18 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       if (lane == 0) {
         mbar_expect_tx(k_full, (unsigned)(dslabs * LP_SLAB));
         for (int s = 0; s < dslabs; ++s)
-          tma_load_2d(k_off + s * LP_SLAB, &map_k, h * a.dim + s * 64, b * a.key_rows + j0, k_full);
+          tma_load_2d(k_off + s * LP_SLAB, &map_k, kcol + s * 64, key0 + j0, k_full);
       }
       ++k_loads;
       if (i > 0) ok = mbar_wait(o_full, (unsigned)(i - 1) & 1u, abort_flag, err, 22);  // P V has read the V tile
       __syncwarp();
       if (!ok) break;
       if (lane == 0) {
-        mbar_expect_tx(v_full, 2u * vslab);
-        for (int s = 0; s < 2; ++s) tma_load_2d(v_off + s * vslab, &map_vt, b * a.key_rows + j0 + s * 64, h * a.vdim, v_full);
+        mbar_expect_tx(v_full, (unsigned)vslabs * vslab);
+        for (int s = 0; s < vslabs; ++s) {
+          if (V_ROWS) tma_load_2d(v_off + s * vslab, &map_v, vcol + s * 64, key0 + j0, v_full);
+          else tma_load_2d(v_off + s * vslab, &map_v, key0 + j0 + s * 64, vcol, v_full);
+        }
       }
       ++v_loads;
       __syncwarp();
@@ -126,7 +141,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       while (v_loads > 0 && !mbar_try_wait(v_full, (unsigned)(v_loads - 1) & 1u) && global_timer() < limit) {}
     }
   } else if (warp == 1) {
-    const unsigned idesc_s = umma_idesc_bf16(LP_BK), idesc_o = umma_idesc_bf16(a.vdim);
+    const unsigned idesc_s = umma_idesc_bf16(LP_BK), idesc_o = umma_idesc_bf16(a.vdim) | (V_ROWS ? UMMA_B_MN_MAJOR : 0u);
     const int ksteps = a.dim >> 4;
     bool ok = mbar_wait(q_full, 0, abort_flag, err, 23);
     __syncwarp();
@@ -158,8 +173,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
         for (int ks = 0; ks < LP_BK / 16; ++ks)
           tc_mma_f16_ts(tmem_o, tmem_s + (unsigned)(ks * 8),
-                        umma_desc_k128(v_off + (unsigned)(ks >> 2) * vslab) + (unsigned long long)((ks & 3) * 2), idesc_o,
-                        (i | ks) ? 1u : 0u);
+                        V_ROWS ? umma_desc_mn128(v_off + (unsigned)(ks * 16 * 128), vslab)
+                               : umma_desc_k128(v_off + (unsigned)(ks >> 2) * vslab) + (unsigned long long)((ks & 3) * 2),
+                        idesc_o, (i | ks) ? 1u : 0u);
         tc_commit(o_full);
       }
       __syncwarp();
@@ -174,7 +190,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const int q = warp & 3;
     const unsigned lanes = (unsigned)(q * 32) << 16;
     const int t = t0 + q * 32 + lane;     // this thread's row of the portion
-    const int qrel = a.q0_rel + t;        // its own key row
+    const int qrel = qrel0 + q * 32 + lane;  // its own key row
+    const int row_lo = a.span.first(a.pos0 + t) - a.first, warp_lo = a.span.first(a.pos0 + t0 + q * 32 + 31) - a.first;
     const int wq0 = qrel0 + q * 32;       // the warp's first row
     float m = LP_NEG, l = 0.f;
     bool ok = true;
@@ -183,9 +200,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       ok = mbar_wait_warp(s_full, (unsigned)i & 1u, abort_flag, err, 27);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      // keys j0 + c seen by this row: c in [c_lo, c_hi]; whole tiles inside every row's window need no mask
-      const int c_hi = qrel - j0, c_lo = qrel - a.window + 1 - j0;
-      const bool inside = wq0 - j0 >= LP_BK - 1 && wq0 + 31 - a.window + 1 - j0 <= 0;
+      // keys j0 + c seen by this row: c in [c_lo, c_hi]; whole tiles inside every row's span need no mask
+      const int c_hi = qrel - j0, c_lo = row_lo - j0;
+      const bool inside = wq0 - j0 >= LP_BK - 1 && warp_lo <= j0;
       // the row's scores stay in registers; independent chains for the maximum and the sum
       float s[LP_BK];
       {
@@ -277,15 +294,28 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   }
 }
 
-size_t lp_smem(int dim, int vdim) {
-  return (size_t)2 * ((dim + 63) / 64) * LP_SLAB + (size_t)2 * vdim * 128 + 128 + 1024;
+size_t lp_smem(int dim, int vdim, bool v_rows) {
+  return (size_t)2 * ((dim + 63) / 64) * LP_SLAB + (v_rows ? (size_t)((vdim + 63) / 64) * LP_SLAB : (size_t)2 * vdim * 128) +
+         128 + 1024;
+}
+
+bool lp_sizes(int dim, int vdim) {
+  return dim % 16 == 0 && vdim % 16 == 0 && dim >= 16 && vdim >= 16 && dim <= 256 && vdim <= 256;
+}
+
+template <bool V_ROWS>
+void lp_launch(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const LpArgs &a, int heads, int streams,
+               cudaStream_t st, DevErr *err) {
+  const size_t smem = lp_smem(a.dim, a.vdim, V_ROWS);
+  LB_CUDA(cudaFuncSetAttribute(prefill_attention_kernel<V_ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  launch_pdl(prefill_attention_kernel<V_ROWS>, dim3((unsigned)((a.n + LP_BQ - 1) / LP_BQ), (unsigned)heads, (unsigned)streams),
+             dim3(LP_THREADS), smem, st, false, mq, mk, mv, a, err);
 }
 
 }  // namespace
 
-bool latent_prefill_supports(int dim, int vdim) {
-  return dim % 16 == 0 && vdim % 16 == 0 && dim >= 16 && vdim >= 16 && dim <= 256 && vdim <= 256;
-}
+bool latent_prefill_supports(int dim, int vdim) { return lp_sizes(dim, vdim); }
+bool grouped_prefill_supports(int dim, int vdim) { return lp_sizes(dim, vdim); }
 
 void launch_latent_prefill(const LatentAttention &at, const void *k, int k_ld, const void *vt, int vt_ld, int key_rows,
                            int first, const RowBatch &b, cudaStream_t st, DevErr *err) {
@@ -293,10 +323,12 @@ void launch_latent_prefill(const LatentAttention &at, const void *k, int k_ld, c
   a.dim = at.dim;
   a.vdim = at.vdim;
   a.n = b.n;
-  a.q0_rel = b.p0 - first;
+  a.group = 1;
+  a.pos0 = b.p0;
+  a.first = first;
   a.key_rows = key_rows;
   a.n_keys = b.p0 + b.n - first;
-  a.window = at.window;
+  a.span.size = at.window;
   a.factor = at.scale * 1.4426950408889634f;
   a.out = static_cast<bf16 *>(at.out);
   a.out_ld = at.out_ld;
@@ -306,10 +338,31 @@ void launch_latent_prefill(const LatentAttention &at, const void *k, int k_ld, c
   tc_make_map_bf16(&mq, at.q, (unsigned long long)b.rows(), hd, (unsigned long long)at.q_ld, LP_BQ);
   tc_make_map_bf16(&mk, k, keys, hd, (unsigned long long)k_ld, LP_BK);
   tc_make_map_bf16(&mv, vt, hv, keys, (unsigned long long)vt_ld, (unsigned)at.vdim);
-  const size_t smem = lp_smem(at.dim, at.vdim);
-  LB_CUDA(cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  launch_pdl(latent_prefill_kernel, dim3((unsigned)((b.n + LP_BQ - 1) / LP_BQ), (unsigned)at.heads, (unsigned)b.streams),
-             dim3(LP_THREADS), smem, st, false, mq, mk, mv, a, err);
+  lp_launch<false>(mq, mk, mv, a, at.heads, b.streams, st, err);
+}
+
+void launch_grouped_prefill(const GroupedAttention &at, const RowBatch &b, cudaStream_t st, DevErr *err) {
+  LpArgs a{};
+  a.dim = at.dim;
+  a.vdim = at.vdim;
+  a.n = b.n;
+  a.group = at.heads / at.groups;
+  a.pos0 = b.p0;
+  a.key_base = b.slot0 * at.cap;
+  a.key_rows = at.cap;
+  a.n_keys = b.p0 + b.n;
+  a.span = at.span;
+  a.factor = at.scale * 1.4426950408889634f;
+  a.out = static_cast<bf16 *>(at.out);
+  a.out_ld = at.out_ld;
+  CUtensorMap mq, mk, mv;
+  const unsigned long long kd = (unsigned long long)at.groups * at.dim, vd = (unsigned long long)at.groups * at.vdim;
+  const unsigned long long keys = (unsigned long long)at.slots * at.cap;
+  tc_make_map_bf16(&mq, at.q, (unsigned long long)b.rows(), (unsigned long long)at.heads * at.dim, (unsigned long long)at.q_ld,
+                   LP_BQ);
+  tc_make_map_bf16(&mk, at.k_cache, keys, kd, kd, LP_BK);
+  tc_make_map_bf16(&mv, at.v_cache, keys, vd, vd, LP_BK);
+  lp_launch<true>(mq, mk, mv, a, at.heads, b.streams, st, err);
 }
 
 }  // namespace lb

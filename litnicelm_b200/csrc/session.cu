@@ -1074,6 +1074,9 @@ static void session_loop_buffers(litnice_b200_session *s, size_t logit_rows) {
   LB_CUDA(cudaMemsetAsync(s->state, 0, sizeof(LoopState) + 16, s->st));
 }
 
+// Positions a session keeps token ids for when the design itself has no bound.
+constexpr int UNBOUNDED_POSITIONS = 1 << 20;
+
 // Names the reason a model folder was refused when no session exists to carry it.
 static thread_local std::string g_create_error = "null session";
 
@@ -1109,7 +1112,7 @@ int litnice_b200_session_create_model(const char *model_dir, int32_t dtype, int3
   s->dims.n_heads = 1;
   s->dims.d_model = s->model->width();
   s->dims.vocab_size = s->model->vocab();
-  s->dims.max_seq_len = s->model->max_positions();
+  s->dims.max_seq_len = s->model->max_positions() > 0 ? s->model->max_positions() : UNBOUNDED_POSITIONS;
   s->slot_len.assign((size_t)max_streams, 0);
   *out = s;  // handed out even on failure below so the caller can read the error text
   const int rc = guarded(s, [&]() {

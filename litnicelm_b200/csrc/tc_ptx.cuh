@@ -160,6 +160,19 @@ __device__ __forceinline__ unsigned long long umma_desc_k128(unsigned smem_addr)
   d |= 2ull << 61;
   return d;
 }
+// The same for an operand whose M or N index is contiguous: rows of one k with 64 elements (128 bytes, 128-byte
+// swizzle), eight k per 1024-byte atom (stride byte offset from one atom to the next in k), the next 64
+// elements of M or N `slab` bytes further (leading byte offset). The instruction descriptor says so too.
+__device__ __forceinline__ unsigned long long umma_desc_mn128(unsigned smem_addr, unsigned slab) {
+  unsigned long long d = 0;
+  d |= (unsigned long long)((smem_addr & 0x3FFFFu) >> 4);
+  d |= (unsigned long long)((slab & 0x3FFFFu) >> 4) << 16;
+  d |= (unsigned long long)(1024 >> 4) << 32;
+  d |= 1ull << 46;
+  d |= 2ull << 61;
+  return d;
+}
+constexpr unsigned UMMA_B_MN_MAJOR = 1u << 16;
 
 // Instruction descriptor: D fp32, A and B TF32, both K-major, M = 128, N = bn.
 // The same with fp16 operands (format code 0).
