@@ -16,8 +16,8 @@ prints one JSON line. Beside the headline the default line carries: `parity`
 `extra` (config 3: 64 lockstep streams with the fused sampler; config 5 cut
 over the GPUs; config 2 in the opt-in cached mode).
 
-`--design mitilix` measures a registered decoder design instead (prefill and decode at a few
-sizes, beside the transformer of equal size), one JSON line per size.
+`--design mitilix` or `--design gobesun` measures a registered decoder design instead (prefill and decode
+at a few sizes, beside the closest model of equal size: the transformer, or Mitilix), one JSON line per size.
 
 `--impl reference` times the reference's own CPU backend (oracle/_ref, built
 from the reference sources) on a bounded sample of the same workload.
@@ -711,21 +711,47 @@ DESIGN_STREAMS = (1, 8, 64)
 DESIGN_NEW = 64                  # timed tokens per stream
 
 
-def design_config(z: dict) -> dict:
+def mitilix_design(z: dict) -> dict:
     layers = [{"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"], "window": z["window"],
                "scale": z["dim"] ** -0.5, "ff": z["ff"], "kv_from": i - 1 if i % 3 == 2 else None}
               for i in range(z["n_layers"])]
     return formats.mitilix_config(z["width"], z["vocab"], 2048, layers, taps=4, eps=1e-6)
 
 
+def gobesun_design(z: dict) -> dict:
+    """As many layer runs as the other models have layers: three delta layers to one attention layer, a third of the
+    runs repeats of a loop. The gated feed-forward's three matrices hold about what their two do; delta heads of 128 (64
+    in the smallest), half as many key heads; attention heads as the others', a quarter as many key heads, chunks as long
+    as the others' windows."""
+    layers, ff = [], (z["ff"] * 2 // 3 + 63) // 64 * 64
+    n = z["n_layers"] * 2 // 3
+    for i in range(n):
+        if i % 4 == 3:
+            rot = {"dims": z["dim"], "base": 1e6, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}
+            layers.append(formats.chunk_attention_layer(z["heads"], z["heads"] // 4, z["dim"], z["vdim"], z["window"], rot,
+                                                        ff=ff))
+        else:
+            dim = 128 if z["width"] > 512 else 64
+            heads = z["width"] // dim * (2 if z["dim"] == 128 else 1)
+            layers.append(formats.delta_layer(heads, heads // 2, dim, dim, 4, ff=ff))
+    repeat = z["n_layers"] - n
+    return formats.gobesun_config(z["width"], z["vocab"], layers, (n - repeat, n, 2), z["width"] ** 0.5, 1e-6)
+
+
 def design_weights(config: dict, seed: int):
     """Random bfloat16 weights of the configuration's shapes, drawn on the device."""
     import torch
     g = torch.Generator(device="cuda").manual_seed(seed)
+    gobesun = config["architecture"] == "Gobesun"
     out = {}
-    for name, shape in formats.mitilix_shapes(config).items():
-        if name.endswith("norm1") or name in ("final.norm",) or name.endswith("dkv.norm"):
+    for name, shape in (formats.gobesun_shapes if gobesun else formats.mitilix_shapes)(config).items():
+        last = name.rsplit(".", 1)[-1]
+        if gobesun and (last in ("norm1", "norm1b", "norm2", "norm2b", "dt_bias") or name == "final.norm"):
+            t = torch.zeros(shape, device="cuda")
+        elif last in ("norm", "norm1"):
             t = torch.ones(shape, device="cuda")
+        elif last == "A_log":
+            t = torch.linspace(-4.0, 1.0, shape[0], device="cuda")
         else:
             fan = 1.0 if name in ("embed", "pos") else shape[-1]
             t = torch.randn(shape, generator=g, device="cuda") * fan ** -0.5
@@ -733,15 +759,37 @@ def design_weights(config: dict, seed: int):
     return out
 
 
-def design_work(z: dict, config: dict):
-    """Algorithmic flops per prefill token (projections) and per visible key (attention), and the bytes of the
-    layers' and the head's weights a decoding step reads."""
+def mitilix_work(z: dict, config: dict):
+    """Algorithmic flops per prefill token, bytes of the layers' and the head's weights a decoding step reads, and bytes of
+    cache and state it moves per stream."""
     d, n = z["width"], z["n_layers"]
     own = sum(e["mixer"].get("kv_from") is None for e in config["layers"])
     q, o, r = z["heads"] * z["dim"], z["heads"] * z["vdim"], z["kv_rank"]
-    per_layer = d * q + r * (q + o) + d * o + 2 * d * z["ff"]
-    weights = n * per_layer + own * d * r
-    return 2.0 * weights, 2.0 * n * (q + o), 2.0 * (weights + d * z["vocab"]), 2.0 * n * r
+    weights = n * (d * q + r * (q + o) + d * o + 2 * d * z["ff"]) + own * d * r
+    s, w = DESIGN_PREFILL[1], z["window"]
+    keys = sum(min(i + 1, w) for i in range(s)) / s
+    return 2.0 * weights + 2.0 * n * (q + o) * keys, 2.0 * (weights + d * z["vocab"]), 2.0 * n * r * min(w, DESIGN_CONTEXT)
+
+
+def gobesun_work(z: dict, config: dict):
+    d, lp, layers = z["width"], config["loop"], config["layers"]
+    runs = layers[:lp["start"]] + layers[lp["start"]:lp["stop"]] * lp["times"] + layers[lp["stop"]:]
+    weights = flops = moved = 0.0
+    s = DESIGN_PREFILL[1]
+    for e in runs:
+        m = e["mixer"]
+        h, g, dim, vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        weights += 3.0 * d * e["mlp"]["ff"] + d * h * vdim
+        if e["type"] == "delta":
+            weights += d * (2 * g * dim + 2 * h * vdim + 2 * h)
+            flops += 6.0 * h * dim * vdim           # the rule itself: two reads and one write of the state
+            moved += 8.0 * h * dim * vdim           # float state, read and written
+        else:
+            c = m["mask"]["size"]
+            weights += d * ((h + g) * dim + g * vdim)
+            flops += 2.0 * h * (dim + vdim) * sum(i % c + 1 for i in range(s)) / s
+            moved += 2.0 * g * (dim + vdim) * sum(i % c + 1 for i in range(DESIGN_CONTEXT, DESIGN_CONTEXT + DESIGN_NEW)) / DESIGN_NEW
+    return 2.0 * weights + flops, 2.0 * (weights + d * z["vocab"]), moved
 
 
 def measure_session(box, sess, vocab, steps, warmup, streams_list, context, new, prefill):
@@ -777,76 +825,90 @@ def measure_session(box, sess, vocab, steps, warmup, streams_list, context, new,
     return out
 
 
-def run_design_arm(args, rank, local_rank, world):
-    """Prefill and decode throughput of the registered design beside the litnicelm transformer of equal size (its
-    cached mode for decoding, its whole-context pass for prefill). One JSON line per size."""
+def measure_design(box, z, name, args):
+    """Figures of one registered design at one size, with its fractions of the measured peaks, and the clocks meanwhile."""
     import shutil
-    from litnicelm_b200.plugin import ModelSession, Session
+    from litnicelm_b200.plugin import ModelSession
+    peaks = load_peaks()
+    config = {"mitilix": mitilix_design, "gobesun": gobesun_design}[name](z)
+    folder = tempfile.mkdtemp(prefix=name + "_")
+    clocks = ClockSampler(box.local_rank)
+    try:
+        formats.write_model_folder(folder, config, design_weights(config, 3))
+        with ModelSession(folder, "bfloat16", max(DESIGN_STREAMS)) as sess:
+            clocks.start()
+            out = measure_session(box, sess, z["vocab"], args.steps, args.warmup, DESIGN_STREAMS, DESIGN_CONTEXT,
+                                  DESIGN_NEW, DESIGN_PREFILL)
+            clock_info = clocks.stop()
+    finally:
+        shutil.rmtree(folder, ignore_errors=True)
+    flops, wbytes, cbytes = {"mitilix": mitilix_work, "gobesun": gobesun_work}[name](z, config)
+    pf = out["prefill"]
+    tflops = pf["tokens_per_s"] * flops / 1e12
+    pf.update(achieved_tflops=tflops, frac_of_bf16_peak=tflops / peaks["bf16_tflops"])
+    for n, d in out["decode"].items():
+        by = wbytes + int(n) * cbytes
+        d.update(bytes_per_step=by, achieved_gbs=by / (d["ms_per_token"] * 1e-3) / 1e9)
+        d["frac_of_hbm_peak"] = d["achieved_gbs"] / peaks["hbm_gbs"]
+    return out, clock_info
+
+
+def measure_transformer(box, z, args):
+    """The litnicelm transformer of equal size: its whole-context pass for prefill, its cached mode for decoding."""
+    from litnicelm_b200.plugin import Session
+    peaks = load_peaks()
+    gd = formats.ModelDims(z["n_layers"], z["heads"], z["width"], z["ff"], z["vocab"], 2048)
+    arena = formats.make_param_arena(gd, 1004)
+    base = {}
+    with Session(gd, DESIGN_PREFILL[0]) as sess:
+        sess.load_params(arena)
+        base["prefill"] = measure_session(box, sess, z["vocab"], args.steps, args.warmup, (), DESIGN_CONTEXT,
+                                          DESIGN_NEW, DESIGN_PREFILL)["prefill"]
+    os.environ["LITNICE_B200_KV_CACHE"] = "1"
+    if z["width"] > 1024:             # the resident kernel's CTAs do not fit an SM at this width
+        os.environ["LITNICE_B200_KV_PERSIST"] = "0"
+    try:
+        with Session(gd, max(DESIGN_STREAMS)) as sess:
+            sess.load_params(arena)
+            base["decode"] = measure_session(box, sess, z["vocab"], args.steps, 1, DESIGN_STREAMS, DESIGN_CONTEXT,
+                                             DESIGN_NEW, (1, 64))["decode"]
+    finally:
+        del os.environ["LITNICE_B200_KV_CACHE"]
+        os.environ.pop("LITNICE_B200_KV_PERSIST", None)
+    keys = (DESIGN_PREFILL[1] + 1) / 2
+    flops = gd.n_layers * (2.0 * (4 * gd.d_model ** 2 + 2 * gd.d_model * gd.d_ff) + 4.0 * gd.d_model * keys)
+    b = base["prefill"]
+    b["achieved_tflops"] = b["tokens_per_s"] * flops / 1e12
+    b["frac_of_bf16_peak"] = b["achieved_tflops"] / peaks["bf16_tflops"]
+    for n, d in base["decode"].items():
+        by = 4.0 * (gd.n_layers * (4 * gd.d_model ** 2 + 2 * gd.d_model * gd.d_ff) + gd.d_model * gd.vocab)
+        by += int(n) * 8.0 * gd.n_layers * gd.d_model * DESIGN_CONTEXT
+        d.update(bytes_per_step=by, achieved_gbs=by / (d["ms_per_token"] * 1e-3) / 1e9)
+        d["frac_of_hbm_peak"] = d["achieved_gbs"] / peaks["hbm_gbs"]
+    return base
+
+
+def run_design_arm(args, rank, local_rank, world):
+    """Prefill and decode throughput of a registered design beside the closest model of equal size. One JSON line per
+    size."""
     if world > 1:
         raise SystemExit("--design runs on one GPU")
     box = Box(rank, local_rank, world)
-    peaks = load_peaks()
     names = args.design_sizes.split(",") if args.design_sizes else list(DESIGN_SIZES)
     for name in names:
         z = DESIGN_SIZES[name]
-        config = design_config(z)
-        folder = tempfile.mkdtemp(prefix="mitilix_")
-        clocks = ClockSampler(local_rank)
-        try:
-            formats.write_model_folder(folder, config, design_weights(config, 3))
-            with ModelSession(folder, "bfloat16", max(DESIGN_STREAMS)) as sess:
-                clocks.start()
-                ours = measure_session(box, sess, z["vocab"], args.steps, args.warmup, DESIGN_STREAMS, DESIGN_CONTEXT,
-                                       DESIGN_NEW, DESIGN_PREFILL)
-                clock_info = clocks.stop()
-        finally:
-            shutil.rmtree(folder, ignore_errors=True)
-        proj, per_key, wbytes, cbytes = design_work(z, config)
-        s, w = DESIGN_PREFILL[1], z["window"]
-        keys = sum(min(i + 1, w) for i in range(s)) / s
-        pf = ours["prefill"]
-        tflops = pf["tokens_per_s"] * (proj + per_key * keys) / 1e12
-        pf.update(achieved_tflops=tflops, frac_of_bf16_peak=tflops / peaks["bf16_tflops"])
-        for n, d in ours["decode"].items():
-            by = wbytes + int(n) * cbytes * min(w, DESIGN_CONTEXT)
-            d.update(bytes_per_step=by, achieved_gbs=by / (d["ms_per_token"] * 1e-3) / 1e9)
-            d["frac_of_hbm_peak"] = d["achieved_gbs"] / peaks["hbm_gbs"]
-        base = None
-        if not args.no_extras and z["dim"] == 64 and z["heads"] * z["dim"] == z["width"]:
-            gd = formats.ModelDims(z["n_layers"], z["heads"], z["width"], z["ff"], z["vocab"], 2048)
-            arena = formats.make_param_arena(gd, 1004)
-            base = {}
-            with Session(gd, DESIGN_PREFILL[0]) as sess:
-                sess.load_params(arena)
-                base["prefill"] = measure_session(box, sess, z["vocab"], args.steps, args.warmup, (), DESIGN_CONTEXT,
-                                                  DESIGN_NEW, DESIGN_PREFILL)["prefill"]
-            os.environ["LITNICE_B200_KV_CACHE"] = "1"
-            if z["width"] > 1024:             # the resident kernel's CTAs do not fit an SM at this width
-                os.environ["LITNICE_B200_KV_PERSIST"] = "0"
-            try:
-                with Session(gd, max(DESIGN_STREAMS)) as sess:
-                    sess.load_params(arena)
-                    base["decode"] = measure_session(box, sess, z["vocab"], args.steps, 1, DESIGN_STREAMS, DESIGN_CONTEXT,
-                                                     DESIGN_NEW, (1, 64))["decode"]
-            finally:
-                del os.environ["LITNICE_B200_KV_CACHE"]
-                os.environ.pop("LITNICE_B200_KV_PERSIST", None)
-            keys = (s + 1) / 2
-            flops = gd.n_layers * (2.0 * (4 * gd.d_model ** 2 + 2 * gd.d_model * gd.d_ff) + 4.0 * gd.d_model * keys)
-            b = base["prefill"]
-            b["achieved_tflops"] = b["tokens_per_s"] * flops / 1e12
-            b["frac_of_bf16_peak"] = b["achieved_tflops"] / peaks["bf16_tflops"]
-            for n, d in base["decode"].items():
-                by = 4.0 * (gd.n_layers * (4 * gd.d_model ** 2 + 2 * gd.d_model * gd.d_ff) + gd.d_model * gd.vocab)
-                by += int(n) * 8.0 * gd.n_layers * gd.d_model * DESIGN_CONTEXT
-                d.update(bytes_per_step=by, achieved_gbs=by / (d["ms_per_token"] * 1e-3) / 1e9)
-                d["frac_of_hbm_peak"] = d["achieved_gbs"] / peaks["hbm_gbs"]
+        ours, clock_info = measure_design(box, z, args.design, args)
+        beside = {}
+        if not args.no_extras and args.design == "gobesun":
+            beside["mitilix_of_equal_size"] = measure_design(box, z, "mitilix", args)[0]
+        if not args.no_extras and args.design == "mitilix":
+            fits = z["dim"] == 64 and z["heads"] * z["dim"] == z["width"]
+            beside["transformer_of_equal_size"] = measure_transformer(box, z, args) if fits else None
         print(json.dumps({
-            "metric": "prefill and decode throughput of a registered design", "design": "Mitilix", "size": name,
-            "sizes": z, "value": pf["tokens_per_s"], "unit": "prefill tokens/s", "higher_is_better": True,
-            "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "dtype": "bf16", "data": "synthetic",
-            "design_figures": ours, "transformer_of_equal_size": base,
-            "peaks": peaks, "clocks": clock_info,
+            "metric": "prefill and decode throughput of a registered design", "design": args.design.capitalize(),
+            "size": name, "sizes": z, "value": ours["prefill"]["tokens_per_s"], "unit": "prefill tokens/s",
+            "higher_is_better": True, "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "dtype": "bf16",
+            "data": "synthetic", "design_figures": ours, **beside, "peaks": load_peaks(), "clocks": clock_info,
             "l2": "256 MB buffer written before each prefill; a decoding step's weights exceed L2 from d1024 on"}),
             flush=True)
     box.close()
@@ -864,8 +926,8 @@ def main():
                     help="run the workload in the opt-in cached mode (an extension; not the headline)")
     ap.add_argument("--no-extras", action="store_true",
                     help="skip the output-head bandwidth block and the config-3 / config-5 side measurements")
-    ap.add_argument("--design", default=None, choices=["mitilix"],
-                    help="throughput of a registered decoder design beside the transformer of equal size (not the headline)")
+    ap.add_argument("--design", default=None, choices=["mitilix", "gobesun"],
+                    help="throughput of a registered decoder design beside the closest model of equal size (not the headline)")
     ap.add_argument("--design-sizes", default="", help="sizes of --design to run, with commas between them (default: all)")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))

@@ -362,10 +362,33 @@ int litnice_b200_gemv_time(int32_t m, int32_t k, int32_t n, int32_t repeats, int
  * their own device memory.
  *
  * c[m, n] = a[m, k] w[n, k]^T on bfloat16 operands. engine 0: few-row kernel (m <= 64), 1: tensor-core
- * kernel. Columns below n_half come back rounded to bfloat16 (through GELU when gelu is set), the
- * others as floats, added to what c holds when accumulate is set. */
+ * kernel. Columns below n_half come back rounded to bfloat16 (through the activation: 0 none, 1 GELU with the
+ * error function, 2 its tanh form), the others as floats, added to what c holds when accumulate is set. gated:
+ * columns 2 j and 2 j + 1 below n_half make one column act(c_2j) * c_2j+1, and c has n - n_half / 2 columns. */
 int litnice_b200_bf16_product_host(int32_t engine, const float *a, int32_t m, int32_t k, const float *w, int32_t n,
-                                   int32_t n_half, int32_t gelu, int32_t accumulate, float *c);
+                                   int32_t n_half, int32_t act, int32_t gated, int32_t accumulate, float *c);
+/* x [n, d] += rms(y) * (base + after) (y may be null), h = rms(x) * (base + before) (h may be null); rms(z) =
+ * z / sqrt(mean(z^2) + eps) per row. */
+int litnice_b200_residual_norm_host(int32_t dtype, float *x, const float *y, const float *after, const float *before,
+                                    float base, int32_t n, int32_t d, float eps, float *h);
+/* The gated delta rule on projected rows [n_streams, n, q | k | v | gate] (groups * dim twice, heads * vdim twice) and
+ * ba [n_streams, n, beta | decay] (heads each), in the given portions with state and history carried between them, from
+ * zero: convolution conv [2 groups dim + heads vdim, taps] and SiLU, recurrence, norm and gate. out [n_streams, n,
+ * heads * vdim], state [n_streams, heads, dim, vdim]: what the sequences leave behind. */
+int litnice_b200_delta_host(int32_t dtype, const float *rows, const float *ba, const float *conv, const float *a_log,
+                            const float *dt_bias, const float *norm, float eps, int32_t n_streams, int32_t n, int32_t heads,
+                            int32_t groups, int32_t dim, int32_t vdim, int32_t taps, const int32_t *portions,
+                            int32_t n_portions, float *out, float *state);
+/* Grouped attention of the rows p0 .. p0 + n - 1 of n_streams sequences, rows [n_streams, p0 + n, q | k | v] (heads * dim,
+ * groups * dim, groups * vdim): norm over whole rows of q and of k, rotation by p * turns[i] half turns, softmax over the
+ * keys of the span (0: the last span_size positions, 1: the query's own chunk of span_size). q_out [n_streams, n,
+ * heads * dim] and k_out [n_streams, p0 + n, groups * dim]: rotated; out [n_streams, n, heads * vdim]. engine 0: 32-bit,
+ * 1: the same on bfloat16 storage, 2: tensor-core kernel. */
+int litnice_b200_grouped_attention_host(int32_t engine, const float *rows, const float *q_weight, const float *k_weight,
+                                        float eps, int32_t rot_dims, const double *turns, float amplitude, int32_t n_streams,
+                                        int32_t p0, int32_t n, int32_t heads, int32_t groups, int32_t dim, int32_t vdim,
+                                        float scale, int32_t span_kind, int32_t span_size, float *q_out, float *k_out,
+                                        float *out);
 /* h = x / sqrt(mean(x^2) + eps) * gain for the rows of one sequence, out_i = h + conv_i(h) with the causal
  * per-channel convolutions w_i [d, taps] (w2 and out2 both or neither), computed in the given portions
  * with the state carried between them. */

@@ -402,3 +402,78 @@ def mitilix_random_weights(config: dict, seed: int) -> Dict[str, np.ndarray]:
             a = rng.standard_normal(shape, dtype=np.float32) * (shape[-1] ** -0.5)
         out[name] = from_bf16_bits(to_bf16_bits(np.asarray(a, np.float32)))
     return out
+
+
+def delta_layer(heads: int, kv_heads: int, dim: int, vdim: int, conv: int, ff: int = 0) -> dict:
+    """A Gobesun layer whose mixer is the gated delta rule (ff 0: no feed-forward)."""
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def chunk_attention_layer(heads: int, kv_heads: int, dim: int, vdim: int, chunk: int, rot: dict, scale: float = 0.0,
+                          ff: int = 0) -> dict:
+    """A Gobesun layer whose mixer is attention inside chunks. rot: dims, base and optionally scaling (factor, original,
+    fast, slow); scale 0: dim^-1/2."""
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim,
+                                           "mask": {"size": chunk}, "rot": rot, "scale": scale or dim ** -0.5},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def gobesun_config(width: int, vocab: int, layers: List[dict], loop: Tuple[int, int, int], embed_scale: float,
+                   eps: float) -> dict:
+    """config.json of a Gobesun model. loop: layers start .. stop - 1 run `times` times."""
+    return {"architecture": "Gobesun", "width": width, "vocab": vocab, "embedding": {"scale": embed_scale},
+            "norm": {"eps": eps}, "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]}, "layers": layers}
+
+
+def gobesun_shapes(config: dict) -> Dict[str, Tuple[int, ...]]:
+    """Name and shape of every tensor of a Gobesun model."""
+    d = config["width"]
+    shapes: Dict[str, Tuple[int, ...]] = {"embed": (config["vocab"], d)}
+    for i, e in enumerate(config["layers"]):
+        m, p = e["mixer"], f"l{i}."
+        heads, kv, dim, vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        delta = e["type"] == "delta"
+        for name in ("norm1", "norm1b") + (("norm2", "norm2b") if e.get("mlp") else ()):
+            shapes[p + name] = (d,)
+        rows = {"q": (kv if delta else heads) * dim, "k": kv * dim, "v": (heads if delta else kv) * vdim}
+        for t, n in rows.items():
+            shapes[p + f"mix.{t}"] = (n, d)
+            if delta:
+                shapes[p + f"mix.{t}.conv"] = (n, m["conv"])
+            elif t != "v":
+                shapes[p + f"mix.{t}.norm"] = (n,)
+        if delta:
+            shapes.update({p + "mix.b": (heads, d), p + "mix.a": (heads, d), p + "mix.A_log": (heads,),
+                           p + "mix.dt_bias": (heads,), p + "mix.norm": (vdim,), p + "mix.g": (heads * vdim, d)})
+        shapes[p + "mix.o"] = (d, heads * vdim)
+        if e.get("mlp"):
+            ff = e["mlp"]["ff"]
+            shapes.update({p + "mlp.gate": (ff, d), p + "mlp.up": (ff, d), p + "mlp.down": (d, ff)})
+    shapes["final.norm"] = (d,)
+    shapes["head"] = (config["vocab"], d)
+    return shapes
+
+
+def gobesun_random_weights(config: dict, seed: int) -> Dict[str, np.ndarray]:
+    """Random weights with moderate scores, decays from slow to fast and a stream of moderate size (rounded to bfloat16)."""
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in gobesun_shapes(config).items():
+        last = name.rsplit(".", 1)[-1]
+        if name.endswith("mix.norm") or name.endswith("q.norm") or name.endswith("k.norm"):
+            a = 1.0 + 0.2 * rng.standard_normal(shape)
+        elif last.startswith("norm"):
+            a = 0.2 * rng.standard_normal(shape)
+        elif last == "conv":
+            a = rng.standard_normal(shape) * (shape[-1] ** -0.5)
+        elif last == "A_log":
+            a = rng.uniform(-4.0, 1.0, shape)
+        elif last == "dt_bias":
+            a = 0.5 * rng.standard_normal(shape)
+        elif name == "embed":
+            a = rng.standard_normal(shape, dtype=np.float32) / config["embedding"]["scale"]
+        else:
+            a = rng.standard_normal(shape, dtype=np.float32) * (shape[-1] ** -0.5)
+        out[name] = from_bf16_bits(to_bf16_bits(np.asarray(a, np.float32)))
+    return out

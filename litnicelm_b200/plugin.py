@@ -570,22 +570,94 @@ class ModelSession(Session):
             raise NativeError(f"release failed ({rc})")
 
 
-def bf16_product_host(a: np.ndarray, w: np.ndarray, engine: int, n_half: int = 0, gelu: bool = False,
-                      c: Optional[np.ndarray] = None, lib: Optional[C.CDLL] = None) -> np.ndarray:
+ACTIVATIONS = {None: 0, "gelu": 1, "gelu_tanh": 2}
+
+
+def bf16_product_host(a: np.ndarray, w: np.ndarray, engine: int, n_half: int = 0, act: Optional[str] = None,
+                      gated: bool = False, c: Optional[np.ndarray] = None, lib: Optional[C.CDLL] = None) -> np.ndarray:
     """c[m, n] = a[m, k] w[n, k]^T on bfloat16 operands (litnice_b200_bf16_product_host); c given: added to."""
     lib = lib or load_library()
     f32p = C.POINTER(C.c_float)
     fn = lib.litnice_b200_bf16_product_host
-    fn.argtypes = [C.c_int32, f32p, C.c_int32, C.c_int32, f32p, C.c_int32, C.c_int32, C.c_int32, C.c_int32, f32p]
+    fn.argtypes = [C.c_int32, f32p, C.c_int32, C.c_int32, f32p] + [C.c_int32] * 5 + [f32p]
     a, w = np.ascontiguousarray(a, np.float32), np.ascontiguousarray(w, np.float32)
     m, k = a.shape
     n = w.shape[0]
-    out = np.zeros((m, n), np.float32) if c is None else np.array(c, np.float32, order="C")
+    out = np.zeros((m, n - n_half // 2 if gated else n), np.float32) if c is None else np.array(c, np.float32, order="C")
     p = lambda x: x.ctypes.data_as(f32p)
-    rc = fn(engine, p(a), m, k, p(w), n, n_half, int(gelu), int(c is not None), p(out))
+    rc = fn(engine, p(a), m, k, p(w), n, n_half, ACTIVATIONS[act], int(gated), int(c is not None), p(out))
     if rc != 0:
         raise RuntimeError(f"litnice_b200_bf16_product_host failed with status {rc}")
     return out
+
+
+def _floats(*arrays):
+    """Contiguous float32 arrays and their pointers (None stays None)."""
+    f32p = C.POINTER(C.c_float)
+    held = [None if a is None else np.ascontiguousarray(a, np.float32) for a in arrays]
+    return held, [None if a is None else a.ctypes.data_as(f32p) for a in held]
+
+
+def residual_norm_host(x: np.ndarray, y: Optional[np.ndarray], after: Optional[np.ndarray], before: Optional[np.ndarray],
+                       base: float, eps: float, dtype: str = "float32", lib: Optional[C.CDLL] = None):
+    """(x + rms(y) (base + after), rms of that times (base + before) or None) (litnice_b200_residual_norm_host)."""
+    lib = lib or load_library()
+    f32p = C.POINTER(C.c_float)
+    fn = lib.litnice_b200_residual_norm_host
+    fn.argtypes = [C.c_int32] + [f32p] * 4 + [C.c_float, C.c_int32, C.c_int32, C.c_float, f32p]
+    n, d = x.shape
+    x = np.array(x, np.float32, order="C")
+    h = None if before is None else np.empty((n, d), np.float32)
+    held, p = _floats(x, y, after, before, h)
+    rc = fn(DTYPES[dtype], p[0], p[1], p[2], p[3], base, n, d, eps, p[4])
+    if rc != 0:
+        raise RuntimeError(f"litnice_b200_residual_norm_host failed with status {rc}")
+    return held[0], held[4]
+
+
+def delta_host(rows: np.ndarray, ba: np.ndarray, conv: np.ndarray, a_log: np.ndarray, dt_bias: np.ndarray, norm: np.ndarray,
+               eps: float, heads: int, groups: int, dim: int, vdim: int, portions: Optional[Sequence[int]] = None,
+               dtype: str = "float32", lib: Optional[C.CDLL] = None):
+    """rows [streams, n, q | k | v | gate], ba [streams, n, 2 * heads]: (outputs [streams, n, heads * vdim], final states
+    [streams, heads, dim, vdim]) of the gated delta rule (litnice_b200_delta_host)."""
+    lib = lib or load_library()
+    f32p, i32p = C.POINTER(C.c_float), C.POINTER(C.c_int32)
+    fn = lib.litnice_b200_delta_host
+    fn.argtypes = [C.c_int32] + [f32p] * 6 + [C.c_float] + [C.c_int32] * 7 + [i32p, C.c_int32, f32p, f32p]
+    b, n = rows.shape[:2]
+    out, state = np.empty((b, n, heads * vdim), np.float32), np.empty((b, heads, dim, vdim), np.float32)
+    por = np.ascontiguousarray([n] if portions is None else portions, np.int32)
+    held, p = _floats(rows, ba, conv, a_log, dt_bias, norm, out, state)
+    rc = fn(DTYPES[dtype], *p[:6], eps, b, n, heads, groups, dim, vdim, conv.shape[1], por.ctypes.data_as(i32p), len(por), p[6],
+            p[7])
+    if rc != 0:
+        raise RuntimeError(f"litnice_b200_delta_host failed with status {rc}")
+    return held[6], held[7]
+
+
+SPANS = {"window": 0, "chunk": 1}
+
+
+def grouped_attention_host(engine: int, rows: np.ndarray, n: int, q_weight: np.ndarray, k_weight: np.ndarray, eps: float,
+                           turns: np.ndarray, amplitude: float, heads: int, groups: int, dim: int, vdim: int, scale: float,
+                           span: str, size: int, lib: Optional[C.CDLL] = None):
+    """rows [streams, T, q | k | v]: (rotated queries of the last n positions, rotated keys of all, outputs of the last n)
+    (litnice_b200_grouped_attention_host)."""
+    lib = lib or load_library()
+    f32p, f64p = C.POINTER(C.c_float), C.POINTER(C.c_double)
+    fn = lib.litnice_b200_grouped_attention_host
+    fn.argtypes = ([C.c_int32] + [f32p] * 3 + [C.c_float, C.c_int32, f64p, C.c_float] + [C.c_int32] * 7 +
+                   [C.c_float, C.c_int32, C.c_int32, f32p, f32p, f32p])
+    b, t = rows.shape[:2]
+    turns = np.ascontiguousarray(turns, np.float64)
+    q, k = np.empty((b, n, heads * dim), np.float32), np.empty((b, t, groups * dim), np.float32)
+    out = np.empty((b, n, heads * vdim), np.float32)
+    held, p = _floats(rows, q_weight, k_weight, q, k, out)
+    rc = fn(engine, *p[:3], eps, 2 * len(turns), turns.ctypes.data_as(f64p), amplitude, b, t - n, n, heads, groups, dim, vdim,
+            scale, SPANS[span], size, *p[3:])
+    if rc != 0:
+        raise RuntimeError(f"litnice_b200_grouped_attention_host failed with status {rc}")
+    return held[3], held[4], held[5]
 
 
 def rms_canon_host(x: np.ndarray, gain: float, eps: float, w1: np.ndarray, w2: Optional[np.ndarray] = None,

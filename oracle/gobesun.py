@@ -2,6 +2,10 @@
 
 One function per mechanism, written from the equations in double precision; nothing here is
 shared with the product path. Weights are a dict name -> array (linear weights [out, in]).
+
+``cast`` (the identity unless given) is applied to what a served model may hold in 16 bits: inputs and
+results of the matrix products, convolved vectors, rotated queries and keys. With a rounding function it
+shows how far rounding alone moves each position.
 """
 from __future__ import annotations
 
@@ -9,6 +13,10 @@ import math
 from typing import Dict, List, Optional
 
 import numpy as np
+
+
+def exact(x: np.ndarray) -> np.ndarray:
+    return x
 
 
 def rms_normalise(x: np.ndarray, eps: float) -> np.ndarray:
@@ -80,9 +88,9 @@ def gated_head_norm(o: np.ndarray, gate: np.ndarray, w: np.ndarray, eps: float) 
     return rms_normalise(o, eps) * w * silu(gate)
 
 
-def delta_mixer(h: np.ndarray, w: Dict[str, np.ndarray], p: str, m: dict, eps: float) -> np.ndarray:
+def delta_mixer(h: np.ndarray, w: Dict[str, np.ndarray], p: str, m: dict, eps: float, cast=exact) -> np.ndarray:
     n, heads, kv, dim, vdim = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q, k, v = (silu(causal_channel_conv(h @ w[p + t].T, w[p + t + ".conv"])) for t in "qkv")
+    q, k, v = (cast(silu(causal_channel_conv(cast(h @ w[p + t].T), w[p + t + ".conv"]))) for t in "qkv")
     q = unit_vector(q.reshape(n, kv, dim)) * dim ** -0.5
     k = unit_vector(k.reshape(n, kv, dim))
     v = v.reshape(n, heads, vdim)
@@ -90,8 +98,8 @@ def delta_mixer(h: np.ndarray, w: Dict[str, np.ndarray], p: str, m: dict, eps: f
     log_g = log_decay(h @ w[p + "a"].T, w[p + "A_log"], w[p + "dt_bias"])
     o = np.stack([delta_rule(q[:, i * kv // heads], k[:, i * kv // heads], v[:, i], beta[:, i], log_g[:, i])
                   for i in range(heads)], axis=1)
-    o = gated_head_norm(o, (h @ w[p + "g"].T).reshape(n, heads, vdim), w[p + "norm"], eps)
-    return o.reshape(n, heads * vdim) @ w[p + "o"].T
+    o = gated_head_norm(o, cast(h @ w[p + "g"].T).reshape(n, heads, vdim), w[p + "norm"], eps)
+    return cast(o.reshape(n, heads * vdim)) @ w[p + "o"].T
 
 
 def yarn_frequencies(rot: dict) -> np.ndarray:
@@ -151,18 +159,18 @@ def grouped_attention(q: np.ndarray, k: np.ndarray, v: np.ndarray, scale: float,
     return out
 
 
-def attention_mixer(h: np.ndarray, w: Dict[str, np.ndarray], p: str, m: dict, eps: float) -> np.ndarray:
+def attention_mixer(h: np.ndarray, w: Dict[str, np.ndarray], p: str, m: dict, eps: float, cast=exact) -> np.ndarray:
     n, heads, kv, dim, vdim = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q = plain_rms_norm(h @ w[p + "q"].T, w[p + "q.norm"], eps).reshape(n, heads, dim)
-    k = plain_rms_norm(h @ w[p + "k"].T, w[p + "k.norm"], eps).reshape(n, kv, dim)
-    v = (h @ w[p + "v"].T).reshape(n, kv, vdim)
+    q = plain_rms_norm(cast(h @ w[p + "q"].T), w[p + "q.norm"], eps).reshape(n, heads, dim)
+    k = plain_rms_norm(cast(h @ w[p + "k"].T), w[p + "k.norm"], eps).reshape(n, kv, dim)
+    v = cast(h @ w[p + "v"].T).reshape(n, kv, vdim)
     at = np.arange(n, dtype=np.float64)
-    o = grouped_attention(rotate(q, at, m["rot"]), rotate(k, at, m["rot"]), v, m["scale"], m["mask"]["size"])
-    return o.reshape(n, heads * vdim) @ w[p + "o"].T
+    o = grouped_attention(cast(rotate(q, at, m["rot"])), cast(rotate(k, at, m["rot"])), v, m["scale"], m["mask"]["size"])
+    return cast(o.reshape(n, heads * vdim)) @ w[p + "o"].T
 
 
-def gated_feed_forward(h: np.ndarray, gate: np.ndarray, up: np.ndarray, down: np.ndarray) -> np.ndarray:
-    return (gelu_tanh(h @ gate.T) * (h @ up.T)) @ down.T
+def gated_feed_forward(h: np.ndarray, gate: np.ndarray, up: np.ndarray, down: np.ndarray, cast=exact) -> np.ndarray:
+    return cast(gelu_tanh(h @ gate.T) * (h @ up.T)) @ down.T
 
 
 def layer_order(cfg: dict) -> List[int]:
@@ -172,7 +180,8 @@ def layer_order(cfg: dict) -> List[int]:
     return list(range(a)) + list(range(a, b)) * lp["times"] + list(range(b, len(cfg["layers"])))
 
 
-def forward(cfg: dict, w: Dict[str, np.ndarray], tokens, layers_out: Optional[List[np.ndarray]] = None) -> np.ndarray:
+def forward(cfg: dict, w: Dict[str, np.ndarray], tokens, layers_out: Optional[List[np.ndarray]] = None,
+            cast=exact) -> np.ndarray:
     """Logits [T, vocab] of one sequence; layers_out receives the residual stream after every layer run."""
     w = {k: np.asarray(v, np.float64) for k, v in w.items()}
     eps = cfg["norm"]["eps"]
@@ -180,15 +189,15 @@ def forward(cfg: dict, w: Dict[str, np.ndarray], tokens, layers_out: Optional[Li
     for i in layer_order(cfg):
         e, p = cfg["layers"][i], f"l{i}."
         mixer = {"delta": delta_mixer, "attention": attention_mixer}[e["type"]]
-        h = centred_rms_norm(x, w[p + "norm1"], eps)
-        x = x + centred_rms_norm(mixer(h, w, p + "mix.", e["mixer"], eps), w[p + "norm1b"], eps)
+        h = cast(centred_rms_norm(x, w[p + "norm1"], eps))
+        x = x + centred_rms_norm(mixer(h, w, p + "mix.", e["mixer"], eps, cast), w[p + "norm1b"], eps)
         if e.get("mlp") is not None:
-            h = centred_rms_norm(x, w[p + "norm2"], eps)
-            f = gated_feed_forward(h, w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"])
+            h = cast(centred_rms_norm(x, w[p + "norm2"], eps))
+            f = gated_feed_forward(h, w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"], cast)
             x = x + centred_rms_norm(f, w[p + "norm2b"], eps)
         if layers_out is not None:
             layers_out.append(x.copy())
-    return centred_rms_norm(x, w["final.norm"], eps) @ w["head"].T
+    return cast(centred_rms_norm(x, w["final.norm"], eps)) @ w["head"].T
 
 
 def greedy(cfg: dict, w: Dict[str, np.ndarray], prompt, steps: int) -> List[int]:

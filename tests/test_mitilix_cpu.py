@@ -95,7 +95,7 @@ def create(lib, folder, dtype=0):
 def test_registry_names_the_design(lib):
     assert "Mitilix" in plugin.architectures()
     p = subprocess.run([DRIVER, "designs"], capture_output=True, text=True, timeout=60)
-    assert p.returncode == 0 and "Mitilix" in p.stdout.split()
+    assert p.returncode == 0 and "Mitilix" in p.stdout.strip().split(",")
 
 
 @pytest.mark.parametrize("change,words", [

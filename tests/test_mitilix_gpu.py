@@ -54,7 +54,7 @@ def test_product(engine, m, n, k):
     assert np.abs(got - want).max() < 2e-5 * max(1.0, k ** 0.5)
     c = rng.standard_normal((m, n)).astype(np.float32)
     assert np.abs(bf16_product_host(a, w, engine, c=c) - (want + c)).max() < 2e-5 * max(1.0, k ** 0.5)
-    got = bf16_product_host(a, w, engine, n_half=n, gelu=True)
+    got = bf16_product_host(a, w, engine, n_half=n, act="gelu")
     assert np.abs(got - om.gelu_exact(want)).max() < 2 ** -8 * np.abs(want).max()
     half = n // 2 & ~7
     got = bf16_product_host(a, w, engine, n_half=half, c=c)
