@@ -721,15 +721,15 @@ def mitilix_design(z: dict) -> dict:
 def gobesun_design(z: dict) -> dict:
     """As many layer runs as the other models have layers: three delta layers to one attention layer, a third of the
     runs repeats of a loop. The gated feed-forward's three matrices hold about what their two do; delta heads of 128 (64
-    in the smallest), half as many key heads; attention heads as the others', a quarter as many key heads, chunks as long
-    as the others' windows."""
+    in the smallest), half as many key heads; attention heads as the others', a quarter as many key heads, chunks of the
+    prompt's length (decoding sees the whole context)."""
     layers, ff = [], (z["ff"] * 2 // 3 + 63) // 64 * 64
     n = z["n_layers"] * 2 // 3
     for i in range(n):
         if i % 4 == 3:
             rot = {"dims": z["dim"], "base": 1e6, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}
-            layers.append(formats.chunk_attention_layer(z["heads"], z["heads"] // 4, z["dim"], z["vdim"], z["window"], rot,
-                                                        ff=ff))
+            layers.append(formats.chunk_attention_layer(z["heads"], z["heads"] // 4, z["dim"], z["vdim"], DESIGN_PREFILL[1],
+                                                        rot, ff=ff))
         else:
             dim = 128 if z["width"] > 512 else 64
             heads = z["width"] // dim * (2 if z["dim"] == 128 else 1)

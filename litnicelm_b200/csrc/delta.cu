@@ -44,9 +44,6 @@ __device__ __forceinline__ void store4(bf16 *p, float4 v) {
   u.y = *reinterpret_cast<const unsigned *>(&b);
   *reinterpret_cast<uint2 *>(p) = u;
 }
-__device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) {
-  return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w));
-}
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -56,22 +53,74 @@ __device__ __forceinline__ float warp_sum(float v) {
 // ---- convolution -----------------------------------------------------------------
 
 constexpr int DC_THREADS = 128;
-constexpr int DC_STRIP = 16;  // rows per CTA (more when taps - 1 is larger)
+constexpr int DC_STRIP = 32;  // rows per CTA (more when taps - 1 is larger)
 
-// TAPS > 0: that many taps, the window of inputs in registers; 0: any number. Four channels per thread.
+// 16 bytes of a row.
+template <typename T>
+struct Wide;
+template <>
+struct Wide<float> {
+  static constexpr int N = 4;
+  static __device__ __forceinline__ void unpack(uint4 u, float (&f)[4]) {
+    f[0] = __uint_as_float(u.x);
+    f[1] = __uint_as_float(u.y);
+    f[2] = __uint_as_float(u.z);
+    f[3] = __uint_as_float(u.w);
+  }
+  static __device__ __forceinline__ void store(float *p, const float (&f)[4]) {
+    *reinterpret_cast<float4 *>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  }
+  static __device__ __forceinline__ float silu(float z) { return silu_f32(z); }
+};
+template <>
+struct Wide<bf16> {
+  static constexpr int N = 8;
+  static __device__ __forceinline__ void unpack(uint4 u, float (&f)[8]) {
+    const unsigned w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      f[2 * i] = __uint_as_float(w[i] << 16);
+      f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+  }
+  static __device__ __forceinline__ void store(bf16 *p, const float (&f)[8]) {
+    unsigned w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const __nv_bfloat162 v = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+      w[i] = *reinterpret_cast<const unsigned *>(&v);
+    }
+    *reinterpret_cast<uint4 *>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+  }
+  static __device__ __forceinline__ float silu(float z) { return silu_fast(z); }
+};
+
+__device__ __forceinline__ uint4 load16(const void *p) { return *reinterpret_cast<const uint4 *>(p); }
+
+// TAPS > 0: that many taps, the window of inputs in registers; 0: any number. 16 bytes of channels per thread.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(DC_THREADS)
 delta_conv_kernel(const T *in, int in_ld, const float *__restrict__ w, int taps_any, int channels, T *history, T *out,
                   DeltaRows g, int strip) {
+  constexpr int N = Wide<T>::N, TP = TAPS > 0 ? TAPS : 1;
   pdl_launch_dependents();
   const int taps = TAPS > 0 ? TAPS : taps_any;
-  const int c = (blockIdx.z * DC_THREADS + threadIdx.x) * 4;
+  const int c = (blockIdx.z * DC_THREADS + threadIdx.x) * N;
   const bool mine = c < channels;
-  constexpr int TP = TAPS > 0 ? TAPS : 1;
-  float4 wt[TP];
+  float wt[TP][N];
+  auto weights = [&](int j, float (&f)[N]) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+      const float4 v = load4(w + (long long)j * channels + c + i);
+      f[i] = v.x;
+      f[i + 1] = v.y;
+      f[i + 2] = v.z;
+      f[i + 3] = v.w;
+    }
+  };
   if (TAPS > 0 && mine) {
 #pragma unroll
-    for (int j = 0; j < TP; ++j) wt[j] = load4(w + (long long)j * channels + c);
+    for (int j = 0; j < TP; ++j) weights(j, wt[j]);
   }
   pdl_wait();
   if (!mine) return;
@@ -80,39 +129,64 @@ delta_conv_kernel(const T *in, int in_ld, const float *__restrict__ w, int taps_
   const T *x = in + (long long)b * g.n * in_ld + c;
   T *hist = history + (long long)(g.slot0 + b) * taps * channels + c;
   T *o = out + (long long)b * g.n * channels + c;
-  auto input = [&](int t) -> float4 {
-    if (t >= 0) return load4(x + (long long)t * in_ld);
+  auto input = [&](int t, float (&f)[N]) {
     const int p = p0 + t;
-    return p >= 0 ? load4(hist + (long long)(p % taps) * channels) : make_float4(0.f, 0.f, 0.f, 0.f);
-  };
-  auto finish = [&](int t, float4 a) {
-    store4(o + (long long)t * channels, make_float4(silu_f32(a.x), silu_f32(a.y), silu_f32(a.z), silu_f32(a.w)));
+    if (t >= 0) {
+      Wide<T>::unpack(load16(x + (long long)t * in_ld), f);
+    } else if (p >= 0) {
+      Wide<T>::unpack(load16(hist + (long long)(p % taps) * channels), f);
+    } else {
+#pragma unroll
+      for (int i = 0; i < N; ++i) f[i] = 0.f;
+    }
   };
   if (TAPS > 0) {
-    float4 win[TP];
+    float win[TP][N];
 #pragma unroll
-    for (int j = 0; j < TP - 1; ++j) win[j + 1] = input(t0 - (TP - 1) + j);
-#pragma unroll 4
-    for (int t = t0; t < t1; ++t) {
+    for (int j = 0; j < TP - 1; ++j) input(t0 - (TP - 1) + j, win[j + 1]);
+    constexpr int AHEAD = 8;  // rows requested together
+    for (int ta = t0; ta < t1; ta += AHEAD) {
+      uint4 raw[AHEAD];
 #pragma unroll
-      for (int j = 0; j + 1 < TP; ++j) win[j] = win[j + 1];
-      win[TP - 1] = input(t);
-      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int k = 0; k < AHEAD; ++k) raw[k] = load16(x + (long long)min(ta + k, t1 - 1) * in_ld);
 #pragma unroll
-      for (int j = 0; j < TP; ++j) a = fma4(wt[j], win[j], a);
-      finish(t, a);
+      for (int k = 0; k < AHEAD; ++k) {
+        if (ta + k >= t1) break;
+#pragma unroll
+        for (int j = 0; j + 1 < TP; ++j)
+#pragma unroll
+          for (int i = 0; i < N; ++i) win[j][i] = win[j + 1][i];
+        Wide<T>::unpack(raw[k], win[TP - 1]);
+        float y[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          float a = 0.f;
+#pragma unroll
+          for (int j = 0; j < TP; ++j) a = fmaf(wt[j][i], win[j][i], a);
+          y[i] = Wide<T>::silu(a);
+        }
+        Wide<T>::store(o + (long long)(ta + k) * channels, y);
+      }
     }
   } else {
     for (int t = t0; t < t1; ++t) {
-      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int j = 0; j < taps; ++j) a = fma4(load4(w + (long long)j * channels + c), input(t - taps + 1 + j), a);
-      finish(t, a);
+      float y[N] = {};
+      for (int j = 0; j < taps; ++j) {
+        float f[N], v[N];
+        weights(j, f);
+        input(t - taps + 1 + j, v);
+#pragma unroll
+        for (int i = 0; i < N; ++i) y[i] = fmaf(f[i], v[i], y[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < N; ++i) y[i] = Wide<T>::silu(y[i]);
+      Wide<T>::store(o + (long long)t * channels, y);
     }
   }
   // Only a stream's first strip reads the history, and this thread alone these channels of it.
   if (blockIdx.x == 0)
     for (int t = max(0, g.n - taps + 1); t < g.n; ++t)
-      store4(hist + (long long)((p0 + t) % taps) * channels, load4(x + (long long)t * in_ld));
+      *reinterpret_cast<uint4 *>(hist + (long long)((p0 + t) % taps) * channels) = load16(x + (long long)t * in_ld);
 }
 
 // ---- recurrence --------------------------------------------------------------------
@@ -193,7 +267,7 @@ delta_step_kernel(StepArgs a, const T *in, T *history, float *o_rows, T *out, De
           if (p >= 0) y = fmaf(a.conv[(long long)j * channels + c], to_f(hist[(long long)(p % a.taps) * channels]), y);
         }
         y = fmaf(a.conv[(long long)(a.taps - 1) * channels + c], to_f(x), y);
-        next[i] = to_f(from_f<T>(silu_f32(y)));
+        next[i] = to_f(from_f<T>(Wide<T>::silu(y)));
         if (tid + i * THREADS >= 2 * DIMS || h % (a.heads / a.groups) == 0) hist[(long long)(p0 % a.taps) * channels] = x;
       } else {
         next[i] = to_f(in[r * a.rows_ld + c]);
@@ -325,7 +399,7 @@ Scratch scratch_parts(const DeltaMixer &m, long long rows, int streams, Precisio
 constexpr int DELTA_CHUNK_ROWS = 17;  // portions of so many rows per stream and more take the chunked form
 
 template <typename T>
-int launch_t(const DeltaMixer &m, void *scratch, Precision type, const RowBatch &b, cudaStream_t st) {
+int launch_t(const DeltaMixer &m, void *scratch, Precision type, const RowBatch &b, cudaStream_t st, DevErr *err) {
   const Scratch part = scratch_parts(m, b.rows(), b.streams, type);
   char *at = static_cast<char *>(scratch);
   T *conv = reinterpret_cast<T *>(at);
@@ -365,7 +439,7 @@ int launch_t(const DeltaMixer &m, void *scratch, Precision type, const RowBatch 
   const int strip = m.taps - 1 > DC_STRIP ? m.taps - 1 : DC_STRIP, channels = m.conv_channels();
   auto convolve = [&](auto kernel) {
     launch_pdl(kernel, dim3((unsigned)((b.n + strip - 1) / strip), (unsigned)b.streams,
-                            (unsigned)((channels / 4 + DC_THREADS - 1) / DC_THREADS)),
+                            (unsigned)((channels / Wide<T>::N + DC_THREADS - 1) / DC_THREADS)),
                dim3(DC_THREADS), 0, st, g_pdl_enabled, in, m.in_ld, m.conv, m.taps, channels, static_cast<T *>(m.history), conv, g,
                strip);
   };
@@ -379,7 +453,7 @@ int launch_t(const DeltaMixer &m, void *scratch, Precision type, const RowBatch 
   int launches = 1;
   if (type == Precision::BF16 && b.n >= DELTA_CHUNK_ROWS && delta_chunk_supports(m)) {
     bool normed = false;
-    launches += launch_delta_chunks(m, conv, o, at + part.conv + part.o, b, &normed, st);
+    launches += launch_delta_chunks(m, conv, o, at + part.conv + part.o, b, &normed, st, err);
     if (normed) return launches;
   } else {
     const T *src = conv;
@@ -404,8 +478,8 @@ size_t delta_scratch_bytes(const DeltaMixer &m, long long rows, int streams, Pre
   return p.conv + p.o + p.chunk;
 }
 
-int launch_delta(const DeltaMixer &m, void *scratch, Precision type, const RowBatch &b, cudaStream_t st) {
-  return type == Precision::BF16 ? launch_t<bf16>(m, scratch, type, b, st) : launch_t<float>(m, scratch, type, b, st);
+int launch_delta(const DeltaMixer &m, void *scratch, Precision type, const RowBatch &b, cudaStream_t st, DevErr *err) {
+  return type == Precision::BF16 ? launch_t<bf16>(m, scratch, type, b, st, err) : launch_t<float>(m, scratch, type, b, st, err);
 }
 
 }  // namespace lb

@@ -10,8 +10,8 @@
 // bfloat16 values themselves. Everything else that enters a product (the state, (I + L)^-1 diag(beta), A, the
 // right-hand side, U) is 32-bit and enters as two bfloat16 terms.
 //
-//   delta_prepare_kernel   per chunk and key head: K'K'^T and Q'K'^T, then per head L, its inverse by blocks of
-//                          32, A, and the factors of a token; no chunk depends on another
+//   delta_prepare_kernel   per chunk and head: Q'K'^T and A, K'K'^T and L, the inverse by blocks of 32, and the
+//                          factors of a token; no chunk depends on another
 //   delta_scan_kernel      per stream, head and tile of value columns: the chunks in order. A warp owns 16 value
 //                          columns and keeps their part of S^T in registers as accumulators of mma.sync tiles,
 //                          whose layout is that of the next product's left operand: the chain
@@ -28,7 +28,7 @@ namespace {
 
 typedef __nv_bfloat16 bf16;
 
-constexpr int CH = 64;           // tokens per chunk
+constexpr int CH = DELTA_CHUNK;
 constexpr int MP = CH + 8;       // pitch of the chunk's matrices in shared memory
 constexpr int PREP_THREADS = 128;
 constexpr int TP = 68;           // pitch of the float matrices
@@ -44,8 +44,9 @@ __device__ __forceinline__ void ldmatrix4_trans(unsigned (&r)[4], const bf16 *p)
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
                : "r"(smem_addr(p)));
 }
+// (Not volatile: a function of registers, the compiler may spread them between the loads.)
 __device__ __forceinline__ void mma(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -76,38 +77,47 @@ __device__ __forceinline__ void operand(const float (&c0)[4], const float (&c1)[
   split(c1[2], c1[3], hi[3], lo[3]);
 }
 
-struct ChunkArgs {
-  int heads, groups, dim, vdim, channels, n, chunks;
+// acc += a x over the right operand's blocks of 16 rows from the given one on.
+__device__ __forceinline__ void terms(float (&acc)[8][4], const unsigned (&a)[4], const unsigned (&x)[4][4], int from = 0) {
+#pragma unroll
+  for (int j = 0; j < 4; ++j)
+    if (j >= from) {
+      mma(acc[2 * j], a, x[j][0], x[j][1]);
+      mma(acc[2 * j + 1], a, x[j][2], x[j][3]);
+    }
+}
+
+struct PrepareArgs {
+  DeltaChunks c;
   float q_scale;
   const float *a_log, *dt_bias;
   const float *ba;
   int ba_ld;
 };
 
-// Matrices of a chunk and head: [inverse high, low, A high, low][64][64], only blocks of 16 columns that start at or
-// below the diagonal of their 16 rows are written and read.
+// Of a chunk's matrices only blocks of 16 columns that start at or below the diagonal of their 16 rows are written and read.
 constexpr int MAT = CH * CH;
-// Factors of a token: e^G r, e^G r', e^(G_last - G) r, e^G_last.
-__device__ __forceinline__ long long chunk_at(const ChunkArgs &a, int b, int h, int chunk) {
+__device__ __forceinline__ long long chunk_at(const DeltaChunks &a, int b, int h, int chunk) {
   return ((long long)b * a.heads + h) * a.chunks + chunk;
 }
 
-__global__ void __launch_bounds__(PREP_THREADS)
-delta_prepare_kernel(ChunkArgs a, const bf16 *conv, bf16 *mats, float4 *factors) {
+__global__ void __launch_bounds__(PREP_THREADS, 5)
+delta_prepare_kernel(PrepareArgs p) {
+  const DeltaChunks &a = p.c;
   extern __shared__ __align__(16) unsigned char raw[];
   const int pitch = a.dim + 8;
   bf16 *ks = reinterpret_cast<bf16 *>(raw), *qs = ks + CH * pitch;
-  float *ls = reinterpret_cast<float *>(qs + CH * pitch);  // [64][TP] L
-  float *ts = ls + CH * TP;                                // [64][TP] its inverse
+  float *lt = reinterpret_cast<float *>(raw);  // [64][TP] L transposed, over the vectors once the products are done
+  float *ts = lt + CH * TP;                    // [64][TP] its inverse
   __shared__ double gs[CH];
   __shared__ float rk[CH], rq[CH], bs[CH];
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, g = lane >> 2, t2 = (lane & 3) * 2;
-  const int chunk = blockIdx.x, grp = blockIdx.y, b = blockIdx.z;
+  const int chunk = blockIdx.x, h = blockIdx.y, b = blockIdx.z, grp = h / (a.heads / a.groups);
   const int t0 = chunk * CH, nt = min(CH, a.n - t0);
   const long long r0 = (long long)b * a.n + t0;
-  const bf16 *src = conv + r0 * a.channels + grp * a.dim;
+  const bf16 *src = a.conv + r0 * a.channels + grp * a.dim;
   const int pieces = a.dim >> 3;
   for (int i = tid; i < CH * pieces; i += PREP_THREADS) {
     const int t = i / pieces, c = (i - t * pieces) * 8;
@@ -116,164 +126,192 @@ delta_prepare_kernel(ChunkArgs a, const bf16 *conv, bf16 *mats, float4 *factors)
     copy16(ks + t * pitch + c, row + a.groups * a.dim, t < nt);
   }
   copy_commit();
+  if (wid == 0) {  // sums of the decays' logarithms, two tokens per lane
+    double x[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int t = lane * 2 + i;
+      const float *row = p.ba + (r0 + t) * p.ba_ld + h;
+      x[i] = t < nt ? (double)delta_log_decay(row[a.heads], p.a_log[h], p.dt_bias[h]) : 0.0;
+      bs[t] = t < nt ? sigmoid_f32(row[0]) : 0.f;
+    }
+    double sum = x[0] + x[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const double y = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += y;
+    }
+    gs[lane * 2] = sum - x[1];
+    gs[lane * 2 + 1] = sum;
+  }
   copy_wait_all();
   __syncthreads();
+  const long long at = chunk_at(a, b, h, chunk);
   {  // one thread per row and kind
     const int t = tid & 63;
     const bf16 *row = (tid < 64 ? ks : qs) + t * pitch;
-    float s = 0.f;
+    float s0 = 0.f, s1 = 0.f;
+#pragma unroll 4
     for (int c = 0; c < a.dim; c += 8) {
       const uint4 u = *reinterpret_cast<const uint4 *>(row + c);
-      const unsigned w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-      for (int i = 0; i < 4; ++i) s += low_half(w[i]) * low_half(w[i]) + high_half(w[i]) * high_half(w[i]);
+      s0 += low_half(u.x) * low_half(u.x) + low_half(u.y) * low_half(u.y) + low_half(u.z) * low_half(u.z) + low_half(u.w) * low_half(u.w);
+      s1 += high_half(u.x) * high_half(u.x) + high_half(u.y) * high_half(u.y) + high_half(u.z) * high_half(u.z) +
+            high_half(u.w) * high_half(u.w);
     }
-    if (tid < 64) rk[t] = 1.0f / sqrtf(s + DELTA_UNIT_EPS);
-    else rq[t] = a.q_scale / sqrtf(s + DELTA_UNIT_EPS);
+    if (tid < 64) rk[t] = 1.0f / sqrtf(s0 + s1 + DELTA_UNIT_EPS);
+    else rq[t] = p.q_scale / sqrtf(s0 + s1 + DELTA_UNIT_EPS);
   }
+  __syncthreads();
+  if (tid < CH) {
+    const double last = gs[CH - 1];
+    const float e = expf((float)gs[tid]);
+    a.factors[at * CH + tid] = make_float4(e * rk[tid], e * rq[tid], expf((float)(last - gs[tid])) * rk[tid], expf((float)last));
+  }
+  bf16 *mat = a.mats + at * 4 * MAT;
   // products of the warp's 16 rows with the tokens up to its last row
   const int w0 = wid * 16;
-  float kk[8][4], qk[8][4];
-#pragma unroll
-  for (int i = 0; i < 8; ++i)
-#pragma unroll
-    for (int j = 0; j < 4; ++j) kk[i][j] = qk[i][j] = 0.f;
   const int ar = w0 + (lane & 15), ac = (lane >> 4) * 8;                        // left operand's row and column
   const int br = (lane & 7) + ((lane >> 4) << 3), bc = ((lane >> 3) & 1) * 8;  // right operand: two tiles of 8 tokens
-  for (int c = 0; c < a.dim; c += 16) {
-    unsigned ak[4], aq[4];
-    ldmatrix4(ak, ks + ar * pitch + c + ac);
-    ldmatrix4(aq, qs + ar * pitch + c + ac);
+  float acc[8][4];
+  auto product = [&](const bf16 *left) {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      if (j > wid) break;
-      unsigned bk[4];
-      ldmatrix4(bk, ks + (j * 16 + br) * pitch + c + bc);
-      mma(kk[2 * j], ak, bk[0], bk[1]);
-      mma(kk[2 * j + 1], ak, bk[2], bk[3]);
-      mma(qk[2 * j], aq, bk[0], bk[1]);
-      mma(qk[2 * j + 1], aq, bk[2], bk[3]);
-    }
-  }
-  const int per = a.heads / a.groups;
-  for (int hh = 0; hh < per; ++hh) {
-    const int h = grp * per + hh;
-    const long long at = chunk_at(a, b, h, chunk);
-    __syncthreads();  // norms are there; the previous head is done with ls, ts and the factors
-    if (wid == 0) {  // sums of the decays' logarithms, two tokens per lane
-      double x[2];
+    for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = lane * 2 + i;
-        const float *row = a.ba + (r0 + t) * a.ba_ld + h;
-        x[i] = t < nt ? (double)delta_log_decay(row[a.heads], a.a_log[h], a.dt_bias[h]) : 0.0;
-        bs[t] = t < nt ? sigmoid_f32(row[0]) : 0.f;
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+#pragma unroll 2
+    for (int c = 0; c < a.dim; c += 16) {
+      unsigned x[4];
+      ldmatrix4(x, left + ar * pitch + c + ac);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        if (j <= wid) {
+          unsigned y[4];
+          ldmatrix4(y, ks + (j * 16 + br) * pitch + c + bc);
+          mma(acc[2 * j], x, y[0], y[1]);
+          mma(acc[2 * j + 1], x, y[2], y[3]);
+        }
       }
-      double sum = x[0] + x[1];
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const double y = __shfl_up_sync(0xffffffffu, sum, o);
-        if (lane >= o) sum += y;
-      }
-      gs[lane * 2] = sum - x[1];
-      gs[lane * 2 + 1] = sum;
     }
-    __syncthreads();
-    const double last = gs[CH - 1];
-    if (tid < CH) {
-      const float e = expf((float)gs[tid]);
-      factors[at * CH + tid] = make_float4(e * rk[tid], e * rq[tid], expf((float)(last - gs[tid])) * rk[tid], expf((float)last));
-    }
-    bf16 *mat = mats + at * 4 * MAT;
+  };
+  const double gi[2] = {gs[w0 + g], gs[w0 + g + 8]};
+  const float ri[2] = {rk[w0 + g] * bs[w0 + g], rk[w0 + g + 8] * bs[w0 + g + 8]}, qi[2] = {rq[w0 + g], rq[w0 + g + 8]};
+  product(qs);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      if (j > 2 * wid + 1) break;
+  for (int j = 0; j < 8; ++j) {
+    if (j <= 2 * wid + 1) {
+      const int col = j * 8 + t2;
+      const double g0 = gs[col], g1 = gs[col + 1];
+      const float r0k = rk[col], r1k = rk[col + 1];
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int i = w0 + g + half * 8;
-        float e[2], av[2];
-#pragma unroll
-        for (int k = 0; k < 2; ++k) {
-          const int col = j * 8 + t2 + k;
-          e[k] = col <= i ? expf((float)(gs[i] - gs[col])) * rk[col] : 0.f;
-          av[k] = e[k] * rq[i] * qk[j][half * 2 + k];
-          ls[i * TP + col] = col < i ? e[k] * bs[i] * rk[i] * kk[j][half * 2 + k] : 0.f;
-        }
+        const float v0 = col <= i ? expf((float)(gi[half] - g0)) * r0k * qi[half] * acc[j][half * 2] : 0.f;
+        const float v1 = col + 1 <= i ? expf((float)(gi[half] - g1)) * r1k * qi[half] * acc[j][half * 2 + 1] : 0.f;
         unsigned hi, lo;
-        split(av[0], av[1], hi, lo);
-        *reinterpret_cast<unsigned *>(mat + 2 * MAT + i * CH + j * 8 + t2) = hi;
-        *reinterpret_cast<unsigned *>(mat + 3 * MAT + i * CH + j * 8 + t2) = lo;
+        split(v0, v1, hi, lo);
+        *reinterpret_cast<unsigned *>(mat + 2 * MAT + i * CH + col) = hi;
+        *reinterpret_cast<unsigned *>(mat + 3 * MAT + i * CH + col) = lo;
       }
     }
+  }
+  product(ks);
+  __syncthreads();  // the vectors are read
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    if (j <= 2 * wid + 1) {
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int col = j * 8 + t2 + k;
+        const double gc = gs[col];
+        const float rc = rk[col];
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int i = w0 + g + half * 8;
+          lt[col * TP + i] = col < i ? expf((float)(gi[half] - gc)) * rc * ri[half] * acc[j][half * 2 + k] : 0.f;
+        }
+      }
+    }
+  }
+  __syncthreads();
+  // inverse of I + L: the two diagonal blocks of 32 by substitution, one column per lane; a solved entry is taken out of
+  // all later ones at once
+  if (wid < 2) {
+    const float *lb = lt + wid * 32 * TP + wid * 32;
+    float x[32];
+#pragma unroll
+    for (int i = 0; i < 32; ++i) x[i] = i == lane ? 1.f : 0.f;
+#pragma unroll
+    for (int j = 0; j < 31; ++j) {
+#pragma unroll
+      for (int i = j / 4 * 4; i < 32; i += 4) {
+        const float4 l = *reinterpret_cast<const float4 *>(lb + j * TP + i);
+        if (i > j) x[i] = fmaf(-l.x, x[j], x[i]);
+        if (i + 1 > j) x[i + 1] = fmaf(-l.y, x[j], x[i + 1]);
+        if (i + 2 > j) x[i + 2] = fmaf(-l.z, x[j], x[i + 2]);
+        if (i + 3 > j) x[i + 3] = fmaf(-l.w, x[j], x[i + 3]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 32; ++i) ts[(wid * 32 + i) * TP + wid * 32 + lane] = x[i];
+  }
+  __syncthreads();
+  {  // the block below them: -(second inverse) L21 (first inverse); the upper right block holds L21 (first inverse)
+    const int r = tid >> 2, c = (tid & 3) * 8;
+    float m[8] = {};
+#pragma unroll 8
+    for (int j = 0; j < 32; ++j) {
+      const float l = lt[j * TP + 32 + r];
+      const float4 x = *reinterpret_cast<const float4 *>(ts + j * TP + c), y = *reinterpret_cast<const float4 *>(ts + j * TP + c + 4);
+      m[0] = fmaf(l, x.x, m[0]);
+      m[1] = fmaf(l, x.y, m[1]);
+      m[2] = fmaf(l, x.z, m[2]);
+      m[3] = fmaf(l, x.w, m[3]);
+      m[4] = fmaf(l, y.x, m[4]);
+      m[5] = fmaf(l, y.y, m[5]);
+      m[6] = fmaf(l, y.z, m[6]);
+      m[7] = fmaf(l, y.w, m[7]);
+    }
+    *reinterpret_cast<float4 *>(ts + r * TP + 32 + c) = make_float4(m[0], m[1], m[2], m[3]);
+    *reinterpret_cast<float4 *>(ts + r * TP + 32 + c + 4) = make_float4(m[4], m[5], m[6], m[7]);
     __syncthreads();
-    // inverse of I + L: the two diagonal blocks of 32 by forward substitution, one column per lane
-    if (wid < 2) {
-      const float *lb = ls + wid * 32 * TP + wid * 32;
-      float x[32];
-#pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        float s = i == lane ? 1.f : 0.f;
-#pragma unroll
-        for (int j = 0; j < i; ++j) s = fmaf(-lb[i * TP + j], x[j], s);
-        x[i] = s;
-      }
-#pragma unroll
-      for (int i = 0; i < 32; ++i) ts[(wid * 32 + i) * TP + wid * 32 + lane] = x[i];
+    float n[8] = {};
+#pragma unroll 8
+    for (int j = 0; j < 32; ++j) {
+      const float l = -ts[(32 + r) * TP + 32 + j];
+      const float *row = ts + j * TP + 32 + c;
+      const float4 x = *reinterpret_cast<const float4 *>(row), y = *reinterpret_cast<const float4 *>(row + 4);
+      n[0] = fmaf(l, x.x, n[0]);
+      n[1] = fmaf(l, x.y, n[1]);
+      n[2] = fmaf(l, x.z, n[2]);
+      n[3] = fmaf(l, x.w, n[3]);
+      n[4] = fmaf(l, y.x, n[4]);
+      n[5] = fmaf(l, y.y, n[5]);
+      n[6] = fmaf(l, y.z, n[6]);
+      n[7] = fmaf(l, y.w, n[7]);
     }
-    __syncthreads();
-    {  // the block below them: -(second inverse) L21 (first inverse); the upper right block holds L21 (first inverse)
-      const int r = tid >> 2, c = (tid & 3) * 8;
-      float m[8] = {};
-      for (int j = 0; j < 32; ++j) {
-        const float l = ls[(32 + r) * TP + j];
-        const float4 x = *reinterpret_cast<const float4 *>(ts + j * TP + c), y = *reinterpret_cast<const float4 *>(ts + j * TP + c + 4);
-        m[0] = fmaf(l, x.x, m[0]);
-        m[1] = fmaf(l, x.y, m[1]);
-        m[2] = fmaf(l, x.z, m[2]);
-        m[3] = fmaf(l, x.w, m[3]);
-        m[4] = fmaf(l, y.x, m[4]);
-        m[5] = fmaf(l, y.y, m[5]);
-        m[6] = fmaf(l, y.z, m[6]);
-        m[7] = fmaf(l, y.w, m[7]);
-      }
+    *reinterpret_cast<float4 *>(ts + (32 + r) * TP + c) = make_float4(n[0], n[1], n[2], n[3]);
+    *reinterpret_cast<float4 *>(ts + (32 + r) * TP + c + 4) = make_float4(n[4], n[5], n[6], n[7]);
+  }
+  __syncthreads();
+  for (int i = tid; i < CH * (CH / 8); i += PREP_THREADS) {
+    const int r = i >> 3, c = (i & 7) * 8;
+    if (c >= (r / 16 + 1) * 16) continue;
+    const float *row = ts + r * TP + c;
+    const float4 x = *reinterpret_cast<const float4 *>(row), y = *reinterpret_cast<const float4 *>(row + 4);
+    const float e[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
+    unsigned hi[4], lo[4];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) ts[r * TP + 32 + c + i] = m[i];
-      __syncthreads();
-      float n[8] = {};
-      for (int j = 0; j < 32; ++j) {
-        const float l = -ts[(32 + r) * TP + 32 + j];
-        const float *row = ts + j * TP + 32 + c;
-        const float4 x = *reinterpret_cast<const float4 *>(row), y = *reinterpret_cast<const float4 *>(row + 4);
-        n[0] = fmaf(l, x.x, n[0]);
-        n[1] = fmaf(l, x.y, n[1]);
-        n[2] = fmaf(l, x.z, n[2]);
-        n[3] = fmaf(l, x.w, n[3]);
-        n[4] = fmaf(l, y.x, n[4]);
-        n[5] = fmaf(l, y.y, n[5]);
-        n[6] = fmaf(l, y.z, n[6]);
-        n[7] = fmaf(l, y.w, n[7]);
-      }
-#pragma unroll
-      for (int i = 0; i < 8; ++i) ts[(32 + r) * TP + c + i] = n[i];
+    for (int k = 0; k < 4; ++k) {
+      const int c0 = c + 2 * k, c1 = c0 + 1;
+      split(c0 <= r ? e[2 * k] * bs[c0] : 0.f, c1 <= r ? e[2 * k + 1] * bs[c1] : 0.f, hi[k], lo[k]);
     }
-    __syncthreads();
-    for (int i = tid; i < CH * (CH / 8); i += PREP_THREADS) {
-      const int r = i >> 3, c = (i & 7) * 8;
-      if (c >= (r / 16 + 1) * 16) continue;
-      unsigned hi[4], lo[4];
-#pragma unroll
-      for (int k = 0; k < 4; ++k) {
-        const int c0 = c + 2 * k, c1 = c0 + 1;
-        split(c0 <= r ? ts[r * TP + c0] * bs[c0] : 0.f, c1 <= r ? ts[r * TP + c1] * bs[c1] : 0.f, hi[k], lo[k]);
-      }
-      *reinterpret_cast<uint4 *>(mat + r * CH + c) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-      *reinterpret_cast<uint4 *>(mat + MAT + r * CH + c) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-    }
+    *reinterpret_cast<uint4 *>(mat + r * CH + c) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    *reinterpret_cast<uint4 *>(mat + MAT + r * CH + c) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
   }
 }
 
 struct ScanArgs {
-  ChunkArgs c;
+  DeltaChunks c;
   int p0, slot0, stages;
   float *state, *o;
   const bf16 *gate;
@@ -292,10 +330,10 @@ __host__ __device__ __forceinline__ int stage_elems(int dim, int vt) {
 // with keys and with queries one after the other (fewer registers).
 template <int NT, int WARPS, bool TWO_PASS>
 __global__ void __launch_bounds__(WARPS * 32)
-delta_scan_kernel(ScanArgs s, const bf16 *conv, const bf16 *mats, const float4 *factors) {
+delta_scan_kernel(ScanArgs s) {
   constexpr int THREADS = WARPS * 32, VT = WARPS * 16, SP = VT + 4;
   extern __shared__ __align__(16) unsigned char raw[];
-  const ChunkArgs &a = s.c;
+  const DeltaChunks &a = s.c;
   const int pitch = a.dim + 8, vp = VT + 8, elems = stage_elems(a.dim, VT);
   bf16 *stages = reinterpret_cast<bf16 *>(raw);
   float *stage_o = reinterpret_cast<float *>(stages + (size_t)s.stages * elems);  // [64][SP] outputs of the chunk
@@ -306,7 +344,7 @@ delta_scan_kernel(ScanArgs s, const bf16 *conv, const bf16 *mats, const float4 *
   const int h = blockIdx.x / tiles, vt = (blockIdx.x - h * tiles) * VT, b = blockIdx.y;
   const int grp = h / (a.heads / a.groups);
   const int cols = min(VT, a.vdim - vt);
-  const bf16 *base = conv + (long long)b * a.n * a.channels;
+  const bf16 *base = a.conv + (long long)b * a.n * a.channels;
   const int q_at = grp * a.dim, k_at = (a.groups + grp) * a.dim, v_at = 2 * a.groups * a.dim + h * a.vdim + vt;
   auto load = [&](int chunk) {
     bf16 *ks = stages + (size_t)(chunk % s.stages) * elems, *qs = ks + CH * pitch, *vs = qs + CH * pitch, *ms = vs + CH * vp;
@@ -327,9 +365,9 @@ delta_scan_kernel(ScanArgs s, const bf16 *conv, const bf16 *mats, const float4 *
     const long long at = chunk_at(a, b, h, chunk);
     for (int i = tid; i < 4 * CH * 8; i += THREADS) {
       const int m = i >> 9, r = (i >> 3) & 63, c = (i & 7) * 8;
-      if (c < (r / 16 + 1) * 16) copy16(ms + (m * CH + r) * MP + c, mats + (at * 4 + m) * MAT + r * CH + c, true);
+      if (c < (r / 16 + 1) * 16) copy16(ms + (m * CH + r) * MP + c, a.mats + (at * 4 + m) * MAT + r * CH + c, true);
     }
-    for (int i = tid; i < CH; i += THREADS) copy16(fs + i, factors + at * CH + i, true);
+    for (int i = tid; i < CH; i += THREADS) copy16(fs + i, a.factors + at * CH + i, true);
     copy_commit();
   };
   load(0);
@@ -362,24 +400,17 @@ delta_scan_kernel(ScanArgs s, const bf16 *conv, const bf16 *mats, const float4 *
 #pragma unroll
     for (int kt = 0; kt < NT / 2; ++kt) {
       if (kt * 16 < a.dim) {
-        unsigned hi[4], lo[4];
+        unsigned hi[4], lo[4], x[4][4], y[4][4];
         operand(st[2 * kt], st[2 * kt + 1], hi, lo);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          unsigned x[4];
-          ldmatrix4(x, ks + (j * 16 + br) * pitch + kt * 16 + bc);
-          mma(pk[2 * j], lo, x[0], x[1]);
-          mma(pk[2 * j + 1], lo, x[2], x[3]);
-          mma(pk[2 * j], hi, x[0], x[1]);
-          mma(pk[2 * j + 1], hi, x[2], x[3]);
-          if (!TWO_PASS) {
-            ldmatrix4(x, qs + (j * 16 + br) * pitch + kt * 16 + bc);
-            mma(pq[2 * j], lo, x[0], x[1]);
-            mma(pq[2 * j + 1], lo, x[2], x[3]);
-            mma(pq[2 * j], hi, x[0], x[1]);
-            mma(pq[2 * j + 1], hi, x[2], x[3]);
-          }
+          ldmatrix4(x[j], ks + (j * 16 + br) * pitch + kt * 16 + bc);
+          if (!TWO_PASS) ldmatrix4(y[j], qs + (j * 16 + br) * pitch + kt * 16 + bc);
         }
+        terms(pk, lo, x);  // products that add to one accumulator stand far apart
+        if (!TWO_PASS) terms(pq, lo, y);
+        terms(pk, hi, x);
+        if (!TWO_PASS) terms(pq, hi, y);
       }
     }
     // right-hand side V^T - e^G r (S^T K'^T)
@@ -406,36 +437,27 @@ delta_scan_kernel(ScanArgs s, const bf16 *conv, const bf16 *mats, const float4 *
       for (int j = 0; j < 4; ++j) u[i][j] = 0.f;
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
-      unsigned hi[4], lo[4];
+      unsigned hi[4], lo[4], x[4][4], y[4][4];
       operand(pk[2 * kt], pk[2 * kt + 1], hi, lo);
 #pragma unroll
       for (int j = kt; j < 4; ++j) {
-        unsigned x[4], y[4];
-        ldmatrix4(x, ms + (j * 16 + br) * MP + kt * 16 + bc);
-        ldmatrix4(y, ms + (CH + j * 16 + br) * MP + kt * 16 + bc);
-        mma(u[2 * j], lo, x[0], x[1]);
-        mma(u[2 * j + 1], lo, x[2], x[3]);
-        mma(u[2 * j], hi, y[0], y[1]);
-        mma(u[2 * j + 1], hi, y[2], y[3]);
-        mma(u[2 * j], hi, x[0], x[1]);
-        mma(u[2 * j + 1], hi, x[2], x[3]);
+        ldmatrix4(x[j], ms + (j * 16 + br) * MP + kt * 16 + bc);
+        ldmatrix4(y[j], ms + (CH + j * 16 + br) * MP + kt * 16 + bc);
       }
+      terms(u, lo, x, kt);
+      terms(u, hi, y, kt);
+      terms(u, hi, x, kt);
     }
     if (TWO_PASS) {
 #pragma unroll
       for (int kt = 0; kt < NT / 2; ++kt) {
         if (kt * 16 < a.dim) {
-          unsigned hi[4], lo[4];
+          unsigned hi[4], lo[4], x[4][4];
           operand(st[2 * kt], st[2 * kt + 1], hi, lo);
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            unsigned x[4];
-            ldmatrix4(x, qs + (j * 16 + br) * pitch + kt * 16 + bc);
-            mma(pq[2 * j], lo, x[0], x[1]);
-            mma(pq[2 * j + 1], lo, x[2], x[3]);
-            mma(pq[2 * j], hi, x[0], x[1]);
-            mma(pq[2 * j + 1], hi, x[2], x[3]);
-          }
+          for (int j = 0; j < 4; ++j) ldmatrix4(x[j], qs + (j * 16 + br) * pitch + kt * 16 + bc);
+          terms(pq, lo, x);
+          terms(pq, hi, x);
         }
       }
     }
@@ -450,20 +472,16 @@ delta_scan_kernel(ScanArgs s, const bf16 *conv, const bf16 *mats, const float4 *
     }
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
-      unsigned hi[4], lo[4];
+      unsigned hi[4], lo[4], x[4][4], y[4][4];
       operand(u[2 * kt], u[2 * kt + 1], hi, lo);
 #pragma unroll
       for (int j = kt; j < 4; ++j) {
-        unsigned x[4], y[4];
-        ldmatrix4(x, ms + (2 * CH + j * 16 + br) * MP + kt * 16 + bc);
-        ldmatrix4(y, ms + (3 * CH + j * 16 + br) * MP + kt * 16 + bc);
-        mma(pq[2 * j], lo, x[0], x[1]);
-        mma(pq[2 * j + 1], lo, x[2], x[3]);
-        mma(pq[2 * j], hi, y[0], y[1]);
-        mma(pq[2 * j + 1], hi, y[2], y[3]);
-        mma(pq[2 * j], hi, x[0], x[1]);
-        mma(pq[2 * j + 1], hi, x[2], x[3]);
+        ldmatrix4(x[j], ms + (2 * CH + j * 16 + br) * MP + kt * 16 + bc);
+        ldmatrix4(y[j], ms + (3 * CH + j * 16 + br) * MP + kt * 16 + bc);
       }
+      terms(pq, lo, x, kt);
+      terms(pq, hi, y, kt);
+      terms(pq, hi, x, kt);
     }
     // S^T <- e^G_last S^T + (U^T diag(e^(G_last - G) r)) K'
     const float keep = fs[0].w;
@@ -484,15 +502,19 @@ delta_scan_kernel(ScanArgs s, const bf16 *conv, const bf16 *mats, const float4 *
       unsigned hi[4], lo[4];
       operand(u[2 * kt], u[2 * kt + 1], hi, lo);
 #pragma unroll
-      for (int i = 0; i < NT / 2; ++i) {
-        if (i * 16 < a.dim) {
-          unsigned x[4];
-          ldmatrix4_trans(x, ks + (kt * 16 + tr) * pitch + i * 16 + tc);
-          mma(st[2 * i], lo, x[0], x[1]);
-          mma(st[2 * i + 1], lo, x[2], x[3]);
-          mma(st[2 * i], hi, x[0], x[1]);
-          mma(st[2 * i + 1], hi, x[2], x[3]);
-        }
+      for (int i = 0; i < NT / 2; i += 4) {
+        unsigned x[4][4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if ((i + j) * 16 < a.dim) ldmatrix4_trans(x[j], ks + (kt * 16 + tr) * pitch + (i + j) * 16 + tc);
+#pragma unroll
+        for (int term = 0; term < 2; ++term)
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if ((i + j) * 16 < a.dim) {
+              mma(st[2 * (i + j)], term ? hi : lo, x[j][0], x[j][1]);
+              mma(st[2 * (i + j) + 1], term ? hi : lo, x[j][2], x[j][3]);
+            }
       }
     }
     // the chunk's outputs as whole rows
@@ -561,12 +583,9 @@ size_t delta_chunk_bytes(const DeltaMixer &m, long long rows, int streams) {
 }
 
 int launch_delta_chunks(const DeltaMixer &m, const void *conv, float *o, void *scratch, const RowBatch &b, bool *normed,
-                        cudaStream_t st) {
+                        cudaStream_t st, DevErr *err) {
   const Parts part = parts(m, b.rows(), b.streams);
-  bf16 *mats = static_cast<bf16 *>(scratch);
-  float4 *factors = reinterpret_cast<float4 *>(static_cast<char *>(scratch) + part.mats);
-  const bf16 *rows = static_cast<const bf16 *>(conv);
-  ChunkArgs c{};
+  DeltaChunks c{};
   c.heads = m.heads;
   c.groups = m.groups;
   c.dim = m.dim;
@@ -574,15 +593,19 @@ int launch_delta_chunks(const DeltaMixer &m, const void *conv, float *o, void *s
   c.channels = m.conv_channels();
   c.n = b.n;
   c.chunks = (b.n + CH - 1) / CH;
-  c.q_scale = 1.0f / sqrtf((float)m.true_dim);
-  c.a_log = m.a_log;
-  c.dt_bias = m.dt_bias;
-  c.ba = m.ba;
-  c.ba_ld = m.ba_ld;
-  const size_t prep_smem = (size_t)2 * CH * (m.dim + 8) * 2 + (size_t)2 * CH * TP * 4;
+  c.conv = static_cast<const bf16 *>(conv);
+  c.mats = static_cast<bf16 *>(scratch);
+  c.factors = reinterpret_cast<float4 *>(static_cast<char *>(scratch) + part.mats);
+  const PrepareArgs p{c, 1.0f / sqrtf((float)m.true_dim), m.a_log, m.dt_bias, m.ba, m.ba_ld};
+  const size_t vectors = (size_t)2 * CH * (m.dim + 8) * 2, floats = (size_t)2 * CH * TP * 4;
+  const size_t prep_smem = vectors > floats ? vectors : floats;
   LB_CUDA(cudaFuncSetAttribute(delta_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem));
-  launch_pdl(delta_prepare_kernel, dim3((unsigned)c.chunks, (unsigned)m.groups, (unsigned)b.streams), dim3(PREP_THREADS),
-             prep_smem, st, g_pdl_enabled, c, rows, mats, factors);
+  launch_pdl(delta_prepare_kernel, dim3((unsigned)c.chunks, (unsigned)m.heads, (unsigned)b.streams), dim3(PREP_THREADS),
+             prep_smem, st, g_pdl_enabled, p);
+  if (delta_scan_tc_supports(m)) {
+    *normed = launch_delta_scan_tc(m, c, o, b, st, err);
+    return 2;
+  }
   ScanArgs s{};
   s.c = c;
   s.p0 = b.p0;
@@ -608,7 +631,7 @@ int launch_delta_chunks(const DeltaMixer &m, const void *conv, float *o, void *s
     const size_t smem = s.stages * stage + extra;
     LB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     launch_pdl(kernel, dim3((unsigned)(m.heads * ((m.vdim + vt - 1) / vt)), (unsigned)b.streams), dim3((unsigned)(warps * 32)),
-               smem, st, g_pdl_enabled, s, rows, (const bf16 *)mats, (const float4 *)factors);
+               smem, st, g_pdl_enabled, s);
   };
   if (m.dim <= 64) {
     if (vt == 128) scan(delta_scan_kernel<8, 8, false>, 8);

@@ -323,6 +323,7 @@ int litnice_b200_delta_host(int32_t dtype, const float *rows, const float *ba, c
     const Precision type = dtype == LITNICE_B200_DTYPE_F32 ? Precision::F32 : Precision::BF16;
     const size_t es = type == Precision::BF16 ? 2 : 4;
     Dev dev;
+    ErrWord err;
     DeltaMixer m{};
     m.heads = heads;
     m.groups = groups;
@@ -377,8 +378,9 @@ int litnice_b200_delta_host(int32_t dtype, const float *rows, const float *ba, c
       m.ba = static_cast<float *>(put(dev, gates.data(), b.rows(), 2 * heads, 2 * heads, Precision::F32));
       m.out = dev.alloc((size_t)b.rows() * m.out_ld * es);
       void *scratch = dev.alloc(delta_scratch_bytes(m, b.rows(), n_streams, type));
-      launch_delta(m, scratch, type, b, nullptr);
+      launch_delta(m, scratch, type, b, nullptr, err.dev);
       LB_CUDA(cudaDeviceSynchronize());
+      if (err.host->code != DEVERR_NONE) return LITNICE_B200_EDEVICE;
       std::vector<float> o((size_t)b.rows() * m.out_ld);
       get(m.out, b.rows(), m.out_ld, m.out_ld, type, o.data());
       for (int st = 0; st < n_streams; ++st)

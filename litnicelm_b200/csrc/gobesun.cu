@@ -441,7 +441,7 @@ class Gobesun final : public DecoderModel {
     m.ba_ld = half ? 2 * l.heads : m.in_ld;
     m.out = mix_.p;
     m.out_ld = l.o_cols();
-    launches_ += launch_delta(m, delta_.p, prec_, b, st);
+    launches_ += launch_delta(m, delta_.p, prec_, b, st, err);
   }
 
   void attention(const Layer &l, Run &r, const RowBatch &b, cudaStream_t st, DevErr *err) {

@@ -90,8 +90,9 @@ struct RowsShape {
   }
 };
 
-// One CTA per row. Shared memory: the row's queries and keys in 32-bit, then cosines and sines.
-template <typename T>
+// One CTA per row. Shared memory: the row's queries and keys times their weights in 32-bit, then cosines and sines.
+// FOUR: four neighbouring coordinates rotate (or pass) alike and stay within one half (rot.dims % 8 == 0).
+template <typename T, bool FOUR>
 __global__ void __launch_bounds__(GA_THREADS)
 qk_norm_rotate_kernel(const T *src, int ld, const float *__restrict__ q_weight, const float *__restrict__ k_weight, float eps,
                       int q_cols, int k_cols, int v_cols, int dim, float q_count, float k_count, Rotation rot, T *q, int q_ld,
@@ -113,13 +114,15 @@ qk_norm_rotate_kernel(const T *src, int ld, const float *__restrict__ q_weight, 
   for (int c = tid * P; c < cols; c += GA_THREADS * P) {
     Piece<T> v;
     v.load(x + c);
+    const float *w = c < q_cols ? q_weight + c : k_weight + (c - q_cols);
     float f[P];
     v.unpack(f);
     float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < P; ++i) {
-      s = fmaf(f[i], f[i], s);
-      row[c + i] = f[i];
+    for (int i = 0; i < P; i += 4) {
+      const float4 y = *reinterpret_cast<const float4 *>(w + i);
+      s = fmaf(f[i], f[i], fmaf(f[i + 1], f[i + 1], fmaf(f[i + 2], f[i + 2], fmaf(f[i + 3], f[i + 3], s))));
+      *reinterpret_cast<float4 *>(row + c + i) = make_float4(f[i] * y.x, f[i + 1] * y.y, f[i + 2] * y.z, f[i + 3] * y.w);
     }
     if (c < q_cols) sq += s;
     else sk += s;
@@ -129,7 +132,7 @@ qk_norm_rotate_kernel(const T *src, int ld, const float *__restrict__ q_weight, 
     v.load(x + cols + c);
     *reinterpret_cast<decltype(v.u) *>(v_cache + at * v_cols + c) = v.u;
   }
-  for (int i = tid; i < half; i += GA_THREADS) {
+  for (int i = GA_THREADS - 1 - tid; i < half; i += GA_THREADS) {  // the last threads have the fewest pieces
     double t = (double)p * rot.turns[i];
     t -= 2.0 * rint(0.5 * t);
     float s, c;
@@ -151,25 +154,33 @@ qk_norm_rotate_kernel(const T *src, int ld, const float *__restrict__ q_weight, 
     sk += part[1][i];
   }
   const float iq = 1.0f / sqrtf(sq / q_count + eps), ik = 1.0f / sqrtf(sk / k_count + eps);
+  auto four = [](const float *s) { return *reinterpret_cast<const float4 *>(s); };
   for (int c = tid * P; c < cols; c += GA_THREADS * P) {
     const bool is_q = c < q_cols;
     const float inv = is_q ? iq : ik;
-    const int base = is_q ? 0 : q_cols;
-    const float *w = (is_q ? q_weight : k_weight) - base;
-    const int e0 = (c - base) % dim, h0 = c - e0;  // head's first column
+    const int e0 = (is_q ? c : c - q_cols) % dim, h0 = c - e0;  // head's first column
     float f[P];
 #pragma unroll
-    for (int i = 0; i < P; ++i) {
+    for (int i = 0; i < P; i += FOUR ? 4 : 1) {
       const int e = e0 + i;
-      const float own = row[h0 + e] * inv * w[h0 + e];
-      if (e < half) {
-        const float other = row[h0 + e + half] * inv * w[h0 + e + half];
-        f[i] = own * cs[e] - other * sn[e];
-      } else if (e < 2 * half) {
-        const float other = row[h0 + e - half] * inv * w[h0 + e - half];
-        f[i] = own * cs[e - half] + other * sn[e - half];
+      if constexpr (FOUR) {
+        float4 v = four(row + h0 + e);
+        if (e < 2 * half) {
+          const bool low = e < half;
+          const float4 w = four(row + h0 + (low ? e + half : e - half)), y = four(cs + (low ? e : e - half));
+          float4 z = four(sn + (low ? e : e - half));
+          if (low) z = make_float4(-z.x, -z.y, -z.z, -z.w);
+          v = make_float4(v.x * y.x + w.x * z.x, v.y * y.y + w.y * z.y, v.z * y.z + w.z * z.z, v.w * y.w + w.w * z.w);
+        }
+        f[i] = v.x * inv;
+        f[i + 1] = v.y * inv;
+        f[i + 2] = v.z * inv;
+        f[i + 3] = v.w * inv;
       } else {
-        f[i] = own;
+        float v = row[h0 + e];
+        if (e < half) v = v * cs[e] - row[h0 + e + half] * sn[e];
+        else if (e < 2 * half) v = v * cs[e - half] + row[h0 + e - half] * sn[e - half];
+        f[i] = v * inv;
       }
     }
     Piece<T>::store(is_q ? q + r * q_ld + c : k_cache + at * k_cols + (c - q_cols), f);
@@ -379,7 +390,7 @@ void norm_rotate_t(const void *src, int ld, const float *qw, const float *kw, fl
                    const GroupedAttention &a, void *q, const RowBatch &b, cudaStream_t st) {
   const int qc = a.heads * a.dim, kc = a.groups * a.dim;
   const size_t smem = (size_t)(qc + kc + rot.dims) * sizeof(float);
-  auto kernel = qk_norm_rotate_kernel<T>;
+  auto kernel = rot.dims % 8 == 0 ? qk_norm_rotate_kernel<T, true> : qk_norm_rotate_kernel<T, false>;
   if (smem > 40 * 1024) LB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   launch_pdl(kernel, dim3((unsigned)b.rows()), dim3(GA_THREADS), smem, st, g_pdl_enabled, static_cast<const T *>(src), ld, qw,
              kw, eps, qc, kc, a.groups * a.vdim, a.dim, (float)(a.heads * true_dim), (float)(a.groups * true_dim), rot,

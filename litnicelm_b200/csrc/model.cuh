@@ -249,7 +249,7 @@ struct DeltaMixer {
 // [rows][heads * vdim] float, and the chunked form's matrices.
 size_t delta_scratch_bytes(const DeltaMixer &m, long long rows, int streams, Precision type);
 // The new rows' recurrence and gated norm, state and history advanced; returns the kernels launched.
-int launch_delta(const DeltaMixer &m, void *scratch, Precision type, const RowBatch &b, cudaStream_t st);
+int launch_delta(const DeltaMixer &m, void *scratch, Precision type, const RowBatch &b, cudaStream_t st, DevErr *err);
 bool delta_supports(int dim, int vdim);
 
 // Activations of the products and of launch_activation_f32: GELU in its error-function and tanh forms.

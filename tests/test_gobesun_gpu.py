@@ -127,6 +127,8 @@ DELTA_SHAPES = [  # streams, n, heads, groups, dim, vdim, taps
     (1, 150, 2, 1, 256, 48, 4),
     (1, 33, 2, 2, 272, 80, 2),
     (8, 70, 12, 6, 32, 256, 3),
+    (2, 150, 3, 3, 80, 100, 3),
+    (1, 700, 2, 1, 128, 128, 4),
 ]
 
 
