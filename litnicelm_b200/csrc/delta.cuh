@@ -24,12 +24,12 @@ __device__ __forceinline__ float delta_log_decay(float a, float a_log, float dt_
 constexpr int DELTA_CHUNK = 64;  // tokens per chunk of the chunked form
 
 // What the scan of a portion's chunks reads: the convolved rows [rows][channels], and per stream, head and chunk the
-// matrices [inverse high, low, A high, low][64][64] and a token's factors {e^G r, e^G r', e^(G_last - G) r, e^G_last}.
+// matrices [inverse high, low, A high, low][64][64] and the tokens' factors [e^G r, e^G r', e^(G_last - G) r, e^G_last][64].
 struct DeltaChunks {
   int heads, groups, dim, vdim, channels, n, chunks;
   const __nv_bfloat16 *conv;
   __nv_bfloat16 *mats;
-  float4 *factors;
+  float *factors;
 };
 
 // delta_chunk.cu: the recurrence of many rows on bfloat16 in chunks of 64 tokens. conv: the convolved rows

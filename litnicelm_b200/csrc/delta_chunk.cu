@@ -87,6 +87,15 @@ __device__ __forceinline__ void terms(float (&acc)[8][4], const unsigned (&a)[4]
     }
 }
 
+constexpr double LOG2E = 1.4426950408889634;
+__device__ __forceinline__ float exp2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// Difference of two numbers in two terms each.
+__device__ __forceinline__ float apart(float2 a, float2 b) { return (a.x - b.x) + (a.y - b.y); }
+
 struct PrepareArgs {
   DeltaChunks c;
   float q_scale;
@@ -109,7 +118,7 @@ delta_prepare_kernel(PrepareArgs p) {
   bf16 *ks = reinterpret_cast<bf16 *>(raw), *qs = ks + CH * pitch;
   float *lt = reinterpret_cast<float *>(raw);  // [64][TP] L transposed, over the vectors once the products are done
   float *ts = lt + CH * TP;                    // [64][TP] its inverse
-  __shared__ double gs[CH];
+  __shared__ float2 gs[CH];  // sums of the decays' logarithms to base 2, in two terms
   __shared__ float rk[CH], rq[CH], bs[CH];
   pdl_launch_dependents();
   pdl_wait();
@@ -141,37 +150,53 @@ delta_prepare_kernel(PrepareArgs p) {
       const double y = __shfl_up_sync(0xffffffffu, sum, o);
       if (lane >= o) sum += y;
     }
-    gs[lane * 2] = sum - x[1];
-    gs[lane * 2 + 1] = sum;
+    auto two = [](double v) {
+      const float hi = (float)v;
+      return make_float2(hi, (float)(v - (double)hi));
+    };
+    gs[lane * 2] = two((sum - x[1]) * LOG2E);
+    gs[lane * 2 + 1] = two(sum * LOG2E);
   }
   copy_wait_all();
   __syncthreads();
   const long long at = chunk_at(a, b, h, chunk);
-  {  // one thread per row and kind
-    const int t = tid & 63;
-    const bf16 *row = (tid < 64 ? ks : qs) + t * pitch;
-    float s0 = 0.f, s1 = 0.f;
-#pragma unroll 4
-    for (int c = 0; c < a.dim; c += 8) {
-      const uint4 u = *reinterpret_cast<const uint4 *>(row + c);
-      s0 += low_half(u.x) * low_half(u.x) + low_half(u.y) * low_half(u.y) + low_half(u.z) * low_half(u.z) + low_half(u.w) * low_half(u.w);
-      s1 += high_half(u.x) * high_half(u.x) + high_half(u.y) * high_half(u.y) + high_half(u.z) * high_half(u.z) +
-            high_half(u.w) * high_half(u.w);
-    }
-    if (tid < 64) rk[t] = 1.0f / sqrtf(s0 + s1 + DELTA_UNIT_EPS);
-    else rq[t] = p.q_scale / sqrtf(s0 + s1 + DELTA_UNIT_EPS);
-  }
-  __syncthreads();
-  if (tid < CH) {
-    const double last = gs[CH - 1];
-    const float e = expf((float)gs[tid]);
-    a.factors[at * CH + tid] = make_float4(e * rk[tid], e * rq[tid], expf((float)(last - gs[tid])) * rk[tid], expf((float)last));
-  }
-  bf16 *mat = a.mats + at * 4 * MAT;
   // products of the warp's 16 rows with the tokens up to its last row
   const int w0 = wid * 16;
   const int ar = w0 + (lane & 15), ac = (lane >> 4) * 8;                        // left operand's row and column
   const int br = (lane & 7) + ((lane >> 4) << 3), bc = ((lane >> 3) & 1) * 8;  // right operand: two tiles of 8 tokens
+  {  // squares of the vectors' norms: the diagonals of the warp's own 16 by 16 blocks
+    float dk[2][4] = {}, dq[2][4] = {};
+#pragma unroll 2
+    for (int c = 0; c < a.dim; c += 16) {
+      unsigned x[4], y[4];
+      ldmatrix4(x, ks + ar * pitch + c + ac);
+      ldmatrix4(y, ks + (w0 + br) * pitch + c + bc);
+      mma(dk[0], x, y[0], y[1]);
+      mma(dk[1], x, y[2], y[3]);
+      ldmatrix4(x, qs + ar * pitch + c + ac);
+      ldmatrix4(y, qs + (w0 + br) * pitch + c + bc);
+      mma(dq[0], x, y[0], y[1]);
+      mma(dq[1], x, y[2], y[3]);
+    }
+    if ((g >> 1) == (lane & 3)) {
+      const bool odd = g & 1;
+      rk[w0 + g] = 1.0f / sqrtf((odd ? dk[0][1] : dk[0][0]) + DELTA_UNIT_EPS);
+      rk[w0 + g + 8] = 1.0f / sqrtf((odd ? dk[1][3] : dk[1][2]) + DELTA_UNIT_EPS);
+      rq[w0 + g] = p.q_scale / sqrtf((odd ? dq[0][1] : dq[0][0]) + DELTA_UNIT_EPS);
+      rq[w0 + g + 8] = p.q_scale / sqrtf((odd ? dq[1][3] : dq[1][2]) + DELTA_UNIT_EPS);
+    }
+  }
+  __syncthreads();
+  if (tid < CH) {
+    const float2 last = gs[CH - 1];
+    const float e = exp2_fast(gs[tid].x);
+    float *f = a.factors + at * 4 * CH + tid;
+    f[0] = e * rk[tid];
+    f[CH] = e * rq[tid];
+    f[2 * CH] = exp2_fast(apart(last, gs[tid])) * rk[tid];
+    f[3 * CH] = exp2_fast(last.x);
+  }
+  bf16 *mat = a.mats + at * 4 * MAT;
   float acc[8][4];
   auto product = [&](const bf16 *left) {
 #pragma unroll
@@ -193,20 +218,20 @@ delta_prepare_kernel(PrepareArgs p) {
       }
     }
   };
-  const double gi[2] = {gs[w0 + g], gs[w0 + g + 8]};
+  const float2 gi[2] = {gs[w0 + g], gs[w0 + g + 8]};
   const float ri[2] = {rk[w0 + g] * bs[w0 + g], rk[w0 + g + 8] * bs[w0 + g + 8]}, qi[2] = {rq[w0 + g], rq[w0 + g + 8]};
   product(qs);
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
     if (j <= 2 * wid + 1) {
       const int col = j * 8 + t2;
-      const double g0 = gs[col], g1 = gs[col + 1];
+      const float2 g0 = gs[col], g1 = gs[col + 1];
       const float r0k = rk[col], r1k = rk[col + 1];
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int i = w0 + g + half * 8;
-        const float v0 = col <= i ? expf((float)(gi[half] - g0)) * r0k * qi[half] * acc[j][half * 2] : 0.f;
-        const float v1 = col + 1 <= i ? expf((float)(gi[half] - g1)) * r1k * qi[half] * acc[j][half * 2 + 1] : 0.f;
+        const float v0 = col <= i ? exp2_fast(apart(gi[half], g0)) * r0k * qi[half] * acc[j][half * 2] : 0.f;
+        const float v1 = col + 1 <= i ? exp2_fast(apart(gi[half], g1)) * r1k * qi[half] * acc[j][half * 2 + 1] : 0.f;
         unsigned hi, lo;
         split(v0, v1, hi, lo);
         *reinterpret_cast<unsigned *>(mat + 2 * MAT + i * CH + col) = hi;
@@ -222,12 +247,12 @@ delta_prepare_kernel(PrepareArgs p) {
 #pragma unroll
       for (int k = 0; k < 2; ++k) {
         const int col = j * 8 + t2 + k;
-        const double gc = gs[col];
+        const float2 gc = gs[col];
         const float rc = rk[col];
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           const int i = w0 + g + half * 8;
-          lt[col * TP + i] = col < i ? expf((float)(gi[half] - gc)) * rc * ri[half] * acc[j][half * 2 + k] : 0.f;
+          lt[col * TP + i] = col < i ? exp2_fast(apart(gi[half], gc)) * rc * ri[half] * acc[j][half * 2 + k] : 0.f;
         }
       }
     }
@@ -321,7 +346,7 @@ struct ScanArgs {
   bf16 *out;
 };
 
-// Shared memory of a stage, in bfloat16 elements (the token factors, 64 float4, behind them).
+// Shared memory of a stage, in bfloat16 elements (the token factors, 256 floats, behind them).
 __host__ __device__ __forceinline__ int stage_elems(int dim, int vt) {
   return 2 * CH * (dim + 8) + CH * (vt + 8) + 4 * CH * MP + CH * 8;
 }
@@ -348,7 +373,7 @@ delta_scan_kernel(ScanArgs s) {
   const int q_at = grp * a.dim, k_at = (a.groups + grp) * a.dim, v_at = 2 * a.groups * a.dim + h * a.vdim + vt;
   auto load = [&](int chunk) {
     bf16 *ks = stages + (size_t)(chunk % s.stages) * elems, *qs = ks + CH * pitch, *vs = qs + CH * pitch, *ms = vs + CH * vp;
-    float4 *fs = reinterpret_cast<float4 *>(ms + 4 * CH * MP);
+    float *fs = reinterpret_cast<float *>(ms + 4 * CH * MP);
     const int t0 = chunk * CH, nt = min(CH, a.n - t0), pieces = a.dim >> 3;
     const bf16 *rows = base + (long long)t0 * a.channels;
     for (int i = tid; i < CH * pieces; i += THREADS) {
@@ -367,7 +392,7 @@ delta_scan_kernel(ScanArgs s) {
       const int m = i >> 9, r = (i >> 3) & 63, c = (i & 7) * 8;
       if (c < (r / 16 + 1) * 16) copy16(ms + (m * CH + r) * MP + c, a.mats + (at * 4 + m) * MAT + r * CH + c, true);
     }
-    for (int i = tid; i < CH; i += THREADS) copy16(fs + i, a.factors + at * CH + i, true);
+    for (int i = tid * 4; i < 4 * CH; i += THREADS * 4) copy16(fs + i, a.factors + at * 4 * CH + i, true);
     copy_commit();
   };
   load(0);
@@ -390,7 +415,7 @@ delta_scan_kernel(ScanArgs s) {
     if (s.stages > 1 && chunk + 1 < a.chunks) load(chunk + 1);
     const bf16 *ks = stages + (size_t)(chunk % s.stages) * elems, *qs = ks + CH * pitch, *vs = qs + CH * pitch,
                *ms = vs + CH * vp;
-    const float4 *fs = reinterpret_cast<const float4 *>(ms + 4 * CH * MP);
+    const float *fs = reinterpret_cast<const float *>(ms + 4 * CH * MP);
     float pk[8][4], pq[8][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i)
@@ -421,7 +446,7 @@ delta_scan_kernel(ScanArgs s) {
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         const int t = j * 16 + i * 8 + t2;
-        const float f0 = fs[t].x, f1 = fs[t + 1].x;
+        const float f0 = fs[t], f1 = fs[t + 1];
         float(&p)[4] = pk[2 * j + i];
         p[0] = low_half(x[2 * i]) - f0 * p[0];
         p[1] = high_half(x[2 * i]) - f1 * p[1];
@@ -464,7 +489,7 @@ delta_scan_kernel(ScanArgs s) {
     // O^T = e^G r' (S^T Q'^T) + U^T A^T
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      const float f0 = fs[i * 8 + t2].y, f1 = fs[i * 8 + t2 + 1].y;
+      const float f0 = fs[CH + i * 8 + t2], f1 = fs[CH + i * 8 + t2 + 1];
       pq[i][0] *= f0;
       pq[i][1] *= f1;
       pq[i][2] *= f0;
@@ -484,7 +509,7 @@ delta_scan_kernel(ScanArgs s) {
       terms(pq, hi, x, kt);
     }
     // S^T <- e^G_last S^T + (U^T diag(e^(G_last - G) r)) K'
-    const float keep = fs[0].w;
+    const float keep = fs[3 * CH];
 #pragma unroll
     for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -493,7 +518,7 @@ delta_scan_kernel(ScanArgs s) {
     for (int kt = 0; kt < 4; ++kt) {
 #pragma unroll
       for (int i = 2 * kt; i < 2 * kt + 2; ++i) {
-        const float f0 = fs[i * 8 + t2].z, f1 = fs[i * 8 + t2 + 1].z;
+        const float f0 = fs[2 * CH + i * 8 + t2], f1 = fs[2 * CH + i * 8 + t2 + 1];
         u[i][0] *= f0;
         u[i][1] *= f1;
         u[i][2] *= f0;
@@ -595,7 +620,7 @@ int launch_delta_chunks(const DeltaMixer &m, const void *conv, float *o, void *s
   c.chunks = (b.n + CH - 1) / CH;
   c.conv = static_cast<const bf16 *>(conv);
   c.mats = static_cast<bf16 *>(scratch);
-  c.factors = reinterpret_cast<float4 *>(static_cast<char *>(scratch) + part.mats);
+  c.factors = reinterpret_cast<float *>(static_cast<char *>(scratch) + part.mats);
   const PrepareArgs p{c, 1.0f / sqrtf((float)m.true_dim), m.a_log, m.dt_bias, m.ba, m.ba_ld};
   const size_t vectors = (size_t)2 * CH * (m.dim + 8) * 2, floats = (size_t)2 * CH * TP * 4;
   const size_t prep_smem = vectors > floats ? vectors : floats;

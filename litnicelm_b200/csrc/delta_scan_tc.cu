@@ -5,16 +5,17 @@
 // S^T as a 32-bit accumulator that stays for the whole sequence, and the left operands as two bfloat16 terms each,
 // written by the thread that owns the lane. So the elementwise steps between the products need no other thread, and
 // the right operands are the shared-memory tiles as TMA brings them (128-byte swizzle):
-//   PK = S^T K'^T, PQ = S^T Q'^T        right operand: K' and Q' rows
+//   [PK | PQ] = S^T [K'^T | Q'^T]       right operand: K' and Q' rows
 //   U  = (V^T - PK diag(e^G r)) T^T     right operand: T = (I + L)^-1 diag(beta), blocks of 16 on or below the diagonal
 //   S^T <- e^G_last S^T + (U diag(e^(G_last - G) r)) K'      right operand: K' again, its dimensions contiguous
-//   O  = PQ diag(e^G r') + U A^T        right operand: A
+//   UA = U A^T                          right operand: A;  the output is PQ diag(e^G r') + UA
+// Columns serve one thing after another: the operand of S becomes U, PK the right-hand side and then UA.
 //
 //   warp 0        TMA: K', Q', V tiles, the chunk's matrices and factors, two stages
 //   warp 1        owns tensor memory and issues the products
 //   warps 2-9     the chain: S to operand and decayed, right-hand side, U to operands; two warps share 32 lanes and take
 //                 alternating blocks of 16 columns
-//   warps 10-13   outputs, behind the chain: PQ scaled, O to shared memory, norm and gate over whole rows, store
+//   warps 10-17   outputs, behind the chain: to shared memory, norm and gate over whole rows, store
 // Every mbarrier wait is bounded; a wait that runs out sets the error word and ends the kernel after its copies have
 // landed and tensor memory is freed. No clusters, no multicast.
 #include "delta.cuh"
@@ -28,12 +29,13 @@ namespace {
 typedef __nv_bfloat16 bf16;
 
 constexpr int CH = DELTA_CHUNK;
-constexpr int DS_THREADS = 14 * 32;
-constexpr int DS_CHAIN = 8, DS_OUT = 4;  // warps
+constexpr int DS_CHAIN = 8, DS_OUT = 8;  // warps
+constexpr int DS_THREADS = (2 + DS_CHAIN + DS_OUT) * 32;
+constexpr int DS_PIECES = CH * 16 / (DS_OUT * 32);  // pieces of eight outputs per thread
 constexpr int DS_BOX = CH * 128;         // 64 rows of 64 elements
 constexpr int DS_SP = 132;               // floats per row of the output staging
 // tensor-memory columns
-constexpr unsigned TM_S = 0, TM_X = 128, TM_PK = 256, TM_PQ = 320, TM_U = 448;
+constexpr unsigned TM_S = 0, TM_SH = 128, TM_UH = 256, TM_PK = 384, TM_PQ = 448, TM_U = TM_SH, TM_UA = TM_PK;
 
 struct DsArgs {
   DeltaChunks c;
@@ -50,10 +52,11 @@ struct DsStage {
   static constexpr int KQ = 0;                      // two slabs of [K' rows | Q' rows]
   static constexpr int V = KQ + 4 * DS_BOX;         // two slabs
   static constexpr int MATS = V + 2 * DS_BOX;       // T high, T low, A high, A low
-  static constexpr int FACTORS = MATS + 4 * DS_BOX; // 64 float4
+  static constexpr int FACTORS = MATS + 4 * DS_BOX; // [4][64] floats
   static constexpr int BYTES = FACTORS + CH * 16;
 };
-constexpr int DS_STAGES_OFF = 0, DS_OUT_OFF = 2 * DsStage::BYTES, DS_BAR_OFF = DS_OUT_OFF + CH * DS_SP * 4;
+constexpr int DS_STAGES_OFF = 0, DS_OUT_OFF = 2 * DsStage::BYTES, DS_GATE_OFF = DS_OUT_OFF + CH * DS_SP * 4,
+              DS_BAR_OFF = DS_GATE_OFF + DS_PIECES * DS_OUT * 32 * 16;
 constexpr int DS_SMEM = DS_BAR_OFF + 256 + 1024;
 
 __device__ __forceinline__ unsigned pack2(float a, float b) {
@@ -83,10 +86,8 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
   const unsigned bars = base + DS_BAR_OFF;
   auto full = [&](int i) { return bars + 8u * i; };
   auto empty = [&](int i) { return bars + 8u * (2 + i); };
-  auto pq_free = [&](int i) { return bars + 8u * (4 + i); };
-  const unsigned sh_ready = bars + 48, pk_full = bars + 56, pq_full = bars + 64, r_ready = bars + 72, u_full = bars + 80,
-                 uh_ready = bars + 88, s_full = bars + 96, pq_scaled = bars + 104, o_full = bars + 112, rows_in = bars + 120,
-                 rows_out = bars + 128;
+  const unsigned sh_ready = bars + 32, p_full = bars + 40, r_ready = bars + 48, u_full = bars + 56, uh_ready = bars + 64,
+                 s_full = bars + 72, o_full = bars + 80, o_read = bars + 88, rows_in = bars + 96, rows_out = bars + 104;
   volatile unsigned *tmem_holder = reinterpret_cast<volatile unsigned *>(base_ptr + DS_BAR_OFF + 192);
   volatile int *abort_flag = reinterpret_cast<volatile int *>(base_ptr + DS_BAR_OFF + 196);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -95,17 +96,16 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
   const int grp = h / (a.heads / a.groups), vcols = min(128, a.vdim - vt);
   const int slabs = (a.dim + 63) >> 6, vslabs = (vcols + 63) >> 6, blocks = a.dim >> 4;
   auto stage_ptr = [&](int c) { return base_ptr + DS_STAGES_OFF + (c & 1) * DsStage::BYTES; };
-  auto factors_of = [&](int c) { return reinterpret_cast<const float4 *>(stage_ptr(c) + DsStage::FACTORS); };
+  auto factors_of = [&](int c) { return reinterpret_cast<const float *>(stage_ptr(c) + DsStage::FACTORS); };
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < 2; ++i) {
       mbar_init(full(i), 1);
       mbar_init(empty(i), 1 + DS_CHAIN + DS_OUT);
-      mbar_init(pq_free(i), DS_OUT);
     }
-    for (unsigned bar : {pk_full, pq_full, u_full, s_full, o_full}) mbar_init(bar, 1);
+    for (unsigned bar : {p_full, u_full, s_full, o_full}) mbar_init(bar, 1);
     for (unsigned bar : {sh_ready, r_ready, uh_ready}) mbar_init(bar, DS_CHAIN);
-    for (unsigned bar : {pq_scaled, rows_in, rows_out}) mbar_init(bar, DS_OUT);
+    for (unsigned bar : {o_read, rows_in, rows_out}) mbar_init(bar, DS_OUT);
     *abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -141,7 +141,7 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
         for (int k = 0; k < vslabs; ++k)
           tma_load_2d(st + DsStage::V + k * DS_BOX, &map_rows, 2 * a.groups * a.dim + h * a.vdim + vt + k * 64, row, full(i));
         for (int k = 0; k < 4; ++k) tma_load_2d(st + DsStage::MATS + k * DS_BOX, &map_mats, 0, (at * 4 + k) * CH, full(i));
-        bulk_load(st + DsStage::FACTORS, a.factors + (long long)at * CH, CH * 16, full(i));
+        bulk_load(st + DsStage::FACTORS, a.factors + (long long)at * 4 * CH, CH * 16, full(i));
       }
       ++loads;
       __syncwarp();
@@ -152,7 +152,7 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
         while (!mbar_try_wait(full(c & 1), (unsigned)(c >> 1) & 1u) && global_timer() < limit) {}
     }
   } else if (warp == 1) {
-    const unsigned id64 = umma_idesc_bf16(CH), id_s = umma_idesc_bf16(a.dim) | UMMA_B_MN_MAJOR;
+    const unsigned id_p = umma_idesc_bf16(2 * CH), id_s = umma_idesc_bf16(a.dim) | UMMA_B_MN_MAJOR;
     bool ok = true;
     int c = 0;
     auto hold = [&](unsigned bar, unsigned parity, int where) {
@@ -160,14 +160,15 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       return ok;
     };
-    // D[:, 16 kt ..] += A blocks (high at x, low at x + 8) times a lower triangular matrix's rows 16 kt .. of both terms
-    auto triangle = [&](unsigned d, unsigned x, unsigned step, unsigned mat, bool fresh) {
+    // D[:, 16 kt ..] (+)= operand blocks (high at x, low at x + 8) times a lower triangular matrix's rows 16 kt .. of both
+    // terms
+    auto triangle = [&](unsigned d, unsigned x, unsigned step, unsigned mat) {
 #pragma unroll
       for (int kt = 0; kt < 4; ++kt) {
         const unsigned long long hi = umma_desc_k128(mat + (unsigned)(kt * 2048)) + (unsigned long long)(kt * 2);
         const unsigned long long lo = umma_desc_k128(mat + DS_BOX + (unsigned)(kt * 2048)) + (unsigned long long)(kt * 2);
         const unsigned id = umma_idesc_bf16(CH - 16 * kt), at = d + (unsigned)(16 * kt), op = x + (unsigned)kt * step;
-        tc_mma_f16_ts(at, op, hi, id, fresh && kt == 0 ? 0u : 1u);
+        tc_mma_f16_ts(at, op, hi, id, kt ? 1u : 0u);
         tc_mma_f16_ts(at, op, lo, id, 1u);
         tc_mma_f16_ts(at, op + 8, hi, id, 1u);
       }
@@ -175,28 +176,20 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
     for (; c < a.chunks; ++c) {
       const unsigned st = base + DS_STAGES_OFF + (unsigned)((c & 1) * DsStage::BYTES), ph = (unsigned)c & 1u;
       if (!hold(full(c & 1), (unsigned)(c >> 1) & 1u, 42) || !hold(sh_ready, ph, 43)) break;
-      auto state_product = [&](unsigned d, unsigned rows) {
+      if (c > 0 && !hold(o_read, ph ^ 1u, 44)) break;
+      if (lane == 0) {
         for (int ks = 0; ks < blocks; ++ks) {
-          const unsigned long long x = umma_desc_k128(rows + (unsigned)((ks >> 2) * 2 * DS_BOX)) + (unsigned long long)((ks & 3) * 2);
-          tc_mma_f16_ts(d, tmem + TM_X + (unsigned)(ks * 16), x, id64, ks ? 1u : 0u);
-          tc_mma_f16_ts(d, tmem + TM_X + (unsigned)(ks * 16 + 8), x, id64, 1u);
+          const unsigned long long x =
+              umma_desc_k128(st + DsStage::KQ + (unsigned)((ks >> 2) * 2 * DS_BOX)) + (unsigned long long)((ks & 3) * 2);
+          tc_mma_f16_ts(tmem + TM_PK, tmem + TM_SH + (unsigned)(ks * 16), x, id_p, ks ? 1u : 0u);
+          tc_mma_f16_ts(tmem + TM_PK, tmem + TM_SH + (unsigned)(ks * 16 + 8), x, id_p, 1u);
         }
-      };
-      if (lane == 0) {
-        state_product(tmem + TM_PK, st + DsStage::KQ);
-        tc_commit(pk_full);
-      }
-      __syncwarp();
-      if (c >= 2 && !hold(pq_free(c & 1), (unsigned)((c >> 1) - 1) & 1u, 44)) break;
-      const unsigned pq = tmem + TM_PQ + (unsigned)((c & 1) * CH);
-      if (lane == 0) {
-        state_product(pq, st + DsStage::KQ + DS_BOX);
-        tc_commit(pq_full);
+        tc_commit(p_full);
       }
       __syncwarp();
       if (!hold(r_ready, ph, 45)) break;
       if (lane == 0) {
-        triangle(tmem + TM_U, tmem + TM_PK, 16, st + DsStage::MATS, true);
+        triangle(tmem + TM_U, tmem + TM_PK, 16, st + DsStage::MATS);
         tc_commit(u_full);
       }
       __syncwarp();
@@ -205,15 +198,11 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
 #pragma unroll
         for (int kt = 0; kt < 4; ++kt) {
           const unsigned long long x = umma_desc_mn128(st + DsStage::KQ + (unsigned)(kt * 2048), 2 * DS_BOX);
-          tc_mma_f16_ts(tmem + TM_S, tmem + TM_X + (unsigned)(kt * 32 + 16), x, id_s, 1u);
-          tc_mma_f16_ts(tmem + TM_S, tmem + TM_X + (unsigned)(kt * 32 + 24), x, id_s, 1u);
+          tc_mma_f16_ts(tmem + TM_S, tmem + TM_UH + (unsigned)(kt * 32 + 16), x, id_s, 1u);
+          tc_mma_f16_ts(tmem + TM_S, tmem + TM_UH + (unsigned)(kt * 32 + 24), x, id_s, 1u);
         }
         tc_commit(s_full);
-      }
-      __syncwarp();
-      if (!hold(pq_scaled, ph, 47)) break;
-      if (lane == 0) {
-        triangle(pq, tmem + TM_X, 32, st + DsStage::MATS + 2 * DS_BOX, false);
+        triangle(tmem + TM_UA, tmem + TM_UH, 32, st + DsStage::MATS + 2 * DS_BOX);
         tc_commit(o_full);
         tc_commit(empty(c & 1));
       }
@@ -246,36 +235,36 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
     for (int c = 0; c < a.chunks && ok; ++c) {
       const unsigned ph = (unsigned)c & 1u;
       // S: operand blocks for the products with K' and Q', and e^G_last S in place
-      unsigned x[4][16];
-      if (c == 0) {
+      if (!hold(full(c & 1), (unsigned)(c >> 1) & 1u, 48)) break;
+      const float *fs = factors_of(c);
+      const float keep = fs[3 * CH];
+      if (c > 0 && !hold(s_full, ph ^ 1u, 49)) break;
+      unsigned x[2][16];
+#pragma unroll 1
+      for (int k0 = half; k0 < blocks; k0 += 4) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
+        for (int i = 0; i < 2; ++i) {
+          const int kt = k0 + 2 * i;
+          if (kt >= blocks) break;
+          if (c > 0) {
+            tc_ld16(lanes + TM_S + (unsigned)(kt * 16), x[i]);
+          } else {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) {
-            const int d = (2 * i + half) * 16 + j;
-            x[i][j] = s.p0 > 0 && mine && d < a.dim ? __float_as_uint(S[(long long)d * a.vdim]) : 0u;
+            for (int j = 0; j < 16; ++j)
+              x[i][j] = s.p0 > 0 && mine ? __float_as_uint(S[(long long)(kt * 16 + j) * a.vdim]) : 0u;
           }
-      } else {
-        if (!hold(s_full, ph ^ 1u, 48)) break;
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-          if (2 * i + half < blocks) tc_ld16(lanes + TM_S + (unsigned)((2 * i + half) * 16), x[i]);
+        }
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-      }
-      if (!hold(full(c & 1), (unsigned)(c >> 1) & 1u, 49)) break;
-      const float4 *fs = factors_of(c);
-      const float keep = fs[0].w;
-      if (c > 0 && !hold(o_full, ph ^ 1u, 50)) break;  // U's operands are read: their columns are S's now
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int kt = 2 * i + half;
-        if (kt < blocks) {
+        for (int i = 0; i < 2; ++i) {
+          const int kt = k0 + 2 * i;
+          if (kt >= blocks) break;
           float f[16];
           unsigned w[16];
 #pragma unroll
           for (int j = 0; j < 16; ++j) f[j] = __uint_as_float(x[i][j]);
           operand_block<0>(f, w);
-          tc_st16(lanes + TM_X + (unsigned)(kt * 16), w);
+          tc_st16(lanes + TM_SH + (unsigned)(kt * 16), w);
 #pragma unroll
           for (int j = 0; j < 16; ++j) w[j] = __float_as_uint(f[j] * keep);
           tc_st16(lanes + TM_S + (unsigned)(kt * 16), w);
@@ -292,7 +281,7 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
           const int t = (2 * i + half) * 16 + j;
           rhs[i][j] = mine ? __bfloat162float(*reinterpret_cast<const bf16 *>(vs + t * 128 + (((vl & 63) * 2) ^ ((t & 7) << 4)))) : 0.f;
         }
-      if (!hold(pk_full, ph, 51)) break;
+      if (!hold(p_full, ph, 51)) break;
 #pragma unroll
       for (int i = 0; i < 2; ++i) tc_ld16(lanes + TM_PK + (unsigned)((2 * i + half) * 16), x[i]);
       asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -301,7 +290,13 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
         const int kt = 2 * i + half;
         unsigned w[16];
 #pragma unroll
-        for (int j = 0; j < 16; ++j) rhs[i][j] = fmaf(-fs[kt * 16 + j].x, __uint_as_float(x[i][j]), rhs[i][j]);
+        for (int j = 0; j < 16; j += 4) {
+          const float4 y = *reinterpret_cast<const float4 *>(fs + kt * 16 + j);
+          rhs[i][j] = fmaf(-y.x, __uint_as_float(x[i][j]), rhs[i][j]);
+          rhs[i][j + 1] = fmaf(-y.y, __uint_as_float(x[i][j + 1]), rhs[i][j + 1]);
+          rhs[i][j + 2] = fmaf(-y.z, __uint_as_float(x[i][j + 2]), rhs[i][j + 2]);
+          rhs[i][j + 3] = fmaf(-y.w, __uint_as_float(x[i][j + 3]), rhs[i][j + 3]);
+        }
         operand_block<0>(rhs[i], w);
         tc_st16(lanes + TM_PK + (unsigned)(kt * 16), w);
       }
@@ -320,29 +315,33 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
         for (int j = 0; j < 16; ++j) f[j] = __uint_as_float(x[i][j]);
         operand_block<0>(f, w);
 #pragma unroll
-        for (int j = 0; j < 16; ++j) f[j] *= fs[kt * 16 + j].z;
+        for (int j = 0; j < 16; j += 4) {
+          const float4 y = *reinterpret_cast<const float4 *>(fs + 2 * CH + kt * 16 + j);
+          f[j] *= y.x;
+          f[j + 1] *= y.y;
+          f[j + 2] *= y.z;
+          f[j + 3] *= y.w;
+        }
         operand_block<16>(f, w);
-        tc_st32(lanes + TM_X + (unsigned)(kt * 32), w);
+        tc_st32(lanes + TM_UH + (unsigned)(kt * 32), w);
       }
       release(uh_ready);
       if (lane == 0) mbar_arrive(empty(c & 1));
     }
     if (ok && hold(s_full, (unsigned)(a.chunks - 1) & 1u, 53)) {
-      unsigned x[4][16];
+#pragma unroll 1
+      for (int kt = half; kt < blocks; kt += 2) {
+        unsigned x[16];
+        tc_ld16(lanes + TM_S + (unsigned)(kt * 16), x);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        if (mine) {
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-        if (2 * i + half < blocks) tc_ld16(lanes + TM_S + (unsigned)((2 * i + half) * 16), x[i]);
-      asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          const int d = (2 * i + half) * 16 + j;
-          if (mine && d < a.dim) S[(long long)d * a.vdim] = __uint_as_float(x[i][j]);
+          for (int j = 0; j < 16; ++j) S[(long long)(kt * 16 + j) * a.vdim] = __uint_as_float(x[j]);
         }
+      }
     }
   } else {
-    const int q = warp & 3, tid = threadIdx.x - (2 + DS_CHAIN) * 32;
+    const int q = warp & 3, half = (warp - 2 - DS_CHAIN) >> 2, tid = threadIdx.x - (2 + DS_CHAIN) * 32;
     const unsigned lanes = tmem + ((unsigned)(q * 32) << 16);
     const int vl = q * 32 + lane;
     float *staging = reinterpret_cast<float *>(base_ptr + DS_OUT_OFF);
@@ -357,79 +356,115 @@ delta_scan_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
       __syncwarp();
       if (lane == 0) mbar_arrive(bar);
     };
-    // whole rows of outputs: 16 lanes per token, eight columns each, eight tokens at a time
+    // whole rows of outputs: 16 lanes per token, eight columns each
     const int col = (tid & 15) * 8, row0 = tid >> 4;
     const bool in = col < vcols;
-    float4 w0 = make_float4(0.f, 0.f, 0.f, 0.f), w1 = w0;
+    const float inv_count = 1.0f / s.count;
+    float w8[8] = {};
     if (s.normed && in) {
-      w0 = *reinterpret_cast<const float4 *>(s.norm + col);
-      w1 = *reinterpret_cast<const float4 *>(s.norm + col + 4);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) w8[j] = s.norm[col + j];
     }
-    for (int c = 0; c < a.chunks && ok; ++c) {
-      const unsigned ph = (unsigned)c & 1u, pq = lanes + TM_PQ + (unsigned)((c & 1) * CH);
-      const int t0 = c * CH, nt = min(CH, a.n - t0);
-      uint4 gate[8];
+    // the gates of this thread's eight pieces of a chunk, in its own corner of shared memory, a chunk ahead
+    uint4 *gates = reinterpret_cast<uint4 *>(base_ptr + DS_GATE_OFF) + tid;
+    auto fetch_gates = [&](int c) {
+      if (s.normed) {
 #pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const int t = row0 + 8 * k;
-        gate[k] = s.normed && in && t < nt
-                      ? *reinterpret_cast<const uint4 *>(s.gate + ((long long)b * a.n + t0 + t) * s.in_ld + h * a.vdim + col)
-                      : make_uint4(0, 0, 0, 0);
-      }
-      if (!hold(full(c & 1), (unsigned)(c >> 1) & 1u, 54) || !hold(pq_full, ph, 55)) break;
-      const float4 *fs = factors_of(c);
-      unsigned x[2][32];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) tc_ld32(pq + (unsigned)(i * 32), x[i]);
-      asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-#pragma unroll
-        for (int j = 0; j < 32; ++j) x[i][j] = __float_as_uint(__uint_as_float(x[i][j]) * fs[i * 32 + j].y);
-        tc_st32(pq + (unsigned)(i * 32), x[i]);
-      }
-      asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
-      release(pq_scaled);
-      if (lane == 0) mbar_arrive(empty(c & 1));
-      if (!hold(o_full, ph, 56)) break;
-#pragma unroll
-      for (int i = 0; i < 2; ++i) tc_ld32(pq + (unsigned)(i * 32), x[i]);
-      asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-      release(pq_free(c & 1));
-      if (c > 0 && !hold(rows_out, ph ^ 1u, 57)) break;  // the last chunk's rows have been read
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-#pragma unroll
-        for (int j = 0; j < 32; ++j) staging[(i * 32 + j) * DS_SP + vl] = vl < vcols ? __uint_as_float(x[i][j]) : 0.f;
-      release(rows_in);
-      if (!hold(rows_in, ph, 58)) break;
-#pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const int t = row0 + 8 * k;
-        const float4 y = *reinterpret_cast<const float4 *>(staging + t * DS_SP + col);
-        const float4 z = *reinterpret_cast<const float4 *>(staging + t * DS_SP + col + 4);
-        const long long r = (long long)b * a.n + t0 + t;
-        if (!s.normed) {
-          if (in && t < nt) {
-            float *o = s.o + (r * a.heads + h) * a.vdim + vt + col;
-            *reinterpret_cast<float4 *>(o) = y;
-            *reinterpret_cast<float4 *>(o + 4) = z;
-          }
-          continue;
+        for (int k = 0; k < DS_PIECES; ++k) {
+          const int t = c * CH + row0 + k * (CH / DS_PIECES);
+          const bool there = in && t < a.n;
+          const bf16 *src = there ? s.gate + ((long long)b * a.n + t) * s.in_ld + h * a.vdim + col : s.gate;
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(gates + k * DS_OUT * 32)), "l"(src),
+                       "r"(there ? 16 : 0)
+                       : "memory");
         }
-        float sum = y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w + z.x * z.x + z.y * z.y + z.z * z.z + z.w * z.w;
+      }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch_gates(0);
+    for (int c = 0; c < a.chunks && ok; ++c) {
+      const unsigned ph = (unsigned)c & 1u;
+      const int t0 = c * CH, nt = min(CH, a.n - t0);
+      if (!hold(full(c & 1), (unsigned)(c >> 1) & 1u, 54) || !hold(o_full, ph, 55)) break;
+      const float *fs = factors_of(c) + CH;
+      {  // this warp's half of the tokens
+        unsigned x[2][16], y[2][16];
 #pragma unroll
-        for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        if (!in || t >= nt) continue;
-        const float inv = 1.0f / sqrtf(sum / s.count + s.eps);
-        const uint4 g = gate[k];
-        *reinterpret_cast<uint4 *>(s.out + r * s.out_ld + h * a.vdim + col) =
-            make_uint4(pack2(y.x * inv * w0.x * silu_fast(lowf(g.x)), y.y * inv * w0.y * silu_fast(highf(g.x))),
-                       pack2(y.z * inv * w0.z * silu_fast(lowf(g.y)), y.w * inv * w0.w * silu_fast(highf(g.y))),
-                       pack2(z.x * inv * w1.x * silu_fast(lowf(g.z)), z.y * inv * w1.y * silu_fast(highf(g.z))),
-                       pack2(z.z * inv * w1.z * silu_fast(lowf(g.w)), z.w * inv * w1.w * silu_fast(highf(g.w))));
+        for (int i = 0; i < 2; ++i) {
+          tc_ld16(lanes + TM_PQ + (unsigned)(half * 32 + i * 16), x[i]);
+          tc_ld16(lanes + TM_UA + (unsigned)(half * 32 + i * 16), y[i]);
+        }
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        release(o_read);
+        if (c > 0 && !hold(rows_out, ph ^ 1u, 56)) break;  // the last chunk's rows have been read
+        float *to = staging + half * 32 * DS_SP + vl;
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int j = 0; j < 16; j += 4) {
+            const float4 f = *reinterpret_cast<const float4 *>(fs + half * 32 + i * 16 + j);
+            float *at = to + (i * 16 + j) * DS_SP;
+            at[0] = vl < vcols ? fmaf(__uint_as_float(x[i][j]), f.x, __uint_as_float(y[i][j])) : 0.f;
+            at[DS_SP] = vl < vcols ? fmaf(__uint_as_float(x[i][j + 1]), f.y, __uint_as_float(y[i][j + 1])) : 0.f;
+            at[2 * DS_SP] = vl < vcols ? fmaf(__uint_as_float(x[i][j + 2]), f.z, __uint_as_float(y[i][j + 2])) : 0.f;
+            at[3 * DS_SP] = vl < vcols ? fmaf(__uint_as_float(x[i][j + 3]), f.w, __uint_as_float(y[i][j + 3])) : 0.f;
+          }
+      }
+      release(rows_in);
+      if (lane == 0) mbar_arrive(empty(c & 1));
+      if (!hold(rows_in, ph, 57)) break;
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll 1
+      for (int k0 = 0; k0 < DS_PIECES; k0 += 4) {  // four rows together: their sums do not wait for one another
+        float y[4][8], sum[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float *row = staging + (row0 + (CH / DS_PIECES) * (k0 + k)) * DS_SP + col;
+          const float4 u = *reinterpret_cast<const float4 *>(row), w = *reinterpret_cast<const float4 *>(row + 4);
+          const float e[8] = {u.x, u.y, u.z, u.w, w.x, w.y, w.z, w.w};
+          float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+          for (int j = 0; j < 8; j += 2) {
+            y[k][j] = e[j];
+            y[k][j + 1] = e[j + 1];
+            s0 = fmaf(e[j], e[j], s0);
+            s1 = fmaf(e[j + 1], e[j + 1], s1);
+          }
+          sum[k] = s0 + s1;
+        }
+        if (s.normed) {
+#pragma unroll
+          for (int o = 8; o > 0; o >>= 1)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) sum[k] += __shfl_xor_sync(0xffffffffu, sum[k], o);
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const int t = row0 + (CH / DS_PIECES) * (k0 + k);
+          const long long r = (long long)b * a.n + t0 + t;
+          const bool store = in && t < nt;
+          if (!s.normed) {
+            if (store) {
+              float *o = s.o + (r * a.heads + h) * a.vdim + vt + col;
+              *reinterpret_cast<float4 *>(o) = make_float4(y[k][0], y[k][1], y[k][2], y[k][3]);
+              *reinterpret_cast<float4 *>(o + 4) = make_float4(y[k][4], y[k][5], y[k][6], y[k][7]);
+            }
+            continue;
+          }
+          const float inv = rsqrtf(sum[k] * inv_count + s.eps);
+          const uint4 gate = gates[(k0 + k) * DS_OUT * 32];
+          const unsigned g[4] = {gate.x, gate.y, gate.z, gate.w};
+          unsigned out[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            out[j] = pack2(y[k][2 * j] * inv * w8[2 * j] * silu_fast(lowf(g[j])),
+                           y[k][2 * j + 1] * inv * w8[2 * j + 1] * silu_fast(highf(g[j])));
+          if (store)
+            *reinterpret_cast<uint4 *>(s.out + r * s.out_ld + h * a.vdim + col) = make_uint4(out[0], out[1], out[2], out[3]);
+        }
       }
       release(rows_out);
+      if (c + 1 < a.chunks) fetch_gates(c + 1);
     }
   }
   __syncwarp();
