@@ -14,6 +14,7 @@
 // All arithmetic 32-bit; the history is stored by position modulo the number of taps: a single new row
 // never overwrites an input that another CTA still reads.
 #include "delta.cuh"
+#include "tc_ptx.cuh"
 
 namespace lb {
 
@@ -201,14 +202,40 @@ struct StepArgs {
   long long rows_ld;  // of the convolved rows
 };
 
-// WARPS warps share the state's rows, DPW each; a lane holds VPT value columns.
+// VPT neighbouring floats of a state row.
+template <int VPT>
+__device__ __forceinline__ void load_cols(const float *p, bool ok, float (&s)[VPT]) {
+  if constexpr (VPT == 4) {
+    const float4 v = ok ? *reinterpret_cast<const float4 *>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
+    s[0] = v.x;
+    s[1] = v.y;
+    s[2] = v.z;
+    s[3] = v.w;
+  } else if constexpr (VPT == 2) {
+    const float2 v = ok ? *reinterpret_cast<const float2 *>(p) : make_float2(0.f, 0.f);
+    s[0] = v.x;
+    s[1] = v.y;
+  } else {
+    s[0] = ok ? *p : 0.f;
+  }
+}
+template <int VPT>
+__device__ __forceinline__ void store_cols(float *p, const float (&s)[VPT]) {
+  if constexpr (VPT == 4) *reinterpret_cast<float4 *>(p) = make_float4(s[0], s[1], s[2], s[3]);
+  else if constexpr (VPT == 2) *reinterpret_cast<float2 *>(p) = make_float2(s[0], s[1]);
+  else *p = s[0];
+}
+
+// WARPS warps share the state's rows, DPW each; a lane holds VPT value columns. FUSED: the CTAs of a head are a
+// cluster (one CTA: none); the squares of its outputs meet in shared memory while each stores its part of the state.
 template <typename T, int WARPS, int DPW, int VPT, bool FUSED>
-__global__ void __launch_bounds__(WARPS * 32)
+__global__ void __launch_bounds__(WARPS * 32, 512 / (WARPS * 32))
 delta_step_kernel(StepArgs a, const T *in, T *history, float *o_rows, T *out, DeltaRows g) {
   constexpr int THREADS = WARPS * 32, VT = 32 * VPT, DIMS = WARPS * DPW;
   constexpr int FILL = (2 * DIMS + VT + THREADS - 1) / THREADS;
   __shared__ __align__(16) float vec[2][2 * DIMS + VT];  // q', k', v of a token
   __shared__ __align__(16) float red[WARPS][2][VT];
+  __shared__ float squares;
   pdl_launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
   const int tiles = (a.vdim + VT - 1) / VT;
@@ -224,23 +251,18 @@ delta_step_kernel(StepArgs a, const T *in, T *history, float *o_rows, T *out, De
   }
   const float a_exp_log = a.a_log[h], bias = a.dt_bias[h];
   pdl_wait();
-  const int p0 = g.first_position();
   float s[DPW][VPT];
 #pragma unroll
   for (int i = 0; i < DPW; ++i) {
     const float *row = S + (long long)(d0 + i) * a.vdim + v0;
-    const bool ok = p0 > 0 && v_in && d0 + i < a.dim;
-    if constexpr (VPT == 4) {
-      const float4 v = ok ? *reinterpret_cast<const float4 *>(row) : make_float4(0.f, 0.f, 0.f, 0.f);
-      s[i][0] = v.x;
-      s[i][1] = v.y;
-      s[i][2] = v.z;
-      s[i][3] = v.w;
-    } else {
-      const float2 v = ok ? *reinterpret_cast<const float2 *>(row) : make_float2(0.f, 0.f);
-      s[i][0] = v.x;
-      s[i][1] = v.y;
-    }
+    load_cols(row, v_in && d0 + i < a.dim, s[i]);
+  }
+  const int p0 = g.first_position();  // asked for behind the state, whose loads need not wait for it
+  if (p0 == 0) {  // a new sequence
+#pragma unroll
+    for (int i = 0; i < DPW; ++i)
+#pragma unroll
+      for (int j = 0; j < VPT; ++j) s[i][j] = 0.f;
   }
   // channel of entry e of a token's vectors, or -1 for padding
   auto channel = [&](int e) -> int {
@@ -268,7 +290,7 @@ delta_step_kernel(StepArgs a, const T *in, T *history, float *o_rows, T *out, De
         }
         y = fmaf(a.conv[(long long)(a.taps - 1) * channels + c], to_f(x), y);
         next[i] = to_f(from_f<T>(Wide<T>::silu(y)));
-        if (tid + i * THREADS >= 2 * DIMS || h % (a.heads / a.groups) == 0) hist[(long long)(p0 % a.taps) * channels] = x;
+        if (tid + i * THREADS >= 2 * DIMS || (vt == 0 && h % (a.heads / a.groups) == 0)) hist[(long long)(p0 % a.taps) * channels] = x;
       } else {
         next[i] = to_f(in[r * a.rows_ld + c]);
       }
@@ -318,8 +340,9 @@ delta_step_kernel(StepArgs a, const T *in, T *history, float *o_rows, T *out, De
       for (int w = 0; w < WARPS; ++w) sum += red[w][0][lane * VPT + j];
       u[j] = beta * (v[lane * VPT + j] - decay * rk * sum);
     }
+    float o[VPT];
     if (wid == 0) {
-      float o[VPT], ss = 0.f;
+      float ss = 0.f;
 #pragma unroll
       for (int j = 0; j < VPT; ++j) {
         float sum = 0.f;
@@ -328,20 +351,18 @@ delta_step_kernel(StepArgs a, const T *in, T *history, float *o_rows, T *out, De
         o[j] = decay * rq * sum + kq * u[j];
         ss = fmaf(o[j], o[j], ss);
       }
-      const long long r = (long long)b * g.n + t;
       if constexpr (FUSED) {  // padding columns are zeros
-        const float inv = 1.0f / sqrtf(warp_sum(ss) / a.count + a.eps);
-        const T *gate = in + r * a.in_ld + channels + h * a.vdim;
-        T *y = out + r * a.out_ld + h * a.vdim;
-        if (v_in) {
-#pragma unroll
-          for (int j = 0; j < VPT; ++j)
-            y[v0 + j] = from_f<T>(o[j] * inv * a.norm[v0 + j] * silu_f32(to_f(gate[v0 + j])));
-        }
+        ss = warp_sum(ss);
+        if (lane == 0) squares = ss;
       } else if (v_in) {
+        const long long r = (long long)b * g.n + t;
 #pragma unroll
         for (int j = 0; j < VPT; ++j) o_rows[(r * a.heads + h) * a.vdim + v0 + j] = o[j];
       }
+    }
+    if (FUSED && tiles > 1) {
+      __syncwarp();
+      asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
     }
 #pragma unroll
     for (int i = 0; i < DPW; ++i) {
@@ -349,14 +370,38 @@ delta_step_kernel(StepArgs a, const T *in, T *history, float *o_rows, T *out, De
 #pragma unroll
       for (int j = 0; j < VPT; ++j) s[i][j] = fmaf(kd, u[j], decay * s[i][j]);
     }
+    if constexpr (FUSED) {
+#pragma unroll
+      for (int i = 0; i < DPW; ++i)
+        if (v_in && d0 + i < a.dim) store_cols(S + (long long)(d0 + i) * a.vdim + v0, s[i]);
+      if (tiles > 1) {
+        __syncwarp();
+        cluster_wait();
+      }
+      if (wid == 0) {
+        __syncwarp();
+        float ss = tiles == 1 ? squares : 0.f;
+        if (tiles > 1)
+          for (int i = 0; i < tiles; ++i) ss += ld_cluster_f32(cluster_map(smem_u32(&squares), (unsigned)i));
+        const float inv = 1.0f / sqrtf(ss / a.count + a.eps);
+        const T *gate = in + (long long)b * a.in_ld + channels + h * a.vdim;
+        T *y = out + (long long)b * a.out_ld + h * a.vdim;
+        if (v_in) {
+#pragma unroll
+          for (int j = 0; j < VPT; ++j)
+            y[v0 + j] = from_f<T>(o[j] * inv * a.norm[v0 + j] * Wide<T>::silu(to_f(gate[v0 + j])));
+        }
+      }
+      if (tiles > 1) {  // a CTA's shared memory stays until every other has read it
+        __syncwarp();
+        cluster_sync_all();
+      }
+      return;
+    }
   }
 #pragma unroll
-  for (int i = 0; i < DPW; ++i) {
-    if (!v_in || d0 + i >= a.dim) continue;
-    float *row = S + (long long)(d0 + i) * a.vdim + v0;
-    if constexpr (VPT == 4) *reinterpret_cast<float4 *>(row) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
-    else *reinterpret_cast<float2 *>(row) = make_float2(s[i][0], s[i][1]);
-  }
+  for (int i = 0; i < DPW; ++i)
+    if (v_in && d0 + i < a.dim) store_cols(S + (long long)(d0 + i) * a.vdim + v0, s[i]);
 }
 
 // One warp per row and head.
@@ -426,14 +471,25 @@ int launch_t(const DeltaMixer &m, void *scratch, Precision type, const RowBatch 
   a.in_ld = m.in_ld;
   a.out_ld = m.out_ld;
   a.rows_ld = m.conv_channels();
-  auto step = [&](auto kernel, int threads, int vt, const T *src) {
-    launch_pdl(kernel, dim3((unsigned)(m.heads * ((m.vdim + vt - 1) / vt)), (unsigned)b.streams), dim3((unsigned)threads), 0, st,
-               g_pdl_enabled, a, src, static_cast<T *>(m.history), o, out, g);
+  auto step = [&](auto kernel, int threads, int vt, const T *src, bool cluster) {
+    const int tiles = (m.vdim + vt - 1) / vt;
+    launch_pdl_cluster_x(kernel, dim3((unsigned)(m.heads * tiles), (unsigned)b.streams), dim3((unsigned)threads), 0, st,
+                         g_pdl_enabled, cluster ? (unsigned)tiles : 1u, a, src, static_cast<T *>(m.history), o, out, g);
   };
-  if (b.n == 1 && m.dim <= 256 && m.vdim <= 128) {
-    if (m.dim <= 64) step(delta_step_kernel<T, 8, 8, 4, true>, 256, 128, in);
-    else if (m.dim <= 128) step(delta_step_kernel<T, 8, 16, 4, true>, 256, 128, in);
-    else step(delta_step_kernel<T, 16, 16, 4, true>, 512, 128, in);
+  if (b.n == 1 && m.dim <= 256 && m.vdim <= 256) {
+    // the fewest value columns per lane that let one CTA hold a head: splitting a head further gained nothing at any size
+    auto fused = [&](auto one, auto two, auto four, int threads) {
+      if (m.vdim <= 32) step(one, threads, 32, in, true);
+      else if (m.vdim <= 64) step(two, threads, 64, in, true);
+      else step(four, threads, 128, in, true);
+    };
+    if (m.dim <= 64)
+      fused(delta_step_kernel<T, 8, 8, 1, true>, delta_step_kernel<T, 8, 8, 2, true>, delta_step_kernel<T, 8, 8, 4, true>, 256);
+    else if (m.dim <= 128)
+      fused(delta_step_kernel<T, 8, 16, 1, true>, delta_step_kernel<T, 8, 16, 2, true>, delta_step_kernel<T, 8, 16, 4, true>, 256);
+    else
+      fused(delta_step_kernel<T, 16, 16, 1, true>, delta_step_kernel<T, 16, 16, 2, true>, delta_step_kernel<T, 16, 16, 4, true>,
+            512);
     return 1;
   }
   const int strip = m.taps - 1 > DC_STRIP ? m.taps - 1 : DC_STRIP, channels = m.conv_channels();
@@ -457,10 +513,10 @@ int launch_t(const DeltaMixer &m, void *scratch, Precision type, const RowBatch 
     if (normed) return launches;
   } else {
     const T *src = conv;
-    if (m.dim <= 64) step(delta_step_kernel<T, 8, 8, 4, false>, 256, 128, src);
-    else if (m.dim <= 128) step(delta_step_kernel<T, 8, 16, 4, false>, 256, 128, src);
-    else if (m.dim <= 256) step(delta_step_kernel<T, 16, 16, 4, false>, 512, 128, src);
-    else step(delta_step_kernel<T, 16, 32, 2, false>, 512, 64, src);
+    if (m.dim <= 64) step(delta_step_kernel<T, 8, 8, 4, false>, 256, 128, src, false);
+    else if (m.dim <= 128) step(delta_step_kernel<T, 8, 16, 4, false>, 256, 128, src, false);
+    else if (m.dim <= 256) step(delta_step_kernel<T, 16, 16, 4, false>, 512, 128, src, false);
+    else step(delta_step_kernel<T, 16, 32, 2, false>, 512, 64, src, false);
     ++launches;
   }
   const long long total = b.rows() * m.heads;

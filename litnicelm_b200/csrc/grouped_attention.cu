@@ -20,7 +20,7 @@ namespace {
 typedef __nv_bfloat16 bf16;
 
 constexpr int GA_THREADS = 256;
-constexpr int GA_KEYS = 64;     // keys per tile
+constexpr int GA_KEYS = 128;    // keys per tile
 constexpr int GA_CLUSTER = 8;   // CTAs of the largest cluster
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -197,7 +197,7 @@ struct RowsArgs {
 
 // Split blockIdx.x of the keys, R query heads of one group (blockIdx.y), row blockIdx.z.
 template <typename T, int R>
-__global__ void __launch_bounds__(GA_THREADS)
+__global__ void __launch_bounds__(GA_THREADS, R <= 4 ? 2 : 1)
 grouped_rows_kernel(RowsArgs a, const T *q, const T *k_cache, const T *v_cache, T *out, RowsShape g) {
   constexpr int P = Piece<T>::N;
   extern __shared__ __align__(16) float sm[];
@@ -221,8 +221,12 @@ grouped_rows_kernel(RowsArgs a, const T *q, const T *k_cache, const T *v_cache, 
   const int k_ld = a.groups * a.dim, v_ld = a.groups * a.vdim;
   const T *kr = k_cache + ((long long)(g.slot0 + b) * a.cap + j0) * k_ld + grp * a.dim;
   const T *vr = v_cache + ((long long)(g.slot0 + b) * a.cap + j0) * v_ld + grp * a.vdim;
-  for (int i = tid; i < R * a.dim; i += GA_THREADS)
-    qs[i] = i < nh * a.dim ? to_f(q[r * a.q_ld + (long long)h0 * a.dim + i]) * a.factor : 0.f;
+  // queries by planes of four elements of every piece: lanes on neighbouring pieces read neighbouring 16 bytes
+  for (int i = tid; i < R * a.dim; i += GA_THREADS) {
+    const int hh = i / a.dim, e = i - hh * a.dim;
+    qs[hh * a.dim + (e % P / 4) * (a.dim / P * 4) + e / P * 4 + (e & 3)] =
+        i < nh * a.dim ? to_f(q[r * a.q_ld + (long long)h0 * a.dim + i]) * a.factor : 0.f;
+  }
   const int pieces = a.dim / P, cols = a.vdim / P;       // 16-byte pieces of a key and of a value
   const int key_groups = GA_THREADS / cols;
   const int vc = tid % cols * P, vg = tid / cols;        // this thread's value columns and its key group
@@ -236,42 +240,50 @@ grouped_rows_kernel(RowsArgs a, const T *q, const T *k_cache, const T *v_cache, 
   __syncthreads();
   for (int k0 = 0; k0 < total; k0 += GA_KEYS) {
     const int nk = min(GA_KEYS, total - k0);
-    {  // scores: eight lanes per key, two batches of four keys per warp
-      const int sub = lane & 7, ja = wid * 8 + (lane >> 3), jb = ja + 4;
-      const T *ka = kr + (long long)(k0 + min(ja, nk - 1)) * k_ld, *kb = kr + (long long)(k0 + min(jb, nk - 1)) * k_ld;
-      float sa[R], sb[R];
+    {  // scores: eight lanes per key, batches of four keys per warp
+      constexpr int BATCHES = GA_KEYS / (GA_THREADS / 8);
+      const int sub = lane & 7, j0w = wid * (GA_KEYS / (GA_THREADS / 32)) + (lane >> 3);
+      const T *kp[BATCHES];
+      float sum[BATCHES][R];
 #pragma unroll
-      for (int h = 0; h < R; ++h) sa[h] = sb[h] = 0.f;
-#pragma unroll 2
+      for (int i = 0; i < BATCHES; ++i) {
+        kp[i] = kr + (long long)(k0 + min(j0w + 4 * i, nk - 1)) * k_ld;
+#pragma unroll
+        for (int h = 0; h < R; ++h) sum[i][h] = 0.f;
+      }
       for (int c = sub; c < pieces; c += 8) {
-        Piece<T> xa, xb;
-        xa.load(ka + c * P);
-        xb.load(kb + c * P);
-        float fa[P], fb[P];
-        xa.unpack(fa);
-        xb.unpack(fb);
+        Piece<T> x[BATCHES];
+#pragma unroll
+        for (int i = 0; i < BATCHES; ++i) x[i].load(kp[i] + c * P);
+        float f[BATCHES][P];
+#pragma unroll
+        for (int i = 0; i < BATCHES; ++i) x[i].unpack(f[i]);
 #pragma unroll
         for (int h = 0; h < R; ++h) {
-          const float *qh = qs + h * a.dim + c * P;
+          const float *qh = qs + h * a.dim + c * 4;
 #pragma unroll
-          for (int i = 0; i < P; i += 4) {
-            const float4 w = *reinterpret_cast<const float4 *>(qh + i);
-            sa[h] = fmaf(fa[i], w.x, fmaf(fa[i + 1], w.y, fmaf(fa[i + 2], w.z, fmaf(fa[i + 3], w.w, sa[h]))));
-            sb[h] = fmaf(fb[i], w.x, fmaf(fb[i + 1], w.y, fmaf(fb[i + 2], w.z, fmaf(fb[i + 3], w.w, sb[h]))));
+          for (int e = 0; e < P; e += 4) {
+            const float4 w = *reinterpret_cast<const float4 *>(qh + e * pieces);
+#pragma unroll
+            for (int i = 0; i < BATCHES; ++i)
+              sum[i][h] = fmaf(f[i][e], w.x, fmaf(f[i][e + 1], w.y, fmaf(f[i][e + 2], w.z, fmaf(f[i][e + 3], w.w, sum[i][h]))));
           }
         }
       }
 #pragma unroll
-      for (int h = 0; h < R; ++h) {
+      for (int o = 4; o > 0; o >>= 1)
 #pragma unroll
-        for (int o = 4; o > 0; o >>= 1) {
-          sa[h] += __shfl_xor_sync(0xffffffffu, sa[h], o);
-          sb[h] += __shfl_xor_sync(0xffffffffu, sb[h], o);
-        }
-        if (sub == 0) {
-          sc[h * GA_KEYS + ja] = ja < nk ? sa[h] : -INFINITY;
-          sc[h * GA_KEYS + jb] = jb < nk ? sb[h] : -INFINITY;
-        }
+        for (int h = 0; h < R; ++h)
+#pragma unroll
+          for (int i = 0; i < BATCHES; ++i) sum[i][h] += __shfl_xor_sync(0xffffffffu, sum[i][h], o);
+      if (sub == 0) {
+#pragma unroll
+        for (int h = 0; h < R; ++h)
+#pragma unroll
+          for (int i = 0; i < BATCHES; ++i) {
+            const int j = j0w + 4 * i;
+            sc[h * GA_KEYS + j] = j < nk ? sum[i][h] : -INFINITY;
+          }
       }
     }
     constexpr int PRE = 4;  // values on their way under the softmax
@@ -280,15 +292,15 @@ grouped_rows_kernel(RowsArgs a, const T *q, const T *k_cache, const T *v_cache, 
     for (int i = 0; i < PRE; ++i)
       pre[i].load(vr + (long long)(k0 + min(vg + i * key_groups, nk - 1)) * v_ld + (summing ? vc : 0));
     __syncthreads();
-    if (wid < R) {  // weights: a lane takes two keys
-      float *s = sc + wid * GA_KEYS;
-      const float s0 = s[lane], s1 = s[lane + 32];
-      const float mn = fmaxf(m, warp_max(fmaxf(s0, s1)));
-      const float p0 = exp2f(s0 - mn), p1 = exp2f(s1 - mn), keep = exp2f(m - mn);
-      l = l * keep + warp_sum(p0 + p1);
+    if (wid < R) {  // weights: a lane takes four keys
+      float4 *s = reinterpret_cast<float4 *>(sc + wid * GA_KEYS) + lane;
+      float4 v = *s;
+      const float mn = fmaxf(m, warp_max(fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w))));
+      v = make_float4(exp2f(v.x - mn), exp2f(v.y - mn), exp2f(v.z - mn), exp2f(v.w - mn));
+      const float keep = exp2f(m - mn);
+      l = l * keep + warp_sum((v.x + v.y) + (v.z + v.w));
       m = mn;
-      s[lane] = p0;
-      s[lane + 32] = p1;
+      *s = v;
       if (lane == 0) fac[wid] = keep;
     }
     __syncthreads();
@@ -419,11 +431,10 @@ void launch_grouped_attention_rows(const GroupedAttention &at, Precision type, c
   a.q_ld = at.q_ld;
   a.cap = at.cap;
   a.out_ld = at.out_ld;
-  // enough splits for two CTAs per SM, no split without a tile of its own
+  // as many splits as keep every CTA resident (two per SM), no split without a tile of its own
   const int keys = at.span.size < b.s_cap ? at.span.size : b.s_cap, tiles = (keys + GA_KEYS - 1) / GA_KEYS;
-  const long long ctas = b.rows() * at.groups * ((a.per + 7) / 8);
-  int want = 1;
-  while (want < GA_CLUSTER && want < tiles && ctas * want < 2 * 148) want *= 2;
+  const long long ctas = b.rows() * at.groups * ((a.per + 7) / 8), room = 2 * 148 / ctas;
+  int want = room < 1 ? 1 : room > GA_CLUSTER ? GA_CLUSTER : (int)room;
   if (want > tiles) want = tiles;
   const int tiles_per = (tiles + want - 1) / want;
   a.keys_per_split = tiles_per * GA_KEYS;
