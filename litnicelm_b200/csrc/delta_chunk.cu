@@ -12,14 +12,13 @@
 //
 //   delta_prepare_kernel   per chunk and head: Q'K'^T and A, K'K'^T and L, the inverse by blocks of 32, and the
 //                          factors of a token; no chunk depends on another
-//   delta_scan_kernel      per stream, head and tile of value columns: the chunks in order. A warp owns 16 value
-//                          columns and keeps their part of S^T in registers as accumulators of mma.sync tiles,
-//                          whose layout is that of the next product's left operand: the chain
-//                          S^T K'^T -> right-hand side -> U^T -> O^T, S^T runs without leaving the warp, on tiles
-//                          of K', Q', V and the chunk's matrices that all warps share (cp.async, two stages).
-//                          Where the CTA holds a whole head the output's norm and gate follow at once.
-// (A register-resident chain on mma.sync rather than tcgen05: each product's result is the next one's operand
-// after an elementwise step, and tensor memory would put a store, a fence and a barrier between any two.)
+//   delta_scan_kernel      per stream, head and tile of value columns: the chunks in order, for the sizes that
+//                          delta_scan_tc.cu leaves (few value columns, heads beyond 128). A warp owns 16 value columns
+//                          and keeps their part of S^T in registers as accumulators of mma.sync tiles, whose layout is
+//                          that of the next product's left operand: the chain S^T K'^T -> right-hand side -> U^T ->
+//                          O^T, S^T runs without leaving the warp, on tiles of K', Q', V and the chunk's matrices that
+//                          all warps share (cp.async, two stages). Where the CTA holds a whole head the output's norm
+//                          and gate follow at once.
 #include "delta.cuh"
 
 namespace lb {
