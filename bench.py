@@ -727,7 +727,7 @@ def gobesun_design(z: dict) -> dict:
     n = z["n_layers"] * 2 // 3
     for i in range(n):
         if i % 4 == 3:
-            rot = {"dims": z["dim"], "base": 1e6, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}
+            rot = {"dims": z["dim"], "base": 5e5, "scaling": {"factor": 8.0, "original": 4096, "fast": 24.0, "slow": 2.0}}
             layers.append(formats.chunk_attention_layer(z["heads"], z["heads"] // 4, z["dim"], z["vdim"], DESIGN_PREFILL[1],
                                                         rot, ff=ff))
         else:

@@ -117,7 +117,7 @@ def plain_delta(x, eps, heads, groups, dim, vdim, round_conv=False):
 
 DELTA_SHAPES = [  # streams, n, heads, groups, dim, vdim, taps
     (1, 1, 1, 1, 16, 16, 1),
-    (2, 9, 4, 2, 32, 64, 4),
+    (2, 9, 6, 3, 48, 80, 3),
     (1, 70, 3, 1, 20, 28, 2),
     (3, 64, 2, 2, 48, 16, 3),
     (1, 200, 2, 1, 64, 128, 4),
